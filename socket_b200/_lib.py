@@ -1,6 +1,6 @@
-"""ctypes binding of the C-ABI library `libsocket_b200.so` (declared in
-`include/socket_b200.h`).  There is no fallback: if the library is missing, importing an
-operator raises."""
+"""ctypes binding of the C-ABI libraries `libsocket_b200.so` (declared in `include/socket_b200.h`)
+and `libsocket_b200_blocks.so` (`include/socket_b200_blocks.h`).  There is no fallback: if a library
+is missing, calling one of its operators raises."""
 from __future__ import annotations
 
 import ctypes as C
@@ -10,6 +10,7 @@ import torch
 
 _PKG = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_PKG, "libsocket_b200.so")
+BLOCKS_PATH = os.path.join(_PKG, "libsocket_b200_blocks.so")
 
 SK_F32, SK_BF16, SK_F16 = 0, 1, 2
 DTYPE_CODE = {torch.float32: SK_F32, torch.bfloat16: SK_BF16, torch.float16: SK_F16}
@@ -92,24 +93,103 @@ SIGNATURES = {
     "sk_decode_step": (_i, [C.POINTER(DecodeParams), _p]),
 }
 
-_lib = None
+
+class ResidualParams(C.Structure):
+    """Mirror of `sk_residual_params`."""
+    _fields_ = [
+        ("x", _p), ("y", _p), ("w_in", _p), ("x0", _p), ("w_out", _p), ("out", _p),
+        ("rows", _i64), ("y_ld", _i64),
+        ("width", _i), ("in_mode", _i), ("out_mode", _i), ("dtype", _i), ("y_dtype", _i), ("eps", _f),
+    ]
 
 
-def lib() -> C.CDLL:
-    """The loaded library.  Raises if it has not been built (`python -m socket_b200.build`)."""
-    global _lib
-    if _lib is None:
-        if not os.path.exists(LIB_PATH):
-            raise SocketError(
-                f"{LIB_PATH} is missing: build it with `python -m socket_b200.build` "
-                "(there is no fallback implementation)")
-        handle = C.CDLL(LIB_PATH)
-        for name, (res, args) in SIGNATURES.items():
+class AttnParams(C.Structure):
+    """Mirror of `sk_attn_params`."""
+    _fields_ = [
+        ("q", _p), ("k", _p), ("v", _p), ("out", _p), ("bias", _p), ("sink", _p), ("pos", _p), ("status", _p),
+        ("workspace", _p), ("workspace_bytes", _sz),
+        ("q_bs", _i64), ("q_ss", _i64), ("q_hs", _i64), ("k_bs", _i64), ("k_ts", _i64), ("k_hs", _i64),
+        ("v_bs", _i64), ("v_ts", _i64), ("v_hs", _i64), ("o_bs", _i64), ("o_ss", _i64), ("o_hs", _i64),
+        ("start", _i64), ("kv_start", _i64), ("kv_rows", _i64), ("bias_len", _i64),
+        ("dtype", _i), ("B", _i), ("S", _i), ("H", _i), ("G", _i), ("dqk", _i), ("dv", _i), ("chunk", _i),
+        ("ring", _i), ("path", _i), ("scale", _f),
+    ]
+
+
+class LatentParams(C.Structure):
+    """Mirror of `sk_latent_params`."""
+    _fields_ = [
+        ("dkv", _p), ("q", _p), ("norm_w", _p), ("angles", _p), ("cache", _p), ("pos", _p), ("status", _p),
+        ("dkv_ld", _i64), ("q_ld", _i64), ("cap", _i64), ("cache_ld", _i64), ("start", _i64),
+        ("dtype", _i), ("B", _i), ("S", _i), ("H", _i), ("dim", _i), ("rot", _i), ("rot_dims", _i), ("rank", _i),
+        ("eps", _f),
+    ]
+
+
+class SsmParams(C.Structure):
+    """Mirror of `sk_ssm_params`."""
+    _fields_ = [
+        ("xbc_in", _p), ("dt_in", _p), ("conv_w", _p), ("conv_b", _p), ("conv_state", _p), ("xbc", _p), ("y", _p),
+        ("dt_bias", _p), ("A_log", _p), ("D", _p), ("state", _p), ("pos", _p),
+        ("workspace", _p), ("workspace_bytes", _sz), ("in_ld", _i64), ("xbc_ld", _i64), ("start", _i64),
+        ("dtype", _i), ("B", _i), ("S", _i), ("H", _i), ("P", _i), ("N", _i), ("G", _i), ("taps", _i), ("path", _i),
+    ]
+
+
+# the building-block library, in the order of include/socket_b200_blocks.h
+BLOCK_SIGNATURES = {
+    "skb_abi_version": (_i, []),
+    "skb_status_string": (C.c_char_p, [_i]),
+    "skb_last_error": (C.c_char_p, []),
+    "skb_embed_rows": (_i, [_p, _p, _i, _i64, _i64, _i, _f, _p, _p, _p, _p]),
+    "skb_residual_norm": (_i, [C.POINTER(ResidualParams), _p]),
+    "skb_glu_clamped": (_i, [_p, _i, _i64, _i, _i64, _f, _f, _p, _p]),
+    "skb_ring_append": (_i, [_p, _p, _i, _i, _i, _i64, _i64, _i64, _i64, _i, _i, _i, _p, _i64, _p, _p, _p]),
+    "skb_attn_workspace_bytes": (_sz, [C.POINTER(AttnParams)]),
+    "skb_attn": (_i, [C.POINTER(AttnParams), _p]),
+    "skb_attn_path": (_i, [C.POINTER(AttnParams)]),
+    "skb_latent_append": (_i, [C.POINTER(LatentParams), _p]),
+    "skb_latent_absorb": (_i, [_p, _i64, _i, _p, _i64, _i, _i, _i, _i, _i, _p, _p]),
+    "skb_latent_up": (_i, [_p, _i, _p, _i64, _i, _i, _i, _p, _p]),
+    "skb_ssm_conv": (_i, [C.POINTER(SsmParams), _p]),
+    "skb_ssm_workspace_bytes": (_sz, [C.POINTER(SsmParams)]),
+    "skb_ssm_scan": (_i, [C.POINTER(SsmParams), _p]),
+    "skb_ssm_path": (_i, [C.POINTER(SsmParams)]),
+    "skb_gated_group_norm": (_i, [_p, _p, _i64, _p, _i, _i64, _i, _i, _f, _p, _p]),
+}
+
+_handles = {}
+
+
+def _load(path: str, library: str, signatures) -> C.CDLL:
+    handle = _handles.get(path)
+    if handle is None:
+        if not os.path.exists(path):
+            raise SocketError(f"{path} is missing: build it with `python -m socket_b200.build {library}` "
+                              "(there is no fallback implementation)")
+        handle = C.CDLL(path)
+        for name, (res, args) in signatures.items():
             fn = getattr(handle, name)
             fn.restype = res
             fn.argtypes = args
-        _lib = handle
-    return _lib
+        _handles[path] = handle
+    return handle
+
+
+def lib() -> C.CDLL:
+    """The sparse-attention step's library.  Raises if it has not been built (`python -m socket_b200.build`)."""
+    return _load(LIB_PATH, "step", SIGNATURES)
+
+
+def blocks() -> C.CDLL:
+    """The decoder building blocks' library."""
+    return _load(BLOCKS_PATH, "blocks", BLOCK_SIGNATURES)
+
+
+def check_blocks(status: int, what: str) -> None:
+    if status != 0:
+        l = blocks()
+        raise SocketError(f"{what}: {l.skb_status_string(status).decode()} — {l.skb_last_error().decode()}")
 
 
 def check(status: int, what: str) -> None:

@@ -1,60 +1,10 @@
 // extern "C" entry points: argument validation, workspace carving, kernel launches.
-#include <atomic>
-#include <cstdarg>
-#include <cstdio>
 #include <cstdlib>
 #include <cstring>
 
-#include "common.cuh"
+#include "abi_check.cuh"
 
 namespace sk {
-
-static thread_local char g_err[512] = "";
-static thread_local int g_pdl_depth = 0;
-
-bool pdl_chain_active() {
-    static const bool off = getenv("SOCKET_B200_NO_PDL") != nullptr;   // debugging aid: launch the step's kernels unchained
-    return g_pdl_depth > 0 && !off;
-}
-PdlChain::PdlChain() { ++g_pdl_depth; }
-PdlChain::~PdlChain() { --g_pdl_depth; }
-
-int fail(int status, const char* fmt, ...) {
-    va_list ap;
-    va_start(ap, fmt);
-    vsnprintf(g_err, sizeof(g_err), fmt, ap);
-    va_end(ap);
-    return status;
-}
-
-int sm_count() {
-    constexpr int MAX_DEV = 64;
-    static std::atomic<int> cached[MAX_DEV];
-    int dev = -1;
-    if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= MAX_DEV) {
-        cudaGetLastError();   // a size query without a device is not an error of the next launch
-        return 148;
-    }
-    int n = cached[dev].load(std::memory_order_relaxed);
-    if (n > 0) return n;
-    if (cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || n <= 0) {
-        cudaGetLastError();
-        return 148;
-    }
-    cached[dev].store(n, std::memory_order_relaxed);
-    return n;
-}
-
-int check_launch(const char* what) {
-    cudaError_t e = cudaGetLastError();
-    if (e != cudaSuccess) return fail(SK_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
-    return SK_OK;
-}
-
-static inline bool aligned(const void* p, size_t a) { return (reinterpret_cast<uintptr_t>(p) % a) == 0; }
-static inline bool valid_dtype(int d) { return d == SK_F32 || d == SK_BF16 || d == SK_F16; }
-static inline size_t esize(int d) { return d == SK_F32 ? 4 : 2; }
-static inline size_t up256(size_t x) { return (x + 255) & ~(size_t)255; }
 
 static int64_t list_len_host(int64_t T, int sink, int window, int64_t M) {
     if (T <= 0) return 0;
@@ -73,32 +23,13 @@ static int64_t list_len_host(int64_t T, int sink, int window, int64_t M) {
 
 using namespace sk;
 
-#define SK_REQUIRE(cond, ...)                                          \
-    do {                                                               \
-        if (!(cond)) return fail(SK_ERR_INVALID_ARGUMENT, __VA_ARGS__); \
-    } while (0)
-#define SK_ALIGNED(ptr, a, name)                                                         \
-    do {                                                                                 \
-        if (!aligned(ptr, a)) return fail(SK_ERR_MISALIGNED, name " must be %d-byte aligned", (int)(a)); \
-    } while (0)
-
 extern "C" {
 
 int sk_abi_version(void) { return SK_ABI_VERSION; }
 
-const char* sk_status_string(int status) {
-    switch (status) {
-        case SK_OK: return "ok";
-        case SK_ERR_INVALID_ARGUMENT: return "invalid argument";
-        case SK_ERR_UNSUPPORTED: return "unsupported shape or dtype";
-        case SK_ERR_MISALIGNED: return "misaligned pointer or stride";
-        case SK_ERR_WORKSPACE: return "workspace too small";
-        case SK_ERR_CUDA: return "CUDA runtime error";
-        default: return "unknown status";
-    }
-}
+const char* sk_status_string(int status) { return status_string(status); }
 
-const char* sk_last_error(void) { return g_err; }
+const char* sk_last_error(void) { return last_error(); }
 
 int sk_hash_keys(const void* keys, int key_dtype, int64_t key_row_stride, const void* planes,
                  int plane_dtype, int64_t N, int D, int L, int P, void* codes, int code_bytes,

@@ -15,6 +15,8 @@ constexpr unsigned FULL = 0xffffffffu;
 // ---------------------------------------------------------------- host error plumbing
 int fail(int status, const char* fmt, ...);       // records a thread-local message
 int check_launch(const char* what);               // cudaGetLastError -> SK_ERR_CUDA
+const char* last_error();
+const char* status_string(int status);
 // Streaming multiprocessors of the current device (queried once per device; 148, the B200 count,
 // when no device can be asked, e.g. a size query on a machine without a GPU).
 int sm_count();

@@ -1,0 +1,212 @@
+// Everything between two matrix products that touches the fp32 residual stream: the scaled embedding,
+// the residual update with a norm on the sublayer's output fused with the norm of the next sublayer's
+// input, and the clamped gated unit of the feed-forward.
+#include "blocks.cuh"
+
+namespace sk {
+namespace {
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+embed_rows_kernel(const int64_t* __restrict__ tokens, const T* __restrict__ table, int64_t vocab, int width, float scale,
+                  float* __restrict__ x, float* __restrict__ x_copy, int32_t* status) {
+    const int64_t row = blockIdx.x;
+    const int64_t tok = tokens[row];
+    const bool ok = tok >= 0 && tok < vocab;              // outside the table: flagged, the row reads zero
+    if (!ok && threadIdx.x == 0 && status != nullptr) atomicOr(status, SK_DEV_INDEX_OUT_OF_RANGE);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = ok ? to_f32(table[tok * width + i]) * scale : 0.f;
+        x[row * width + i] = v;
+        if (x_copy != nullptr) x_copy[row * width + i] = v;
+    }
+}
+
+// One CTA per row; the row lives in registers (NV vectors of V elements per thread).
+//   in_mode  0: x stays; 1: x += rms(y) * w_in; 2: x = y + w_in
+//   out_mode 0: nothing; 1: out = rms(x) * w_out; 2: out = [x ; x0]
+template <typename T, typename TY, int V, int NV>
+__global__ void __launch_bounds__(1024)
+residual_norm_kernel(sk_residual_params p) {
+    __shared__ float red[2][32];
+    const int64_t row = blockIdx.x;
+    const int W = p.width, nt = blockDim.x, t = threadIdx.x;
+    float* xr = p.x + row * W;
+    const T* w_in = (const T*)p.w_in;
+    const T* w_out = (const T*)p.w_out;
+    float xv[NV][V];
+    if (p.in_mode != 0) {
+        const TY* yr = (const TY*)p.y + row * p.y_ld;
+        float yv[NV][V], ss = 0.f;
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int i = (n * nt + t) * V;
+            if (i < W) {
+                load_vec<TY, V>(yr + i, yv[n]);
+                if (p.in_mode == 1) load_vec<float, V>(xr + i, xv[n]);
+#pragma unroll
+                for (int e = 0; e < V; ++e) ss = fmaf(yv[n][e], yv[n][e], ss);
+            }
+        }
+        float inv = 1.f;
+        if (p.in_mode == 1) inv = 1.f / sqrtf(block_sum(ss, red[0]) / (float)W + p.eps);
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int i = (n * nt + t) * V;
+            if (i < W) {
+                float w[V];
+                load_vec<T, V>(w_in + i, w);
+#pragma unroll
+                for (int e = 0; e < V; ++e)
+                    xv[n][e] = p.in_mode == 1 ? xv[n][e] + yv[n][e] * inv * w[e] : yv[n][e] + w[e];
+                store_vec<float, V>(xr + i, xv[n]);
+            }
+        }
+    } else {
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int i = (n * nt + t) * V;
+            if (i < W) load_vec<float, V>(xr + i, xv[n]);
+        }
+    }
+    if (p.out_mode == 1) {
+        float ss = 0.f;
+#pragma unroll
+        for (int n = 0; n < NV; ++n)
+            if ((n * nt + t) * V < W)
+#pragma unroll
+                for (int e = 0; e < V; ++e) ss = fmaf(xv[n][e], xv[n][e], ss);
+        const float inv = 1.f / sqrtf(block_sum(ss, red[1]) / (float)W + p.eps);
+        T* o = (T*)p.out + row * W;
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int i = (n * nt + t) * V;
+            if (i < W) {
+                float w[V], r[V];
+                load_vec<T, V>(w_out + i, w);
+#pragma unroll
+                for (int e = 0; e < V; ++e) r[e] = xv[n][e] * inv * w[e];
+                store_vec<T, V>(o + i, r);
+            }
+        }
+    } else if (p.out_mode == 2) {
+        T* o = (T*)p.out + row * 2 * W;
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int i = (n * nt + t) * V;
+            if (i < W) {
+                float r[V];
+                load_vec<float, V>(p.x0 + row * W + i, r);
+                store_vec<T, V>(o + i, xv[n]);
+                store_vec<T, V>(o + W + i, r);
+            }
+        }
+    }
+}
+
+// gate_up row = [gate | up]: y = g * sigmoid(slope * g) * (u + 1), g and u clamped
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+glu_clamped_kernel(const T* __restrict__ gu, int64_t n_vec, int ff, int64_t ld, float limit, float slope,
+                   T* __restrict__ out) {
+    const int per_row = ff / V;
+    for (int64_t j = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; j < n_vec; j += (int64_t)gridDim.x * blockDim.x) {
+        const int64_t row = j / per_row;
+        const int i = (int)(j - row * per_row) * V;
+        float g[V], u[V], r[V];
+        load_vec<T, V>(gu + row * ld + i, g);
+        load_vec<T, V>(gu + row * ld + ff + i, u);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+            const float a = fminf(g[e], limit), b = fminf(fmaxf(u[e], -limit), limit);
+            r[e] = a / (1.f + expf(-slope * a)) * (b + 1.f);
+        }
+        store_vec<T, V>(out + row * ff + i, r);
+    }
+}
+
+// The newest tokens of a portion into a ring of `ring` rows (row of position p: p % ring).  Only the
+// positions of the last block of `ring` positions are written: earlier ones are not visible any more,
+// and no two tokens of a portion meet in one row.
+template <typename T>
+__global__ void __launch_bounds__(256)
+ring_append_kernel(const T* __restrict__ k, const T* __restrict__ v, int64_t k_bs, int64_t k_ss, int64_t v_bs,
+                   int64_t v_ss, int k_row, int v_row, int ring, const int64_t* __restrict__ pos, int64_t start, int s0,
+                   T* __restrict__ k_cache, T* __restrict__ v_cache) {
+    const int s = s0 + blockIdx.x, b = blockIdx.y;
+    const int64_t slot = (first_position(pos, start) + s) % ring;
+    const T* ks = k + b * k_bs + s * k_ss;
+    const T* vs = v + b * v_bs + s * v_ss;
+    T* kd = k_cache + ((int64_t)b * ring + slot) * k_row;
+    T* vd = v_cache + ((int64_t)b * ring + slot) * v_row;
+    for (int i = threadIdx.x; i < k_row; i += blockDim.x) kd[i] = ks[i];
+    for (int i = threadIdx.x; i < v_row; i += blockDim.x) vd[i] = vs[i];
+}
+
+template <typename T, typename TY, int V>
+int residual_dispatch(const sk_residual_params& p, cudaStream_t st) {
+    const int vecs = (p.width + V - 1) / V;
+    // few rows: one vector per thread (latency); many rows: smaller blocks, more of them per SM
+    int nt = p.rows < 296 ? 1024 : 256;
+    while (nt > 32 && nt / 2 >= vecs) nt /= 2;
+    while (nt < 1024 && (vecs + nt - 1) / nt > 8) nt *= 2;
+    const int nv = (vecs + nt - 1) / nt;
+    dim3 grid((unsigned)p.rows);
+    if (nv <= 1) residual_norm_kernel<T, TY, V, 1><<<grid, nt, 0, st>>>(p);
+    else if (nv <= 2) residual_norm_kernel<T, TY, V, 2><<<grid, nt, 0, st>>>(p);
+    else if (nv <= 4) residual_norm_kernel<T, TY, V, 4><<<grid, nt, 0, st>>>(p);
+    else if (nv <= 8) residual_norm_kernel<T, TY, V, 8><<<grid, nt, 0, st>>>(p);
+    else return fail(SK_ERR_UNSUPPORTED, "sk_residual_norm: width %d is too large", p.width);
+    return check_launch("residual_norm_kernel");
+}
+
+}  // namespace
+
+int launch_embed_rows(const int64_t* tokens, const void* table, int dtype, int64_t rows, int64_t vocab, int width,
+                      float scale, float* x, float* x_copy, int32_t* status, cudaStream_t st) {
+    if (dtype == SK_BF16)
+        embed_rows_kernel<<<(unsigned)rows, 256, 0, st>>>(tokens, (const __nv_bfloat16*)table, vocab, width, scale, x,
+                                                          x_copy, status);
+    else
+        embed_rows_kernel<<<(unsigned)rows, 256, 0, st>>>(tokens, (const float*)table, vocab, width, scale, x, x_copy,
+                                                          status);
+    return check_launch("embed_rows_kernel");
+}
+
+int launch_residual_norm(const sk_residual_params& p, cudaStream_t st) {
+    const bool v4 = p.width % 4 == 0 && p.y_ld % 4 == 0;
+    if (p.dtype == SK_F32) return v4 ? residual_dispatch<float, float, 4>(p, st) : residual_dispatch<float, float, 1>(p, st);
+    using bf = __nv_bfloat16;
+    if (p.y_dtype == SK_F32) return v4 ? residual_dispatch<bf, float, 4>(p, st) : residual_dispatch<bf, float, 1>(p, st);
+    return v4 ? residual_dispatch<bf, bf, 4>(p, st) : residual_dispatch<bf, bf, 1>(p, st);
+}
+
+int launch_glu_clamped(const void* gate_up, int dtype, int64_t rows, int ff, int64_t ld, float limit, float slope,
+                       void* out, cudaStream_t st) {
+    const bool v4 = ff % 4 == 0 && ld % 4 == 0;
+    const int64_t n = rows * (v4 ? ff / 4 : ff);
+    int64_t blocks = (n + 255) / 256;
+    if (blocks > (int64_t)sm_count() * 16) blocks = (int64_t)sm_count() * 16;
+#define SK_GLU(T, V) glu_clamped_kernel<T, V><<<(unsigned)blocks, 256, 0, st>>>((const T*)gate_up, n, ff, ld, limit, slope, (T*)out)
+    if (dtype == SK_BF16) { if (v4) SK_GLU(__nv_bfloat16, 4); else SK_GLU(__nv_bfloat16, 1); }
+    else { if (v4) SK_GLU(float, 4); else SK_GLU(float, 1); }
+#undef SK_GLU
+    return check_launch("glu_clamped_kernel");
+}
+
+int launch_ring_append(const void* k, const void* v, int dtype, int B, int S, int64_t k_bs, int64_t k_ss, int64_t v_bs,
+                       int64_t v_ss, int k_row, int v_row, int ring, const int64_t* pos, int64_t start, void* k_cache,
+                       void* v_cache, cudaStream_t st) {
+    const int64_t first = (start + S - 1) / ring * ring;       // first position of the last block
+    const int s0 = pos == nullptr && first > start ? (int)(first - start) : 0;   // a device position: one token
+    dim3 grid((unsigned)(S - s0), (unsigned)B);
+    if (dtype == SK_BF16)
+        ring_append_kernel<<<grid, 256, 0, st>>>((const __nv_bfloat16*)k, (const __nv_bfloat16*)v, k_bs, k_ss, v_bs, v_ss,
+                                                 k_row, v_row, ring, pos, start, s0, (__nv_bfloat16*)k_cache,
+                                                 (__nv_bfloat16*)v_cache);
+    else
+        ring_append_kernel<<<grid, 256, 0, st>>>((const float*)k, (const float*)v, k_bs, k_ss, v_bs, v_ss, k_row, v_row,
+                                                 ring, pos, start, s0, (float*)k_cache, (float*)v_cache);
+    return check_launch("ring_append_kernel");
+}
+
+}  // namespace sk

@@ -33,11 +33,8 @@ from torch import Tensor
 
 from . import ops, tp
 from .attention import KVCache
+from .decoder import Decoder, find_multiple, generate  # noqa: F401  (generate: the public entry point)
 from .synth import hypercube_protos
-
-
-def find_multiple(n: int, k: int) -> int:
-    return n if n % k == 0 else n + k - (n % k)
 
 
 @dataclass
@@ -289,10 +286,13 @@ class TransformerBlock(nn.Module):
         return h + self._sum(self.feed_forward(self.ffn_norm(h)))
 
 
-class Transformer(nn.Module):
+class Transformer(Decoder):
     """`world` / `rank`: tensor-parallel layout; every rank builds its own shard (random
     initialisation draws the FULL matrices from one seed and keeps the rank's block, so that the
     ranks together hold exactly the single-GPU model; see `shard_like_reference`)."""
+
+    default_mode = "sparse"
+    libraries = ("step",)
 
     def __init__(self, config: ModelArgs, world: int = 1, rank: int = 0):
         super().__init__()
@@ -302,10 +302,12 @@ class Transformer(nn.Module):
         self.norm = RMSNorm(config.dim, eps=config.norm_eps)
         self.output = nn.Linear(config.dim, config.vocab_size, bias=False)
         self.register_buffer("freqs_cis", None, persistent=False)
-        self.max_batch_size = self.max_seq_length = -1
-        self._graph = None
         self.tp_fused = True                       # decode: fuse wo / w2 with the sum over the ranks (GPU, <= 8 rows)
         self._fused_sum = None
+
+    @property
+    def embedding_table(self) -> Tensor:
+        return self.tok_embeddings.weight
 
     @torch.no_grad()
     def init_random(self, seed: int = 0, std: float = 0.02) -> "Transformer":
@@ -325,65 +327,56 @@ class Transformer(nn.Module):
             blk.attention.planes.copy_(torch.randn(blk.attention.planes.shape, generator=g, device=dev))
         return self
 
-    def setup_caches(self, max_batch_size: int, max_seq_length: int) -> None:
+    @torch.no_grad()
+    def load_tensors(self, tensors) -> None:
+        """Checkpoint tensors, named as in `state_dict()` (hash planes and prototypes included)."""
+        own = {k: v for k, v in self.state_dict().items() if ".kv_cache." not in k}
+        if set(own) != set(tensors):
+            raise ValueError(f"checkpoint does not fit the model: {sorted(set(own) ^ set(tensors))[:8]}")
+        for name, dst in own.items():
+            if dst.shape != tensors[name].shape:
+                raise ValueError(f"{name}: {tuple(tensors[name].shape)} in the checkpoint, {tuple(dst.shape)} in the model")
+            dst.copy_(tensors[name])
+
+    def _alloc_caches(self, batch: int, length: int) -> None:
         """Per-layer caches (K, V, bucket codes, value norms) and the rotary table; as
         GPT-FAST/model.py:251-278 minus the T x T mask."""
-        if self.max_seq_length >= max_seq_length and self.max_batch_size >= max_batch_size:
-            return
-        dev, dt = self.tok_embeddings.weight.device, self.tok_embeddings.weight.dtype
-        max_seq_length = find_multiple(max_seq_length, 8)
-        self.max_seq_length, self.max_batch_size = max_seq_length, max_batch_size
         for b in self.layers:
             a = b.attention
-            a.kv_cache = KVCache(max_batch_size, max_seq_length, a.n_local_heads, a.head_dim, L=a.L, R=a.R,
-                                 dtype=dt, device=dev)
-        self.freqs_cis = precompute_freqs_cis(min(self.config.block_size, max_seq_length), self.config.head_dim,
-                                              self.config.rope_base, device=dev)
-        self._graph = None
+            a.kv_cache = KVCache(batch, length, a.n_local_heads, a.head_dim, L=a.L, R=a.R, dtype=self.dtype,
+                                 device=self.device)
+        self.freqs_cis = precompute_freqs_cis(min(self.config.block_size, length), self.config.head_dim,
+                                              self.config.rope_base, device=self.device)
 
     # ------------------------------------------------------------------------------- prefill
-    @torch.no_grad()
-    def prefill(self, idx: Tensor, chunk: int = 8192) -> Tensor:
-        """idx [B,T] prompt token ids -> logits of the last position [B,vocab].  The prompt is
-        processed `chunk` tokens at a time: each chunk's keys are appended to the caches (hashed on
-        the tensor cores) and its queries attend causally over everything cached so far."""
-        B, T = idx.shape
-        assert T <= self.max_seq_length and B <= self.max_batch_size
-        x_last = None
-        for s0 in range(0, T, chunk):
-            s1 = min(T, s0 + chunk)
-            pos = torch.arange(s0, s1, device=idx.device)
-            x = self.tok_embeddings(idx[:, s0:s1])
-            fc = self.freqs_cis[s0:s1]
-            for layer in self.layers:
-                x = layer.prefill(x, fc, pos, s0)
-            x_last = x[:, -1]
-        return self.output(self.norm(x_last))
+    def _portion(self, idx: Tensor, start: int) -> Tensor:
+        """Each portion's keys are appended to the caches (hashed on the tensor cores) and its queries
+        attend causally over everything cached so far."""
+        end = start + idx.shape[1]
+        pos = torch.arange(start, end, device=idx.device)
+        x = self.tok_embeddings(idx)
+        fc = self.freqs_cis[start:end]
+        for layer in self.layers:
+            x = layer.prefill(x, fc, pos, start)
+        return x
+
+    def _head(self, hidden: Tensor) -> Tensor:
+        return self.output(self.norm(hidden))
 
     # ------------------------------------------------------------------------------- decode
-    def _decode_body(self, mode: str) -> None:
+    def _decode_logits(self, mode: str) -> Tensor:
         x = self.tok_embeddings(self._tok)                      # [B,1,dim]
         fc = None if x.is_cuda else self.freqs_cis[self._pos]   # [1,D/2,2]
         for layer in self.layers:
             x = layer.decode(x, fc, self._pos, self._seqlens, mode, self.freqs_cis)
-        logits = self.output(self.norm(x))[:, -1]
-        self._tok.copy_(torch.argmax(logits, dim=-1, keepdim=True))
-        self._pos.add_(1)
-        self._seqlens.add_(1)
+        return self.output(self.norm(x))[:, -1]
 
-    @torch.no_grad()
-    def setup_decode(self, batch: int, mode: str = "sparse", use_graph: bool = True) -> None:
-        """Allocate the decode-time buffers (current token, position, per-layer q/k/v staging,
-        the per-layer fused steps) and, on a GPU, capture one token's work in a CUDA graph."""
-        dev = self.tok_embeddings.weight.device
-        self._mode = mode
-        self._tok = torch.zeros(batch, 1, dtype=torch.long, device=dev)
-        self._pos = torch.zeros(1, dtype=torch.long, device=dev)
-        self._seqlens = torch.zeros(batch, dtype=torch.int32, device=dev)
+    def _setup_decode_layers(self, batch: int, mode: str) -> None:
+        dev = self.device
         for layer in self.layers:
             layer.attention.setup_decode(batch, self._pos, mode)
         if self.world > 1 and dev.type == "cuda" and self.tp_fused and batch <= 8 and \
-                self.tok_embeddings.weight.dtype in (torch.bfloat16, torch.float16) and \
+                self.dtype in (torch.bfloat16, torch.float16) and \
                 (self.config.dim + 63) // 64 <= torch.cuda.get_device_properties(dev).multi_processor_count:
             if self._fused_sum is None or self._fused_sum.max_batch < batch:
                 self._fused_sum = tp.FusedRowParallel(self.config.dim, max(batch, 1), dev)
@@ -392,106 +385,13 @@ class Transformer(nn.Module):
         else:
             for layer in self.layers:
                 layer.fused_sum = None
-        self._graph = None
-        self._host_pos = 0
-        if use_graph and dev.type == "cuda":
-            saved = (self._tok.clone(), self._pos.clone(), self._seqlens.clone())
-            side = torch.cuda.Stream(dev)
-            side.wait_stream(torch.cuda.current_stream(dev))
-            with torch.cuda.stream(side):
-                # position 0 of every cache is overwritten by this dry run and by the capture;
-                # decoding starts only after `start_decode`, which the caller follows with real tokens
-                self._decode_body(mode)
-                side.synchronize()
-                g = torch.cuda.CUDAGraph()
-                with torch.cuda.graph(g, stream=side):
-                    self._decode_body(mode)
-            torch.cuda.current_stream(dev).wait_stream(side)
-            self._graph = g
-            self._tok.copy_(saved[0]); self._pos.copy_(saved[1]); self._seqlens.copy_(saved[2])
 
-    def release_decode(self) -> None:
-        """Drop the captured graph and the per-layer steps.  Under tensor parallelism call this
-        before `torch.distributed.destroy_process_group()`: a live CUDA graph that holds NCCL
-        kernels keeps the communicator busy and the teardown waits for it."""
-        self._graph = None
+    def _release_decode_layers(self) -> None:
         for layer in self.layers:
             layer.attention._step = None
             layer.fused_sum = None
-        if self.tok_embeddings.weight.is_cuda:
-            torch.cuda.synchronize(self.tok_embeddings.weight.device)
 
-    @torch.no_grad()
-    def start_decode(self, first_token: Tensor, position: int) -> None:
-        """`first_token` [B,1] sits at `position` (= number of tokens already cached)."""
-        if position >= self.max_seq_length:
-            raise RuntimeError(f"start_decode: position {position} outside the caches (max_seq_length="
-                               f"{self.max_seq_length})")
-        self._host_pos = position                 # host mirror of the device-side position counter
-        self._tok.copy_(first_token)
-        self._pos.fill_(position)
-        self._seqlens.fill_(position)
+    def _start_decode_layers(self, position: int) -> None:
         if self._mode == "sparse":
             for layer in self.layers:
                 layer.attention.kv_cache.prefill_len.fill_(position)
-
-    @torch.no_grad()
-    def decode_one_token(self) -> Tensor:
-        """Runs one token through the model (greedy); returns the buffer holding the new token.
-        Raises before anything is launched when the caches are full (same situation as the
-        reference's `_check_input_pos`, GPT-FAST/model.py:279-289, without its device round trip)."""
-        if self._host_pos >= self.max_seq_length:
-            raise RuntimeError(f"decode position {self._host_pos} outside the caches (max_seq_length="
-                               f"{self.max_seq_length}); call setup_caches with a larger length")
-        self._host_pos += 1
-        if self._graph is not None:
-            self._graph.replay()
-        else:
-            self._decode_body(self._mode)
-        return self._tok
-
-
-@torch.no_grad()
-def generate(model: Transformer, prompt: Tensor, max_new_tokens: int, mode: str = "sparse",
-             prefill_chunk: int = 8192, use_graph: bool = True, stream_to_host: bool = False):
-    """Greedy generation as GPT-FAST/generate.py:246-370: prefill the prompt, take the first new
-    token from the prefill logits, then `max_new_tokens - 1` decode steps.  Returns (tokens
-    [B, T + max_new_tokens], stats) with `decode_time_s` measured by CUDA events around the decode
-    loop and `decode_only_tokens = B * (max_new_tokens - 1)` (generate.py:362-368).  `prompt` may be
-    a host tensor; with `stream_to_host` every new token is copied to pinned host memory and waited
-    for before the next step is launched (the end-to-end serving pattern)."""
-    dev = model.tok_embeddings.weight.device
-    B, T = prompt.shape
-    prompt_d = prompt.to(dev, non_blocking=True)
-    model.setup_caches(B, T + max_new_tokens + 8)
-    cuda = dev.type == "cuda"
-    e = [torch.cuda.Event(enable_timing=True) for _ in range(4)] if cuda else None
-    # the decode graph's dry run scribbles on cache position 0: capture before the prefill
-    model.setup_decode(B, mode, use_graph)
-    if cuda:
-        e[0].record()
-    logits = model.prefill(prompt_d, chunk=prefill_chunk)
-    first = torch.argmax(logits, dim=-1, keepdim=True)
-    if cuda:
-        e[1].record()
-    seq = torch.empty(B, T + max_new_tokens, dtype=torch.long, device=dev)
-    seq[:, :T] = prompt_d
-    seq[:, T] = first[:, 0]
-    model.start_decode(first, T)
-    host_tok = torch.empty(B, 1, dtype=torch.long).pin_memory() if (cuda and stream_to_host) else None
-    if cuda:
-        torch.cuda.synchronize(dev)
-        e[2].record()
-    for i in range(1, max_new_tokens):
-        tok = model.decode_one_token()
-        seq[:, T + i] = tok[:, 0]
-        if host_tok is not None:
-            host_tok.copy_(tok, non_blocking=True)
-            torch.cuda.current_stream(dev).synchronize()
-    stats = {"decode_only_tokens": B * max(0, max_new_tokens - 1)}
-    if cuda:
-        e[3].record()
-        torch.cuda.synchronize(dev)
-        stats["prefill_time_s"] = e[0].elapsed_time(e[1]) / 1e3
-        stats["decode_time_s"] = e[2].elapsed_time(e[3]) / 1e3
-    return seq, stats
