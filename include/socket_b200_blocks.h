@@ -75,7 +75,7 @@ SK_API int skb_ring_append(const void* k, const void* v, int dtype, int B, int S
  * key row, _hs head; the last dimension is contiguous.  Key row r holds position kv_start + r, or,
  * with ring != 0, position floor(i / chunk) * chunk + r (one token per call).  kv_rows rows exist.
  * `path`: SKB_ATTN_AUTO picks the kernel, the others pin one (SK_ERR_UNSUPPORTED outside its shapes).
- * `workspace` (skb_attn_workspace_bytes, first 64 KiB zeroed once) serves the split decode kernel. */
+ * `workspace` (skb_attn_workspace_bytes; need not be cleared) serves the split decode kernel. */
 enum { SKB_ATTN_AUTO = 0, SKB_ATTN_ROWS = 1, SKB_ATTN_PREFILL_TC = 2, SKB_ATTN_DECODE = 3 };
 typedef struct sk_attn_params {
     const void *q, *k, *v;

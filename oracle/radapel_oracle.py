@@ -198,3 +198,60 @@ def forward(tokens: List[int], weights: Dict[str, Tensor], cfg: dict, dtype=torc
         if residuals is not None:
             residuals.append(x.clone())
     return rms_norm(x, w["final.norm"], eps) @ w["head"].T
+
+
+def tensor_shapes(cfg: dict, bias_rows: int = 16) -> Dict[str, tuple]:
+    """Checkpoint names and shapes of a configuration."""
+    V, W = cfg["vocab"], cfg["width"]
+    out = {"embed": (V, W), "final.norm": (W,), "head": (V, W)}
+    if cfg.get("loop"):
+        out["loop.in"], out["loop.step"] = (W, 2 * W), (cfg["loop"]["times"], W)
+    for i, e in enumerate(cfg["layers"]):
+        m, p = e["mixer"], f"l{i}."
+        H = m["heads"]
+        out[p + "norm1"] = out[p + "norm1b"] = (W,)
+        if e["type"] == "attention":
+            mix = {"q": (H * m["dim"], W), "k": (m["kv_heads"] * m["dim"], W), "v": (m["kv_heads"] * m["vdim"], W),
+                   "rel": (bias_rows, H), "o": (W, H * m["vdim"])}
+        elif e["type"] == "latent_attention":
+            K, R = m["kv_rank"], m["rot_dim"]
+            mix = {"q": (H * (m["dim"] + R), W), "dkv": (K + R, W), "dkv.norm": (K,), "uk": (H * m["dim"], K),
+                   "uv": (H * m["vdim"], K), "sink": (H,), "o": (W, H * m["vdim"])}
+        else:
+            I, ch = H * m["vdim"], H * m["vdim"] + 2 * m["groups"] * m["state"]
+            mix = {"in": (I + ch + H, W), "conv": (ch, m["conv"]), "conv.b": (ch,), "dt_bias": (H,), "A_log": (H,),
+                   "D": (H,), "norm": (I,), "o": (W, I)}
+        out.update({p + "mix." + k: v for k, v in mix.items()})
+        if e["mlp"] is not None:
+            F = e["mlp"]["ff"]
+            out[p + "norm2"] = out[p + "norm2b"] = (W,)
+            out.update({p + "mlp.gate": (F, W), p + "mlp.up": (F, W), p + "mlp.down": (W, F)})
+    return out
+
+
+def random_weights(cfg: dict, seed: int, bias_rows: int = 16) -> Dict[str, Tensor]:
+    """bfloat16 weights at which every mechanism shows: attention scores of a few units, biases and sinks
+    that matter, decays from slow to fast, norm weights away from one."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in tensor_shapes(cfg, bias_rows).items():
+        leaf = name.split(".", 2)[-1] if name.startswith("l") and name[1].isdigit() else name
+        x = torch.randn(*shape, generator=g)
+        if leaf.endswith("norm") or leaf in ("norm1", "norm1b", "norm2", "norm2b"):
+            x = 1.0 + 0.3 * x
+        elif leaf in ("mix.q", "mix.k", "mix.dkv", "mix.uk"):
+            x = x * 1.6 / shape[-1] ** 0.5
+        elif leaf in ("mix.rel", "mix.sink"):
+            x = 1.5 * x
+        elif leaf == "mix.A_log":
+            x = 0.5 * x - 0.5
+        elif leaf == "mix.dt_bias":
+            x = x - 2.0
+        elif leaf in ("mix.D", "mix.conv.b", "embed", "loop.step"):
+            x = 0.5 * x
+        elif leaf == "mix.conv":
+            x = x / shape[-1] ** 0.5
+        else:
+            x = x / shape[-1] ** 0.5
+        out[name] = x.to(torch.bfloat16)
+    return out

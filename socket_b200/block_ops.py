@@ -127,13 +127,13 @@ def attn_params(q: Tensor, k: Tensor, v: Tensor, out: Tensor, *, scale: float, s
 
 def attn(q: Tensor, k: Tensor, v: Tensor, **kw) -> Tensor:
     """Softmax attention of a portion: q [B,S,H,dqk], k [B,rows,G,dqk], v [B,rows,G,dv] -> [B,S,H,dv].
-    Keyword arguments as in `attn_params`; without a workspace one is allocated when the kernel needs it."""
+    Keyword arguments as in `attn_params`; a workspace that is absent or too small is allocated when the kernel needs one."""
     _require_cuda(q, k, v)
     out = torch.empty(*q.shape[:3], v.shape[3], dtype=q.dtype, device=q.device)
     p = attn_params(q, k, v, out, **kw)
-    if kw.get("workspace") is None:
-        need = int(blocks().skb_attn_workspace_bytes(C.byref(p)))
-        ws = torch.zeros(need, dtype=torch.uint8, device=q.device) if need else None
+    need = int(blocks().skb_attn_workspace_bytes(C.byref(p)))
+    if need > p.workspace_bytes:
+        ws = torch.empty(need, dtype=torch.uint8, device=q.device)
         p.workspace, p.workspace_bytes = ptr(ws), need
     check_blocks(blocks().skb_attn(C.byref(p), stream_ptr(q.device)), "skb_attn")
     return out

@@ -25,7 +25,7 @@ int check_attn(const sk_attn_params* p) {
 
 int attn_path(const sk_attn_params& p) {
     if (p.path != SKB_ATTN_AUTO) return p.path;
-    if (attn_decode_mma_applicable(p) && p.S * (p.H / p.G) <= 1024 && (p.S <= 1 || p.G == 1)) return SKB_ATTN_DECODE;
+    if (p.S <= (p.G == 1 ? 32 : 1) && attn_decode_mma_applicable(p)) return SKB_ATTN_DECODE;
     if (attn_prefill_tc_applicable(p)) return SKB_ATTN_PREFILL_TC;
     return SKB_ATTN_ROWS;
 }

@@ -1,11 +1,410 @@
+// Softmax attention of one or a few query tokens against a long cache (bf16), split over the keys.
+//
+// All query rows that share a key/value head (rep heads x S tokens) are worked on together, 16 or 32 rows per
+// CTA, so a key is read once for all of them; with one key/value head for every query head - attention on
+// latent rows - this is what makes the step read each cache row once.  A CTA walks its share of 64-key tiles
+// (cp.async, double buffer), computes the scores with m16n8k16 MMAs (rows are too few for the 128-row tensor
+// core tiles), keeps the running maximum per row and accumulates P V with each warp owning a slice of the value columns.
+// When the values are a prefix of the key rows in memory, the key tile serves as the value tile.  A second kernel
+// merges the partial results of the splits.  The live length is read on the device; the grid is fixed.
 #include "blocks.cuh"
+#include "warp_mma.cuh"
+
 namespace sk {
-bool attn_decode_mma_applicable(const sk_attn_params& p) { return false; }
-size_t attn_decode_mma_workspace(const sk_attn_params& p) { return 0; }
-int launch_attn_decode_mma(const sk_attn_params& p, cudaStream_t st) { return SK_ERR_UNSUPPORTED; }
-bool attn_prefill_tc_applicable(const sk_attn_params& p) { return false; }
-int launch_attn_prefill_tc(const sk_attn_params& p, cudaStream_t st) { return SK_ERR_UNSUPPORTED; }
-bool ssm_chunks_applicable(const sk_ssm_params& p) { return false; }
-size_t ssm_chunks_workspace(const sk_ssm_params& p) { return 0; }
-int launch_ssm_chunks(const sk_ssm_params& p, cudaStream_t st) { return SK_ERR_UNSUPPORTED; }
+namespace {
+
+constexpr int DM_THREADS = 256, DM_WARPS = 8, DM_KEYS = 64;
+constexpr float DM_LOG2E = 1.4426950408889634f;
+constexpr int DM_MAX_SPLITS = 160;
+
+struct DmPlan {
+    int mt;                 // 16-row tiles per CTA
+    int nvt;                // 8-column value tiles per warp
+    int groups;             // row groups per (batch, key/value head)
+    int splits;
+    bool shared_v;
+    int k_stride, v_stride; // elements per shared-memory row
+    size_t smem;
+    size_t part_floats;     // per split: 16 mt rows x (dv + 2)
+};
+
+bool dm_plan(const sk_attn_params& p, DmPlan* d) {
+    if (p.dtype != SK_BF16 || p.dqk % 8 || p.dv % 8 || p.dv > 512 || p.dqk > 640 || p.kv_rows >= (int64_t)1 << 30) return false;
+    const int rows = p.S * (p.H / p.G);
+    d->mt = rows <= 16 ? 1 : 2;
+    d->nvt = p.dv <= 128 ? 2 : (p.dv <= 256 ? 4 : 8);
+    d->groups = (rows + 16 * d->mt - 1) / (16 * d->mt);
+    d->shared_v = p.v == p.k && p.v_ts == p.k_ts && p.v_bs == p.k_bs && (p.G == 1 || p.v_hs == p.k_hs) && p.dv <= p.dqk;
+    d->k_stride = (p.dqk + 15) / 16 * 16 + 8;
+    d->v_stride = d->shared_v ? d->k_stride : (p.dv + 15) / 16 * 16 + 8;
+    const size_t kv = (size_t)2 * DM_KEYS * (d->k_stride + (d->shared_v ? 0 : d->v_stride)) * 2;
+    d->smem = kv + (size_t)16 * d->mt * d->k_stride * 2 + (size_t)16 * d->mt * (DM_KEYS + 8) * 2;
+    if (d->smem > 220 * 1024) return false;
+    const int per_sm = d->smem > 110 * 1024 ? 1 : (d->smem > 72 * 1024 ? 2 : 3);
+    const int64_t ctas = (int64_t)d->groups * p.G * p.B, tiles = (p.kv_rows + DM_KEYS - 1) / DM_KEYS;
+    int64_t sp = ((int64_t)sm_count() * per_sm) / ctas;
+    if (sp > tiles) sp = tiles;
+    if (sp > DM_MAX_SPLITS) sp = DM_MAX_SPLITS;
+    d->splits = sp < 1 ? 1 : (int)sp;
+    d->part_floats = (size_t)16 * d->mt * (p.dv + 2);
+    return true;
 }
+
+// Visible key rows of one call in key-row coordinates, and how they are dealt to the splits
+struct DmRange {
+    int64_t i_first, base;      // position of token 0, position of key row 0
+    int lo, hi;                 // rows any query of the call sees: [lo, hi]
+    int tiles, per_split;
+};
+__device__ __forceinline__ DmRange dm_range(const sk_attn_params& p, int splits) {
+    DmRange r;
+    r.i_first = first_position(p.pos, p.start);
+    const int64_t chunk_lo = p.chunk > 0 ? r.i_first / p.chunk * p.chunk : 0;
+    r.base = p.ring ? chunk_lo : p.kv_start;
+    r.lo = (int)(chunk_lo > r.base ? chunk_lo - r.base : 0);
+    int64_t hi = r.i_first + p.S - 1 - r.base;
+    if (hi >= p.kv_rows) hi = p.kv_rows - 1;                     // flagged by the first CTA
+    r.hi = (int)hi;
+    r.tiles = r.hi >= r.lo ? (r.hi - r.lo) / DM_KEYS + 1 : 0;
+    r.per_split = (r.tiles + splits - 1) / splits;
+    return r;
+}
+
+template <int MT, int NVT>
+__global__ void __launch_bounds__(DM_THREADS)
+attn_decode_kernel(sk_attn_params p, int splits, int groups, int shared_v, int k_stride, int v_stride, size_t part_floats) {
+    extern __shared__ __align__(16) char dm_raw[];
+    __shared__ float wmax[2][16 * MT][DM_WARPS];
+    __shared__ float row_sum[16 * MT][DM_WARPS];
+    using bf = __nv_bfloat16;
+    constexpr int ROWS = 16 * MT, KG = DM_WARPS / MT, NT = MT;  // key groups of 8 NT keys
+    bf* ks = reinterpret_cast<bf*>(dm_raw);                     // [2][64][k_stride]
+    bf* vs = shared_v ? ks : ks + 2 * DM_KEYS * k_stride;
+    bf* qs = vs + 2 * DM_KEYS * v_stride;                       // [ROWS][k_stride]
+    constexpr int PS = DM_KEYS + 8;
+    bf* ps = qs + ROWS * k_stride;                              // [ROWS][64 + 8]
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int split = blockIdx.x, g = blockIdx.y / groups, grp = blockIdx.y % groups, b = blockIdx.z;
+    const int rep = p.H / p.G, n_rows = p.S * rep, r_first = grp * ROWS;
+    pdl_launch_dependents();
+    const DmRange rg = dm_range(p, splits);
+    if (split == 0 && grp == 0 && tid == 0 && p.status != nullptr && rg.i_first + p.S - 1 - rg.base >= p.kv_rows)
+        atomicOr(p.status, SK_DEV_POS_OUT_OF_RANGE);
+    const int t_beg = split * rg.per_split;
+    const int t_end = t_beg + rg.per_split < rg.tiles ? t_beg + rg.per_split : rg.tiles;
+    if (t_beg >= t_end) return;                                 // the merge knows which splits exist
+
+    const bf* kb = (const bf*)p.k + (int64_t)b * p.k_bs + (int64_t)g * p.k_hs;
+    const bf* vb = (const bf*)p.v + (int64_t)b * p.v_bs + (int64_t)g * p.v_hs;
+    const int kc = p.dqk / 8, vc = p.dv / 8;                    // 16-byte chunks of a row
+    auto fetch = [&](int tile, int stage) {
+        const int r0 = rg.lo + tile * DM_KEYS;
+        for (int e = tid; e < DM_KEYS * kc; e += DM_THREADS) {
+            const int r = e / kc, c = e - r * kc;
+            const bool live = r0 + r <= rg.hi;
+            cp16(saddr(ks + (stage * DM_KEYS + r) * k_stride + c * 8), kb + (int64_t)(live ? r0 + r : rg.hi) * p.k_ts + c * 8, live);
+        }
+        if (!shared_v) {
+            for (int e = tid; e < DM_KEYS * vc; e += DM_THREADS) {
+                const int r = e / vc, c = e - r * vc;
+                const bool live = r0 + r <= rg.hi;
+                cp16(saddr(vs + (stage * DM_KEYS + r) * v_stride + c * 8), vb + (int64_t)(live ? r0 + r : rg.hi) * p.v_ts + c * 8, live);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    fetch(t_beg, 0);
+    const int k16 = (p.dqk + 15) / 16;
+    // queries, and the zero columns that round a row up to 16
+    for (int e = tid; e < ROWS * k16 * 2; e += DM_THREADS) {
+        const int r = e / (k16 * 2), c = e - r * (k16 * 2), row = r_first + r;
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (row < n_rows && c < kc) {
+            const int s = row / rep, hh = row - s * rep;
+            v = *reinterpret_cast<const uint4*>((const bf*)p.q + (int64_t)b * p.q_bs + (int64_t)s * p.q_ss +
+                                                (int64_t)(g * rep + hh) * p.q_hs + c * 8);
+        }
+        *reinterpret_cast<uint4*>(qs + r * k_stride + c * 8) = v;
+    }
+    if (k16 * 2 > kc)
+        for (int e = tid; e < 2 * DM_KEYS; e += DM_THREADS) *reinterpret_cast<uint4*>(ks + e * k_stride + kc * 8) = make_uint4(0, 0, 0, 0);
+
+    // rows of this thread: scores (one 16-row tile per warp) and accumulators (all tiles)
+    const int mtile = MT == 1 ? 0 : (warp & 1), kg = MT == 1 ? warp : (warp >> 1);
+    const int fr = lane >> 2, fc = (lane & 3) * 2;              // fragment row and first column
+    int64_t qi[2];                                              // query's own key row
+    int lo[2];
+    const float* brow[2];
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        const int row = r_first + mtile * 16 + fr + 8 * k, s = row / rep;
+        const int64_t i = rg.i_first + s;
+        qi[k] = row < n_rows ? i - rg.base : -1;                // absent row: sees nothing
+        lo[k] = p.chunk > 0 ? (int)max((int64_t)0, i / p.chunk * p.chunk - rg.base) : 0;
+        brow[k] = p.bias != nullptr && row < n_rows ? p.bias + (int64_t)(g * rep + row - s * rep) * p.bias_len : nullptr;
+    }
+    const float sl = p.scale * DM_LOG2E;
+    float m_own[2] = {-INFINITY, -INFINITY};                    // of the two score rows
+    float m_acc[MT][2], l_own[2] = {0.f, 0.f};
+    float acc[MT][NVT][4];
+#pragma unroll
+    for (int t = 0; t < MT; ++t) {
+        m_acc[t][0] = m_acc[t][1] = -INFINITY;
+#pragma unroll
+        for (int v = 0; v < NVT; ++v)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[t][v][e] = 0.f;
+    }
+    const int col0 = warp * NVT * 8;
+
+    for (int t = t_beg; t < t_end; ++t) {
+        const int stage = (t - t_beg) & 1;
+        __syncthreads();                                        // the other stage is free
+        if (t + 1 < t_end) {
+            fetch(t + 1, stage ^ 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        const bf* kt = ks + stage * DM_KEYS * k_stride;
+        const bf* vt = vs + stage * DM_KEYS * v_stride;
+        // ---- scores of 16 rows x 8 NT keys, two independent sums along the head dimension
+        float sc[2][NT][4];
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+#pragma unroll
+            for (int n = 0; n < NT; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) sc[u][n][e] = 0.f;
+        const uint32_t qa = saddr(qs + (mtile * 16 + (lane & 15)) * k_stride + (lane >> 4) * 8);
+        const uint32_t ka = NT == 1 ? saddr(kt + (kg * 8 + (lane & 7)) * k_stride + ((lane >> 3) & 1) * 8)
+                                    : saddr(kt + (kg * 16 + (lane & 7) + (lane >> 4) * 8) * k_stride + ((lane >> 3) & 1) * 8);
+        auto along = [&](float (&d)[NT][4], int k) {
+            uint32_t a[4];
+            ldsm4(qa + k * 32, a);
+            if constexpr (NT == 1) {
+                uint32_t b0, b1;
+                ldsm2(ka + k * 32, b0, b1);
+                mma16816(d[0], a, b0, b1);
+            } else {
+                uint32_t bb[4];
+                ldsm4(ka + k * 32, bb);
+                mma16816(d[0], a, bb[0], bb[1]);
+                mma16816(d[1], a, bb[2], bb[3]);
+            }
+        };
+        int kk = 0;
+#pragma unroll 2
+        for (; kk + 2 <= k16; kk += 2) {
+            along(sc[0], kk);
+            along(sc[1], kk + 1);
+        }
+        if (kk < k16) along(sc[0], kk);
+        const int r0 = rg.lo + t * DM_KEYS + kg * 8 * NT;       // key row of column 0 of this warp
+        float mt[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int k = e >> 1, r = r0 + n * 8 + fc + (e & 1);
+                float v = (sc[0][n][e] + sc[1][n][e]) * sl;
+                if (r <= qi[k] && r >= lo[k] && r <= rg.hi) {
+                    if (brow[k] != nullptr) {
+                        const int64_t d = qi[k] - r;
+                        v = fmaf(__ldg(brow[k] + (d < p.bias_len ? d : p.bias_len - 1)), DM_LOG2E, v);
+                    }
+                } else {
+                    v = -INFINITY;
+                }
+                sc[0][n][e] = v;
+                mt[k] = fmaxf(mt[k], v);
+            }
+        float (*wm)[DM_WARPS] = wmax[t & 1];
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            mt[k] = fmaxf(mt[k], __shfl_xor_sync(FULL, mt[k], 1));
+            mt[k] = fmaxf(mt[k], __shfl_xor_sync(FULL, mt[k], 2));
+            if ((lane & 3) == 0) wm[mtile * 16 + fr + 8 * k][kg] = mt[k];
+        }
+        __syncthreads();
+        // ---- new maxima: of the score rows for the weights, of all rows for the accumulators
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            float mn = m_own[k];
+#pragma unroll
+            for (int w = 0; w < KG; ++w) mn = fmaxf(mn, wm[mtile * 16 + fr + 8 * k][w]);
+            l_own[k] *= mn == -INFINITY ? 1.f : exp2f(m_own[k] - mn);
+            m_own[k] = mn;
+            const float mc = mn == -INFINITY ? 0.f : mn;
+#pragma unroll
+            for (int n = 0; n < NT; ++n) {
+                const float x = exp2f(sc[0][n][2 * k] - mc), y = exp2f(sc[0][n][2 * k + 1] - mc);
+                l_own[k] += x + y;
+                *reinterpret_cast<__nv_bfloat162*>(ps + (mtile * 16 + fr + 8 * k) * PS + kg * 8 * NT + n * 8 + fc) =
+                    __floats2bfloat162_rn(x, y);
+            }
+        }
+#pragma unroll
+        for (int tt = 0; tt < MT; ++tt)
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                float mn = m_acc[tt][k];
+#pragma unroll
+                for (int w = 0; w < KG; ++w) mn = fmaxf(mn, wm[tt * 16 + fr + 8 * k][w]);
+                if (mn != m_acc[tt][k]) {
+                    const float f = exp2f(m_acc[tt][k] - mn);   // mn is finite here
+#pragma unroll
+                    for (int v = 0; v < NVT; ++v) {
+                        acc[tt][v][2 * k] *= f;
+                        acc[tt][v][2 * k + 1] *= f;
+                    }
+                    m_acc[tt][k] = mn;
+                }
+            }
+        __syncthreads();
+        // ---- P V: every warp all rows, its own value columns
+        if (col0 < p.dv) {
+#pragma unroll
+            for (int k = 0; k < DM_KEYS / 16; ++k) {
+                uint32_t a[MT][4];
+#pragma unroll
+                for (int tt = 0; tt < MT; ++tt) ldsm4(saddr(ps + (tt * 16 + (lane & 15)) * PS + k * 16 + (lane >> 4) * 8), a[tt]);
+#pragma unroll
+                for (int v = 0; v < NVT; v += 2) {
+                    if (col0 + v * 8 < p.dv) {
+                        uint32_t bb[4];
+                        ldsm4t(saddr(vt + (k * 16 + (lane & 15)) * v_stride + col0 + v * 8 + (lane >> 4) * 8), bb);
+#pragma unroll
+                        for (int tt = 0; tt < MT; ++tt) {
+                            mma16816(acc[tt][v], a[tt], bb[0], bb[1]);
+                            mma16816(acc[tt][v + 1], a[tt], bb[2], bb[3]);
+                        }
+                    }
+                }
+            }
+        }
+    }
+    // ---- partial result: rows x (dv sums | maximum | sum of weights)
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        l_own[k] += __shfl_xor_sync(FULL, l_own[k], 1);
+        l_own[k] += __shfl_xor_sync(FULL, l_own[k], 2);
+        if ((lane & 3) == 0) row_sum[mtile * 16 + fr + 8 * k][kg] = l_own[k];
+    }
+    __syncthreads();
+    float* part = (float*)p.workspace + ((((int64_t)b * p.G + g) * groups + grp) * splits + split) * part_floats;
+    if (tid < ROWS) {
+        float l = 0.f;
+#pragma unroll
+        for (int w = 0; w < KG; ++w) l += row_sum[tid][w];
+        part[(int64_t)ROWS * p.dv + ROWS + tid] = l;
+    }
+    if (warp == 0 && (lane & 3) == 0)
+#pragma unroll
+        for (int tt = 0; tt < MT; ++tt)
+#pragma unroll
+            for (int k = 0; k < 2; ++k) part[(int64_t)ROWS * p.dv + tt * 16 + fr + 8 * k] = m_acc[tt][k];
+#pragma unroll
+    for (int tt = 0; tt < MT; ++tt)
+#pragma unroll
+        for (int v = 0; v < NVT; ++v) {
+            const int c = col0 + v * 8 + fc;
+            if (c < p.dv) {
+#pragma unroll
+                for (int k = 0; k < 2; ++k)
+                    *reinterpret_cast<float2*>(part + (int64_t)(tt * 16 + fr + 8 * k) * p.dv + c) =
+                        make_float2(acc[tt][v][2 * k], acc[tt][v][2 * k + 1]);
+            }
+        }
+}
+
+// One CTA per query row: merge the splits that exist, add the sink, divide.
+__global__ void __launch_bounds__(128)
+attn_decode_merge_kernel(sk_attn_params p, int splits, int groups, int rows_per_group, size_t part_floats) {
+    __shared__ float w_s[DM_MAX_SPLITS];
+    __shared__ float red[32];
+    const int rep = p.H / p.G, row = blockIdx.x, g = blockIdx.y, b = blockIdx.z, t = threadIdx.x;
+    const int s = row / rep, h = g * rep + row - s * rep, grp = row / rows_per_group, r = row - grp * rows_per_group;
+    const float sink = p.sink != nullptr ? p.sink[h] * DM_LOG2E : -INFINITY;
+    pdl_wait();
+    const DmRange rg = dm_range(p, splits);
+    const int n = rg.tiles > 0 ? (rg.tiles + rg.per_split - 1) / rg.per_split : 0;
+    const float* part = (const float*)p.workspace + (((int64_t)b * p.G + g) * groups + grp) * splits * part_floats;
+    float m = sink;
+    for (int k = 0; k < n; ++k) m = fmaxf(m, __ldcg(part + k * part_floats + (int64_t)rows_per_group * p.dv + r));
+    const float mc = m == -INFINITY ? 0.f : m;
+    float l = 0.f;
+    for (int k = t; k < n; k += 128) {
+        const float* e = part + k * part_floats + (int64_t)rows_per_group * p.dv;
+        const float w = exp2f(__ldcg(e + r) - mc);
+        w_s[k] = w;
+        l = fmaf(w, __ldcg(e + rows_per_group + r), l);
+    }
+    l = block_sum(l, red);
+    __syncthreads();
+    l += exp2f(sink - mc);
+    const float inv = l > 0.f ? 1.f / l : 0.f;
+    __nv_bfloat16* out = (__nv_bfloat16*)p.out + (int64_t)b * p.o_bs + (int64_t)s * p.o_ss + (int64_t)h * p.o_hs;
+    for (int c = 4 * t; c < p.dv; c += 512) {
+        float a[4] = {0.f, 0.f, 0.f, 0.f};
+        for (int k = 0; k < n; ++k) {
+            const float4 v = __ldcg(reinterpret_cast<const float4*>(part + k * part_floats + (int64_t)r * p.dv + c));
+            a[0] = fmaf(w_s[k], v.x, a[0]);
+            a[1] = fmaf(w_s[k], v.y, a[1]);
+            a[2] = fmaf(w_s[k], v.z, a[2]);
+            a[3] = fmaf(w_s[k], v.w, a[3]);
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) a[e] *= inv;
+        store_vec<__nv_bfloat16, 4>(out + c, a);
+    }
+}
+
+bool rows_16b(const void* base, int64_t a, int64_t b, int64_t c) {
+    return (uintptr_t)base % 16 == 0 && a % 8 == 0 && b % 8 == 0 && c % 8 == 0;
+}
+
+}  // namespace
+
+bool attn_decode_mma_applicable(const sk_attn_params& p) {
+    DmPlan d;
+    return dm_plan(p, &d) && rows_16b(p.q, p.q_bs, p.q_ss, p.q_hs) && rows_16b(p.k, p.k_bs, p.k_ts, p.k_hs) &&
+           rows_16b(p.v, p.v_bs, p.v_ts, p.v_hs) && rows_16b(p.out, p.o_bs, p.o_ss, p.o_hs);
+}
+
+size_t attn_decode_mma_workspace(const sk_attn_params& p) {
+    DmPlan d;
+    if (!dm_plan(p, &d)) return 0;
+    return (size_t)p.B * p.G * d.groups * d.splits * d.part_floats * sizeof(float);
+}
+
+int launch_attn_decode_mma(const sk_attn_params& p, cudaStream_t st) {
+    DmPlan d;
+    if (!dm_plan(p, &d)) return fail(SK_ERR_UNSUPPORTED, "skb_attn: shape outside the decode kernel");
+    dim3 grid((unsigned)d.splits, (unsigned)(p.G * d.groups), (unsigned)p.B);
+#define SK_DM(MT, NVT)                                                                                                   \
+    do {                                                                                                                 \
+        auto kern = attn_decode_kernel<MT, NVT>;                                                                         \
+        const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)d.smem);      \
+        if (e != cudaSuccess) return fail(SK_ERR_CUDA, "attn_decode_kernel smem attribute: %s", cudaGetErrorString(e));  \
+        kern<<<grid, DM_THREADS, d.smem, st>>>(p, d.splits, d.groups, (int)d.shared_v, d.k_stride, d.v_stride, d.part_floats); \
+    } while (0)
+    if (d.mt == 1) {
+        if (d.nvt == 2) SK_DM(1, 2);
+        else if (d.nvt == 4) SK_DM(1, 4);
+        else SK_DM(1, 8);
+    } else {
+        if (d.nvt == 2) SK_DM(2, 2);
+        else if (d.nvt == 4) SK_DM(2, 4);
+        else SK_DM(2, 8);
+    }
+#undef SK_DM
+    if (int rc = check_launch("attn_decode_kernel")) return rc;
+    const cudaError_t e = launch_after(attn_decode_merge_kernel, dim3((unsigned)(p.S * (p.H / p.G)), (unsigned)p.G, (unsigned)p.B), dim3(128),
+                                       0, st, p, d.splits, d.groups, 16 * d.mt, d.part_floats);
+    if (e != cudaSuccess) return fail(SK_ERR_CUDA, "attn_decode_merge_kernel: %s", cudaGetErrorString(e));
+    return SK_OK;
+}
+
+}  // namespace sk
