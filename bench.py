@@ -63,7 +63,7 @@ def parse_args():
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=1000)
     ap.add_argument("--warmup", type=int, default=20)
-    ap.add_argument("--workload", default="c3", choices=sorted(PRESETS) + ["c4", "c4-128k", "c4-128k-b4", "c5"],
+    ap.add_argument("--workload", default="c3", choices=sorted(PRESETS) + ["c4", "c4-128k", "c4-128k-b4", "c5", "radapel"],
                     help="c1-c3: one attention layer (op level); c4 / c5: whole-model greedy decode, "
                          "Llama-3-8B / Llama-3-70B shape with random weights")
     ap.add_argument("--model-record", default="auto", choices=["auto", "on", "off"],
@@ -766,10 +766,274 @@ def measure_model(args, wl, K, W, world, rank, local_rank):
     return out
 
 
+# ------------------------------------------------------------------------------- Radapel
+RADAPEL_SIZES = {
+    # name: (width, query heads, KV heads, head size, feed-forward, latent rank, state-space heads)
+    "2k": (2048, 16, 4, 128, 5632, 512, 64),
+    "4k": (4096, 32, 8, 128, 14336, 512, 128),
+}
+RADAPEL_CHUNK, RADAPEL_ROT, RADAPEL_STATE = 8192, 64, 128
+
+
+def radapel_config(size):
+    """Two attention layers, one latent, one state-space layer; the last three run twice: 7 layer runs."""
+    W, H, G, D, F, K, M = RADAPEL_SIZES[size]
+    mlp = {"kind": "dense", "ff": F, "limit": 7.0}
+    att = {"type": "attention", "mlp": mlp, "mixer": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5,
+                                                       "bias_max": 1024, "mask": {"size": RADAPEL_CHUNK}}}
+    lat = {"type": "latent_attention", "mlp": mlp,
+           "mixer": {"heads": H, "dim": D, "rot_dim": RADAPEL_ROT, "vdim": D, "kv_rank": K, "scale": (D + RADAPEL_ROT) ** -0.5,
+                     "rot": {"base": 500000.0, "dims": RADAPEL_ROT}}}
+    ssm = {"type": "mamba2", "mlp": None, "mixer": {"heads": M, "vdim": 64, "state": RADAPEL_STATE, "groups": 8, "conv": 4,
+                                                     "norm_groups": 8}}
+    return {"architecture": "Radapel", "vocab": 32768, "width": W, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "layers": [att, att, lat, ssm], "loop": {"start": 1, "stop": 4, "times": 2}}
+
+
+def measure_throughput(model, vocab, B, T, K, W, dev, mode=None):
+    """Prefill and decode of one decoder: seconds of a prompt of T tokens (second run), ms per graph-replayed
+    decode token after it, and the same with every token copied to pinned host memory."""
+    model.max_seq_length = -1
+    model.setup_caches(B, T + 2 * K + W + 16)
+    model.setup_decode(B, mode)
+    prompt = torch.randint(0, vocab, (B, T), generator=torch.Generator().manual_seed(5)).pin_memory()
+    ev = lambda: torch.cuda.Event(enable_timing=True)  # noqa: E731
+    for _ in range(2):
+        t0, t1 = ev(), ev()
+        torch.cuda.synchronize()
+        t0.record()
+        logits = model.prefill(prompt.to(dev, non_blocking=True))
+        first = torch.argmax(logits, dim=-1, keepdim=True)
+        t1.record()
+        torch.cuda.synchronize()
+    model.start_decode(first, T)
+    for _ in range(W):
+        model.decode_one_token()
+    torch.cuda.synchronize()
+    e0, e1, e2 = ev(), ev(), ev()
+    e0.record()
+    for _ in range(K):
+        model.decode_one_token()
+    e1.record()
+    torch.cuda.synchronize()
+    host = torch.empty(B, 1, dtype=torch.long).pin_memory()
+    e1b = ev()
+    e1b.record()
+    for _ in range(K):
+        host.copy_(model.decode_one_token(), non_blocking=True)
+        torch.cuda.current_stream(dev).synchronize()
+    e2.record()
+    torch.cuda.synchronize()
+    pre, ms, e2e = t0.elapsed_time(t1), e0.elapsed_time(e1) / K, e1b.elapsed_time(e2) / K
+    return {"prefill_ms": pre, "prefill_tokens_per_s": B * T / pre * 1e3, "decode_ms_per_token": ms,
+            "decode_tokens_per_s": B / ms * 1e3, "e2e_decode_tokens_per_s": B / e2e * 1e3}
+
+
+def time_op(fn, flush, n=20):
+    """Device microseconds of fn(): CUDA graphs of [flush L2, fn] against [flush L2]."""
+    fn()
+    torch.cuda.synchronize()
+
+    def graph(with_fn):
+        g = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(g):
+            for _ in range(4):
+                flush.fill_(1)
+                if with_fn:
+                    fn()
+        return g
+
+    times = []
+    for g in (graph(True), graph(False)):
+        for _ in range(3):
+            g.replay()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        a.record()
+        for _ in range(n):
+            g.replay()
+        b.record()
+        torch.cuda.synchronize()
+        times.append(a.elapsed_time(b) / (4 * n) * 1e3)
+    return times[0] - times[1]
+
+
+def measure_radapel_kernels(size, S, T, B, dev):
+    """Every kernel of the design beside the like kernel of the Llama-shaped model, at one size: prefill
+    kernels on S tokens from position 0, decode kernels for B sequences at context T."""
+    import torch.nn.functional as F
+    from flash_attn import flash_attn_func, flash_attn_with_kvcache
+    from socket_b200 import block_ops as ops
+    from socket_b200.mixers import LatentCache, Mamba2, Portion, rotary_angles  # noqa: F401
+    from socket_b200.model import apply_rotary_emb
+    W, H, G, D, FF, K, M = RADAPEL_SIZES[size]
+    R, N, P = RADAPEL_ROT, RADAPEL_STATE, 64
+    bf = torch.bfloat16
+    rn = lambda *s: torch.randn(*s, device=dev, dtype=bf)  # noqa: E731
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    peaks = measured_peaks()
+    rows = []
+
+    def add(name, us, like, like_us, flops=0.0, nbytes=0.0, like_flops=None, like_bytes=None):
+        def frac(t, f, b):
+            return max(f / (peaks["bf16_tflops"] * 1e12), b / (peaks["hbm_gbs"] * 1e9)) / (t * 1e-6)
+        r = {"kernel": name, "us": round(us, 2), "roofline_frac": round(frac(us, flops, nbytes), 3)}
+        if flops:
+            r["tflops"] = round(flops / us / 1e6, 1)
+        if nbytes:
+            r["gbs"] = round(nbytes / us / 1e3, 1)
+        if like is not None:
+            lf, lb = flops if like_flops is None else like_flops, nbytes if like_bytes is None else like_bytes
+            r.update(like=like, like_us=round(like_us, 2), like_roofline_frac=round(frac(like_us, lf, lb), 3))
+            r["like_frac_over_frac"] = round(r["like_roofline_frac"] / max(r["roofline_frac"], 1e-9), 2)
+        rows.append(r)
+
+    # ---- attention of a prompt
+    q, k, v = rn(1, S, H, D), rn(1, S, G, D), rn(1, S, G, D)
+    fa = time_op(lambda: flash_attn_func(q, k, v, causal=True), flush)
+    pairs = S * (S + 1) / 2
+    bias = torch.randn(H, 1025, device=dev)
+    f = pairs * H * 4 * D
+    add("chunked attention, prefill", time_op(lambda: ops.attn(q, k, v, scale=D ** -0.5, chunk=RADAPEL_CHUNK, bias=bias), flush),
+        "flash_attn_func", fa, flops=f)
+    ql, kl, vl = rn(1, S, H, D + R), rn(1, S, H, D + R), rn(1, S, H, D)
+    sink = torch.randn(H, device=dev)
+    add("latent attention, prefill (expanded)", time_op(lambda: ops.attn(ql, kl, vl, scale=0.07, sink=sink), flush),
+        "flash_attn_func", fa, flops=pairs * H * 2 * (2 * D + R), like_flops=f)
+    # ---- attention of a decoded token
+    pos = torch.tensor([T - 1], device=dev)
+    lens = torch.full((B,), T - 1, dtype=torch.int32, device=dev)
+    q1, k1 = rn(B, 1, H, D), rn(B, 1, G, D)
+    kc, vc = rn(B, T, G, D), rn(B, T, G, D)
+    fad = time_op(lambda: flash_attn_with_kvcache(q1, kc, vc, k=k1, v=k1, cache_seqlens=lens, causal=True), flush)
+    fab = B * T * G * 2 * D * 2
+    C = min(T, RADAPEL_CHUNK)
+    kr, vr = kc[:, :C].contiguous(), vc[:, :C].contiguous()
+    ringpos = torch.tensor([C - 1], device=dev)
+    lens_c = torch.full((B,), C - 1, dtype=torch.int32, device=dev)
+    fac = time_op(lambda: flash_attn_with_kvcache(q1, kr, vr, k=k1, v=k1, cache_seqlens=lens_c, causal=True), flush)
+    ws = torch.empty(64 << 20, dtype=torch.uint8, device=dev)
+    add(f"chunked attention, decode (chunk {C} full)",
+        time_op(lambda: ops.attn(q1, kr, vr, scale=D ** -0.5, pos=ringpos, chunk=C, ring=True, bias=bias, workspace=ws), flush),
+        "flash_attn_with_kvcache, same cache", fac, nbytes=B * C * G * 2 * D * 2)
+    cache = rn(B, T, K + R)
+    qa = rn(B, 1, H, K + R)
+    shared = cache.unsqueeze(2)
+    lat_f = B * H * T * 2 * (2 * K + R)
+    add("latent attention, decode", time_op(lambda: ops.attn(qa, shared, shared[..., :K], scale=0.07, pos=pos, sink=sink, workspace=ws), flush),
+        "flash_attn_with_kvcache, same context", fad, nbytes=B * T * (K + R) * 2, flops=lat_f, like_bytes=fab, like_flops=0.0)
+    # ---- latent up- and down-projections of a decoded token
+    uk, uv, wo = rn(H * D, K), rn(H * D, K), rn(W, H * D)
+    qd, o, ho = rn(B, H * (D + R)), rn(B, H, K), rn(B, H * D)
+    gemv = time_op(lambda: torch.mm(ho, wo.t()), flush)
+    wb = W * H * D * 2
+    add("latent absorb, decode", time_op(lambda: ops.latent_absorb(qd, uk, H, D, R, K + R), flush), "torch.mm wo", gemv,
+        nbytes=H * D * K * 2, like_bytes=wb)
+    add("latent up, decode", time_op(lambda: ops.latent_up(o, uv, D), flush), "torch.mm wo", gemv, nbytes=H * D * K * 2, like_bytes=wb)
+    # ---- residual stream
+    x, y, w = torch.randn(S, W, device=dev), rn(S, W), rn(W)
+    xb = rn(S, W)
+    norm = time_op(lambda: F.rms_norm(xb + y, (W,), w, 1e-5), flush)
+    add("residual + two norms, prefill", time_op(lambda: ops.residual_norm(x, 1e-5, y=y, w_in=w, w_out=w), flush),
+        "add + F.rms_norm", norm, nbytes=S * W * 12, like_bytes=S * W * 8)
+    x1, y1, xb1 = torch.randn(B, W, device=dev), rn(B, W), rn(B, W)
+    norm1 = time_op(lambda: F.rms_norm(xb1 + y1, (W,), w, 1e-5), flush)
+    add("residual + two norms, decode", time_op(lambda: ops.residual_norm(x1, 1e-5, y=y1, w_in=w, w_out=w), flush),
+        "add + F.rms_norm", norm1, nbytes=B * W * 12 + 4 * W, like_bytes=B * W * 8 + 2 * W)
+    gu = rn(S, 2 * FF)
+    add("clamped unit, prefill", time_op(lambda: ops.glu_clamped(gu, FF, 7.0), flush), "silu * up",
+        time_op(lambda: F.silu(gu[:, :FF]) * gu[:, FF:], flush), nbytes=S * FF * 6)
+    gu1 = rn(B, 2 * FF)
+    add("clamped unit, decode", time_op(lambda: ops.glu_clamped(gu1, FF, 7.0), flush), "silu * up",
+        time_op(lambda: F.silu(gu1[:, :FF]) * gu1[:, FF:], flush), nbytes=B * FF * 6)
+    # ---- latent rows of a prompt
+    ang = rotary_angles(S, R, 500000.0, dev)
+    dkv, qq, lw, lc = rn(S, K + R), rn(S, H * (D + R)), rn(K), rn(1, S, K + R)
+    fc = torch.randn(S, D // 2, 2, device=dev).to(bf)
+    add("latent append + rotation, prefill",
+        time_op(lambda: ops.latent_append(dkv, qq, lw, ang, lc, S=S, n_heads=H, dim=D, rot=R, rank=K, eps=1e-5), flush),
+        "apply_rotary_emb of q", time_op(lambda: apply_rotary_emb(q, fc), flush),
+        nbytes=S * (4 * (K + R) + 4 * H * R), like_bytes=S * H * D * 4)
+    # ---- state space
+    mix = Mamba2(W, M, P, N, 8, 4, 8, 1e-5).to(device=dev, dtype=bf)
+    mix.finish_loading()
+    st = mix.make_cache(B, T, bf, dev)
+    proj, inner = rn(S, mix.w_in.shape[0]), mix.inner
+    args = (mix.conv_w, mix.conv_b, mix.dt_bias_f32, mix.A_log_f32, mix.skip_f32)
+    ssm_f = S * M * (2 * 64 * N / 2 + 2 * 64 * P / 2 + 4 * N * P)
+    add("state space, prefill (convolution + scan)",
+        time_op(lambda: ops.ssm(proj, inner, *args, st.conv[:1], st.state[:1], S=S, groups=8), flush), None, 0,
+        flops=ssm_f, nbytes=S * (inner * 2 + mix.channels * 6))
+    p1 = rn(B, mix.w_in.shape[0])
+    add("state space, decode (convolution + step)",
+        time_op(lambda: ops.ssm(p1, inner, *args, st.conv, st.state, S=1, groups=8, start=5), flush), None, 0, nbytes=B * M * N * P * 8)
+    yy = rn(S, inner)
+    add("gated group norm, prefill", time_op(lambda: ops.gated_group_norm(yy, proj, mix.norm_w, 8, 1e-5), flush),
+        "add + F.rms_norm", norm, nbytes=S * inner * 6, like_bytes=S * W * 8)
+    return rows
+
+
+def measured_peaks():
+    try:
+        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+            d = json.load(f)
+        return {"hbm_gbs": d["hbm_gbs"], "bf16_tflops": d["bf16_tflops"], "source": "measured"}
+    except Exception:
+        return {"hbm_gbs": FALLBACK_HBM_GBS, "bf16_tflops": 1590.0, "source": "fallback"}
+
+
+def run_radapel(args, dev):
+    """Prefill and decode throughput of Radapel at two sizes beside the Llama-shaped Transformer with as many
+    layers, the same width, heads and feed-forward (sparse and dense decode), and the kernels one by one."""
+    from socket_b200.model import ModelArgs, Transformer
+    from socket_b200.registry import build_model
+    torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
+    K, W = min(args.steps, 64), max(3, min(args.warmup, 8))
+    clocks = ClockSampler(dev.index or 0)
+    out = {}
+    for size, (width, H, G, D, FF, *_rest) in RADAPEL_SIZES.items():
+        cfg = radapel_config(size)
+        model = build_model(cfg, dtype=torch.bfloat16, device=dev).init_random(args.seed)
+        n_runs = len(model.runs)
+        rec = {"layer_runs": n_runs, "width": width}
+        shapes = [(1, 2048), (1, 8000), (1, 32000), (8, 8000)]   # decoding late in a chunk of 8192
+        for B, T in shapes:
+            rec[f"radapel B={B} T={T}"] = measure_throughput(model, cfg["vocab"], B, T, K, W, dev)
+        flags = model.device_flags()
+        del model
+        torch.cuda.empty_cache()
+        old = torch.get_default_dtype()
+        torch.set_default_dtype(torch.bfloat16)
+        with torch.device(dev):
+            other = Transformer(ModelArgs(block_size=131072, vocab_size=cfg["vocab"], n_layer=n_runs, n_head=H, n_local_heads=G,
+                                          dim=width, intermediate_size=FF, rope_base=500000))
+        torch.set_default_dtype(old)
+        other.init_random(args.seed)
+        for B, T in shapes:
+            for mode in ("sparse", "dense"):
+                rec[f"transformer {mode} B={B} T={T}"] = measure_throughput(other, cfg["vocab"], B, T, K, W, dev, mode)
+        del other
+        torch.cuda.empty_cache()
+        rec["kernels S=8192, decode B=1 T=32768"] = measure_radapel_kernels(size, 8192, 32768, 1, dev)
+        rec["device_flags"] = flags
+        torch.cuda.empty_cache()
+        out[size] = rec
+    main_rec = out["4k"]["radapel B=1 T=32000"]
+    print(json.dumps({
+        "metric": "decode_tokens_per_s", "value": main_rec["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": K,
+        "warmup": W, "ms_per_step": main_rec["decode_ms_per_token"], "higher_is_better": True, "scaling": "weak",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "config": {"model": "Radapel 4k, 7 layer runs, random weights", "global_batch": 1, "seq_len": 32000,
+                   "parallelism": "single GPU", "timing": "CUDA events around K graph-replayed decode tokens; weights exceed L2; "
+                   "kernels one by one with L2 flushed"},
+        "e2e": {"value": main_rec["e2e_decode_tokens_per_s"], "unit": "tokens/s", "h2d_bytes_per_step": 0, "d2h_bytes_per_step": 8},
+        "peaks": measured_peaks(), "clocks": clocks.stop(), "radapel": out}))
+
+
 def main():
     args = parse_args()
     if args.impl == "reference":
-        if args.workload in MODEL_WORKLOADS:
+        if args.workload in MODEL_WORKLOADS or args.workload == "radapel":
             if int(os.environ.get("RANK", "0")) == 0:
                 print(json.dumps({"impl": "reference", "unavailable": "the whole-model workloads have no CPU arm: the "
                                   "reference's CPU path is timed at the op level (c1-c3)"}))
@@ -790,6 +1054,9 @@ def main():
         tp.maybe_init_dist("nccl")
     K, W = args.steps, args.warmup
 
+    if args.workload == "radapel":
+        run_radapel(args, torch.device("cuda", local_rank))
+        return
     if args.workload in MODEL_WORKLOADS:
         K = min(K, MODEL_WORKLOADS[args.workload][3] - 1)
         m = measure_model(args, args.workload, K, W, world, rank, local_rank)

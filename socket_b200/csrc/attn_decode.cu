@@ -99,16 +99,16 @@ attn_decode_kernel(sk_attn_params p, int splits, int groups, int shared_v, int k
     const int kc = p.dqk / 8, vc = p.dv / 8;                    // 16-byte chunks of a row
     auto fetch = [&](int tile, int stage) {
         const int r0 = rg.lo + tile * DM_KEYS;
-        for (int e = tid; e < DM_KEYS * kc; e += DM_THREADS) {
-            const int r = e / kc, c = e - r * kc;
+        for (int r = warp; r < DM_KEYS; r += DM_WARPS) {         // a warp per row, lanes along it
             const bool live = r0 + r <= rg.hi;
-            cp16(saddr(ks + (stage * DM_KEYS + r) * k_stride + c * 8), kb + (int64_t)(live ? r0 + r : rg.hi) * p.k_ts + c * 8, live);
-        }
-        if (!shared_v) {
-            for (int e = tid; e < DM_KEYS * vc; e += DM_THREADS) {
-                const int r = e / vc, c = e - r * vc;
-                const bool live = r0 + r <= rg.hi;
-                cp16(saddr(vs + (stage * DM_KEYS + r) * v_stride + c * 8), vb + (int64_t)(live ? r0 + r : rg.hi) * p.v_ts + c * 8, live);
+            const int64_t row = live ? r0 + r : rg.hi;
+            const bf* src = kb + row * p.k_ts;
+            const uint32_t dst = saddr(ks + (stage * DM_KEYS + r) * k_stride);
+            for (int c = lane; c < kc; c += 32) cp16(dst + c * 16, src + c * 8, live);
+            if (!shared_v) {
+                const bf* vsrc = vb + row * p.v_ts;
+                const uint32_t vdst = saddr(vs + (stage * DM_KEYS + r) * v_stride);
+                for (int c = lane; c < vc; c += 32) cp16(vdst + c * 16, vsrc + c * 8, live);
             }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -319,45 +319,79 @@ attn_decode_kernel(sk_attn_params p, int splits, int groups, int shared_v, int k
         }
 }
 
-// One CTA per query row: merge the splits that exist, add the sink, divide.
-__global__ void __launch_bounds__(128)
+// One CTA per query row: merge the splits that exist, add the sink, divide.  Groups of 128 threads take every
+// fourth split; a thread of a group owns four value columns at a time.
+constexpr int DG_THREADS = 512, DG_GROUPS = DG_THREADS / 128;
+__global__ void __launch_bounds__(DG_THREADS)
 attn_decode_merge_kernel(sk_attn_params p, int splits, int groups, int rows_per_group, size_t part_floats) {
     __shared__ float w_s[DM_MAX_SPLITS];
-    __shared__ float red[32];
+    __shared__ float red[2][DG_THREADS / 32];
+    __shared__ float4 acc_s[DG_GROUPS - 1][128];
     const int rep = p.H / p.G, row = blockIdx.x, g = blockIdx.y, b = blockIdx.z, t = threadIdx.x;
+    const int warp = t >> 5, lane = t & 31;
     const int s = row / rep, h = g * rep + row - s * rep, grp = row / rows_per_group, r = row - grp * rows_per_group;
     const float sink = p.sink != nullptr ? p.sink[h] * DM_LOG2E : -INFINITY;
-    pdl_wait();
     const DmRange rg = dm_range(p, splits);
-    const int n = rg.tiles > 0 ? (rg.tiles + rg.per_split - 1) / rg.per_split : 0;
+    const int n = rg.tiles > 0 ? (rg.tiles + rg.per_split - 1) / rg.per_split : 0;      // <= DM_MAX_SPLITS
     const float* part = (const float*)p.workspace + (((int64_t)b * p.G + g) * groups + grp) * splits * part_floats;
-    float m = sink;
-    for (int k = 0; k < n; ++k) m = fmaxf(m, __ldcg(part + k * part_floats + (int64_t)rows_per_group * p.dv + r));
-    const float mc = m == -INFINITY ? 0.f : m;
-    float l = 0.f;
-    for (int k = t; k < n; k += 128) {
-        const float* e = part + k * part_floats + (int64_t)rows_per_group * p.dv;
-        const float w = exp2f(__ldcg(e + r) - mc);
-        w_s[k] = w;
-        l = fmaf(w, __ldcg(e + rows_per_group + r), l);
+    const float* stat = part + (int64_t)rows_per_group * p.dv + r;
+    pdl_wait();
+    float mk = -INFINITY, lk = 0.f;
+    if (t < n) {
+        mk = __ldcg(stat + t * part_floats);
+        lk = __ldcg(stat + t * part_floats + rows_per_group);
     }
-    l = block_sum(l, red);
+    float m = fmaxf(mk, sink);
+#pragma unroll
+    for (int o = 16; o >= 1; o >>= 1) m = fmaxf(m, __shfl_xor_sync(FULL, m, o));
+    if (lane == 0) red[0][warp] = m;
     __syncthreads();
-    l += exp2f(sink - mc);
+    m = sink;
+#pragma unroll
+    for (int w = 0; w < DG_THREADS / 32; ++w) m = fmaxf(m, red[0][w]);
+    const float mc = m == -INFINITY ? 0.f : m;
+    const float wk = exp2f(mk - mc);
+    if (t < n) w_s[t] = wk;
+    const float lw = warp_sum(t < n ? wk * lk : 0.f);
+    if (lane == 0) red[1][warp] = lw;
+    __syncthreads();
+    float l = exp2f(sink - mc);
+#pragma unroll
+    for (int w = 0; w < DG_THREADS / 32; ++w) l += red[1][w];
     const float inv = l > 0.f ? 1.f / l : 0.f;
     __nv_bfloat16* out = (__nv_bfloat16*)p.out + (int64_t)b * p.o_bs + (int64_t)s * p.o_ss + (int64_t)h * p.o_hs;
-    for (int c = 4 * t; c < p.dv; c += 512) {
+    const int grp_t = t >> 7, tc = t & 127;
+    for (int c0 = 0; c0 < p.dv; c0 += 512) {
+        const int c = c0 + 4 * tc;
         float a[4] = {0.f, 0.f, 0.f, 0.f};
-        for (int k = 0; k < n; ++k) {
-            const float4 v = __ldcg(reinterpret_cast<const float4*>(part + k * part_floats + (int64_t)r * p.dv + c));
-            a[0] = fmaf(w_s[k], v.x, a[0]);
-            a[1] = fmaf(w_s[k], v.y, a[1]);
-            a[2] = fmaf(w_s[k], v.z, a[2]);
-            a[3] = fmaf(w_s[k], v.w, a[3]);
+        if (c < p.dv) {
+            const float* src = part + (int64_t)r * p.dv + c;
+#pragma unroll 8
+            for (int k = grp_t; k < n; k += DG_GROUPS) {
+                const float4 v = __ldcg(reinterpret_cast<const float4*>(src + k * part_floats));
+                const float w = w_s[k];
+                a[0] = fmaf(w, v.x, a[0]);
+                a[1] = fmaf(w, v.y, a[1]);
+                a[2] = fmaf(w, v.z, a[2]);
+                a[3] = fmaf(w, v.w, a[3]);
+            }
         }
+        if (c0 > 0) __syncthreads();
+        if (grp_t > 0) acc_s[grp_t - 1][tc] = make_float4(a[0], a[1], a[2], a[3]);
+        __syncthreads();
+        if (grp_t == 0 && c < p.dv) {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) a[e] *= inv;
-        store_vec<__nv_bfloat16, 4>(out + c, a);
+            for (int k = 0; k < DG_GROUPS - 1; ++k) {
+                const float4 v = acc_s[k][tc];
+                a[0] += v.x;
+                a[1] += v.y;
+                a[2] += v.z;
+                a[3] += v.w;
+            }
+#pragma unroll
+            for (int e = 0; e < 4; ++e) a[e] *= inv;
+            store_vec<__nv_bfloat16, 4>(out + c, a);
+        }
     }
 }
 
@@ -401,8 +435,8 @@ int launch_attn_decode_mma(const sk_attn_params& p, cudaStream_t st) {
     }
 #undef SK_DM
     if (int rc = check_launch("attn_decode_kernel")) return rc;
-    const cudaError_t e = launch_after(attn_decode_merge_kernel, dim3((unsigned)(p.S * (p.H / p.G)), (unsigned)p.G, (unsigned)p.B), dim3(128),
-                                       0, st, p, d.splits, d.groups, 16 * d.mt, d.part_floats);
+    const cudaError_t e = launch_after(attn_decode_merge_kernel, dim3((unsigned)(p.S * (p.H / p.G)), (unsigned)p.G, (unsigned)p.B),
+                                       dim3(DG_THREADS), 0, st, p, d.splits, d.groups, 16 * d.mt, d.part_floats);
     if (e != cudaSuccess) return fail(SK_ERR_CUDA, "attn_decode_merge_kernel: %s", cudaGetErrorString(e));
     return SK_OK;
 }

@@ -35,6 +35,12 @@ template <typename T, int V> __device__ __forceinline__ void load_vec(const T* p
         *reinterpret_cast<uint2*>(e) = a;
 #pragma unroll
         for (int i = 0; i < 4; ++i) r[i] = to_f32(e[i]);
+    } else if constexpr (V == 8 && sizeof(T) == 2) {
+        const uint4 a = *reinterpret_cast<const uint4*>(p);
+        T e[8];
+        *reinterpret_cast<uint4*>(e) = a;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) r[i] = to_f32(e[i]);
     } else {
 #pragma unroll
         for (int i = 0; i < V; ++i) r[i] = to_f32(p[i]);
@@ -48,6 +54,11 @@ template <typename T, int V> __device__ __forceinline__ void store_vec(T* p, con
 #pragma unroll
         for (int i = 0; i < 4; ++i) e[i] = from_f32<T>(r[i]);
         *reinterpret_cast<uint2*>(p) = *reinterpret_cast<uint2*>(e);
+    } else if constexpr (V == 8 && sizeof(T) == 2) {
+        T e[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) e[i] = from_f32<T>(r[i]);
+        *reinterpret_cast<uint4*>(p) = *reinterpret_cast<uint4*>(e);
     } else {
 #pragma unroll
         for (int i = 0; i < V; ++i) p[i] = from_f32<T>(r[i]);

@@ -121,6 +121,117 @@ latent_absorb_kernel(const T* __restrict__ q, int64_t q_ld, const T* __restrict_
     }
 }
 
+// The same for bf16 and a rank that is a multiple of 8: a CTA owns 128 columns of one head, 16 threads along them
+// (8 columns each) and 16 along the head's rows of W_uk, so that a thread's loads are few, wide and in flight together.
+template <int ROWS>
+__global__ void __launch_bounds__(256)
+latent_absorb_vec_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_ld, const __nv_bfloat16* __restrict__ uk, int64_t rows,
+                         int H, int dim, int rot, int rank, int out_ld, __nv_bfloat16* __restrict__ out) {
+    extern __shared__ float sm[];                                // q [ROWS][dim], partials [16][ROWS][128]
+    float* part = sm + ROWS * dim;
+    const int h = blockIdx.x, c0 = blockIdx.y * 128, t = threadIdx.x, cl = t & 15, dg = t >> 4;
+    const int64_t r0 = (int64_t)blockIdx.z * ROWS;
+    const int n = (int)(rows - r0 < ROWS ? rows - r0 : ROWS), c = c0 + cl * 8;
+    float acc[ROWS][8];
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[r][e] = 0.f;
+    const bool live = c < rank;
+    const __nv_bfloat16* w = uk + (int64_t)h * dim * rank + c;
+    constexpr int U = 8;                                         // rows of W_uk in flight per thread
+    uint4 wv[U];
+    auto load = [&](int d0) {
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int d = d0 + dg + 16 * u;
+            wv[u] = live && d < dim ? __ldg(reinterpret_cast<const uint4*>(w + (int64_t)d * rank)) : make_uint4(0, 0, 0, 0);
+        }
+    };
+    load(0);
+    for (int r = 0; r < n; ++r)
+        for (int d = t; d < dim; d += 256) sm[r * dim + d] = to_f32(q[(r0 + r) * q_ld + (int64_t)h * (dim + rot) + d]);
+    for (int r = n; r < ROWS; ++r)
+        for (int d = t; d < dim; d += 256) sm[r * dim + d] = 0.f;
+    __syncthreads();
+    for (int d0 = 0; d0 < dim; d0 += 16 * U) {
+        if (d0 > 0) load(d0);
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int d = d0 + dg + 16 * u;
+            if (d < dim) {
+                const uint32_t x[4] = {wv[u].x, wv[u].y, wv[u].z, wv[u].w};
+#pragma unroll
+                for (int r = 0; r < ROWS; ++r) {
+                    const float qv = sm[r * dim + d];
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        acc[r][2 * e] = fmaf(qv, __uint_as_float(x[e] << 16), acc[r][2 * e]);
+                        acc[r][2 * e + 1] = fmaf(qv, __uint_as_float(x[e] & 0xffff0000u), acc[r][2 * e + 1]);
+                    }
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) part[(dg * ROWS + r) * 128 + cl * 8 + e] = acc[r][e];
+    __syncthreads();
+    for (int j = t; j < n * 128; j += 256) {
+        const int r = j >> 7, cc = c0 + (j & 127);
+        if (cc < out_ld) {
+            float v = 0.f;
+            if (cc < rank) {
+#pragma unroll
+                for (int k = 0; k < 16; ++k) v += part[(k * ROWS + r) * 128 + (j & 127)];
+            } else if (cc < rank + rot) {
+                v = to_f32(q[(r0 + r) * q_ld + (int64_t)h * (dim + rot) + dim + (cc - rank)]);
+            }
+            out[((r0 + r) * H + h) * (int64_t)out_ld + cc] = __float2bfloat16_rn(v);
+        }
+    }
+}
+
+// out[row, h * vdim + e] for bf16 and a rank that is a multiple of 8: one warp per output element and row group
+template <int ROWS>
+__global__ void __launch_bounds__(128)
+latent_up_vec_kernel(const __nv_bfloat16* __restrict__ o, const __nv_bfloat16* __restrict__ uv, int64_t rows, int H, int vdim,
+                     int rank, __nv_bfloat16* __restrict__ out) {
+    const int lane = threadIdx.x & 31;
+    const int e = blockIdx.x * 4 + (threadIdx.x >> 5);
+    const int64_t r0 = (int64_t)blockIdx.y * ROWS;
+    if (e >= H * vdim) return;
+    const int h = e / vdim, n = (int)(rows - r0 < ROWS ? rows - r0 : ROWS);
+    const __nv_bfloat16* w = uv + (int64_t)e * rank;
+    float acc[ROWS];
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) acc[r] = 0.f;
+#pragma unroll 2
+    for (int j = 8 * lane; j < rank; j += 256) {
+        const uint4 wq = __ldg(reinterpret_cast<const uint4*>(w + j));
+        const uint32_t x[4] = {wq.x, wq.y, wq.z, wq.w};
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) {
+            if (r < n) {
+                const uint4 oq = *reinterpret_cast<const uint4*>(o + ((r0 + r) * H + h) * (int64_t)rank + j);
+                const uint32_t y[4] = {oq.x, oq.y, oq.z, oq.w};
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    acc[r] = fmaf(__uint_as_float(x[k] << 16), __uint_as_float(y[k] << 16), acc[r]);
+                    acc[r] = fmaf(__uint_as_float(x[k] & 0xffff0000u), __uint_as_float(y[k] & 0xffff0000u), acc[r]);
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r)
+        if (r < n) {
+            const float v = warp_sum(acc[r]);
+            if (lane == 0) out[(r0 + r) * (int64_t)H * vdim + e] = __float2bfloat16_rn(v);
+        }
+}
+
 // out[row, h * vdim + e] = <W_uv[h * vdim + e, :], o[row, h, :]>: one warp per output element and row group
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -174,6 +285,15 @@ int launch_latent_append(const sk_latent_params& p, cudaStream_t st) {
 
 int launch_latent_absorb(const void* q, int64_t q_ld, int dtype, const void* uk, int64_t rows, int H, int dim, int rot,
                          int rank, int out_ld, void* out, cudaStream_t st) {
+    if (dtype == SK_BF16 && rank % 8 == 0 && (uintptr_t)uk % 16 == 0 && dim <= 512) {
+        const __nv_bfloat16 *qb = (const __nv_bfloat16*)q, *ub = (const __nv_bfloat16*)uk;
+        const int R = rows == 1 ? 1 : 4;
+        dim3 grid((unsigned)H, (unsigned)((out_ld + 127) / 128), (unsigned)((rows + R - 1) / R));
+        const size_t smem = (size_t)(R * dim + 16 * R * 128) * sizeof(float);
+        if (R == 1) latent_absorb_vec_kernel<1><<<grid, 256, smem, st>>>(qb, q_ld, ub, rows, H, dim, rot, rank, out_ld, (__nv_bfloat16*)out);
+        else latent_absorb_vec_kernel<4><<<grid, 256, smem, st>>>(qb, q_ld, ub, rows, H, dim, rot, rank, out_ld, (__nv_bfloat16*)out);
+        return check_launch("latent_absorb_vec_kernel");
+    }
     dim3 grid((unsigned)H, (unsigned)((out_ld + 63) / 64), (unsigned)((rows + AB_ROWS - 1) / AB_ROWS));
     const size_t smem = (size_t)(AB_ROWS * dim + 8 * AB_ROWS * 64) * sizeof(float);
     if (smem > 48 * 1024) return fail(SK_ERR_UNSUPPORTED, "sk_latent_absorb: head size %d is too large", dim);
@@ -188,6 +308,14 @@ int launch_latent_absorb(const void* q, int64_t q_ld, int dtype, const void* uk,
 
 int launch_latent_up(const void* o, int dtype, const void* uv, int64_t rows, int H, int vdim, int rank, void* out,
                      cudaStream_t st) {
+    if (dtype == SK_BF16 && rank % 8 == 0 && (uintptr_t)uv % 16 == 0 && (uintptr_t)o % 16 == 0) {
+        const __nv_bfloat16 *ob = (const __nv_bfloat16*)o, *ub = (const __nv_bfloat16*)uv;
+        const int R = rows == 1 ? 1 : 4;
+        dim3 grid((unsigned)((H * vdim + 3) / 4), (unsigned)((rows + R - 1) / R));
+        if (R == 1) latent_up_vec_kernel<1><<<grid, 128, 0, st>>>(ob, ub, rows, H, vdim, rank, (__nv_bfloat16*)out);
+        else latent_up_vec_kernel<4><<<grid, 128, 0, st>>>(ob, ub, rows, H, vdim, rank, (__nv_bfloat16*)out);
+        return check_launch("latent_up_vec_kernel");
+    }
     dim3 grid((unsigned)((H * vdim + 7) / 8), (unsigned)((rows + AB_ROWS - 1) / AB_ROWS));
     if (dtype == SK_BF16)
         latent_up_kernel<<<grid, 256, 0, st>>>((const __nv_bfloat16*)o, (const __nv_bfloat16*)uv, rows, H, vdim, rank,

@@ -106,12 +106,10 @@ residual_norm_kernel(sk_residual_params p) {
 // gate_up row = [gate | up]: y = g * sigmoid(slope * g) * (u + 1), g and u clamped
 template <typename T, int V>
 __global__ void __launch_bounds__(256)
-glu_clamped_kernel(const T* __restrict__ gu, int64_t n_vec, int ff, int64_t ld, float limit, float slope,
-                   T* __restrict__ out) {
-    const int per_row = ff / V;
-    for (int64_t j = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; j < n_vec; j += (int64_t)gridDim.x * blockDim.x) {
-        const int64_t row = j / per_row;
-        const int i = (int)(j - row * per_row) * V;
+glu_clamped_kernel(const T* __restrict__ gu, int64_t rows, int ff, int64_t ld, float limit, float slope, T* __restrict__ out) {
+    const int i = (blockIdx.x * 256 + threadIdx.x) * V;
+    if (i >= ff) return;
+    for (int64_t row = blockIdx.y; row < rows; row += gridDim.y) {
         float g[V], u[V], r[V];
         load_vec<T, V>(gu + row * ld + i, g);
         load_vec<T, V>(gu + row * ld + ff + i, u);
@@ -182,12 +180,11 @@ int launch_residual_norm(const sk_residual_params& p, cudaStream_t st) {
 
 int launch_glu_clamped(const void* gate_up, int dtype, int64_t rows, int ff, int64_t ld, float limit, float slope,
                        void* out, cudaStream_t st) {
-    const bool v4 = ff % 4 == 0 && ld % 4 == 0;
-    const int64_t n = rows * (v4 ? ff / 4 : ff);
-    int64_t blocks = (n + 255) / 256;
-    if (blocks > (int64_t)sm_count() * 16) blocks = (int64_t)sm_count() * 16;
-#define SK_GLU(T, V) glu_clamped_kernel<T, V><<<(unsigned)blocks, 256, 0, st>>>((const T*)gate_up, n, ff, ld, limit, slope, (T*)out)
-    if (dtype == SK_BF16) { if (v4) SK_GLU(__nv_bfloat16, 4); else SK_GLU(__nv_bfloat16, 1); }
+    const bool v4 = ff % 4 == 0 && ld % 4 == 0, v8 = dtype == SK_BF16 && ff % 8 == 0 && ld % 8 == 0;
+    const int V = v8 ? 8 : (v4 ? 4 : 1);
+    dim3 grid((unsigned)((ff + 256 * V - 1) / (256 * V)), (unsigned)(rows < 32768 ? rows : 32768));
+#define SK_GLU(T, V) glu_clamped_kernel<T, V><<<grid, 256, 0, st>>>((const T*)gate_up, rows, ff, ld, limit, slope, (T*)out)
+    if (dtype == SK_BF16) { if (v8) SK_GLU(__nv_bfloat16, 8); else if (v4) SK_GLU(__nv_bfloat16, 4); else SK_GLU(__nv_bfloat16, 1); }
     else { if (v4) SK_GLU(float, 4); else SK_GLU(float, 1); }
 #undef SK_GLU
     return check_launch("glu_clamped_kernel");

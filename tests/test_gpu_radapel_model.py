@@ -21,7 +21,7 @@ F32, BF16 = torch.float32, torch.bfloat16
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 # rms of the logit error over the rms of the logits: (median, largest) over the positions.  The weights of
 # these tests make scores large, so that in bf16 a few positions amplify rounding; faults show in fp32.
-TOL = {F32: (2e-5, 4e-5), BF16: (3e-2, 3e-1)}
+TOL = {F32: (2e-5, 4e-5), BF16: (6e-2, 3e-1)}
 
 _plain = {}
 
