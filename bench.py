@@ -923,13 +923,13 @@ def measure_radapel_kernels(size, S, T, B, dev):
     add("latent attention, decode", time_op(lambda: ops.attn(qa, shared, shared[..., :K], scale=0.07, pos=pos, sink=sink, workspace=ws), flush),
         "flash_attn_with_kvcache, same context", fad, nbytes=B * T * (K + R) * 2, flops=lat_f, like_bytes=fab, like_flops=0.0)
     # ---- latent up- and down-projections of a decoded token
-    uk, uv, wo = rn(H * D, K), rn(H * D, K), rn(W, H * D)
-    qd, o, ho = rn(B, H * (D + R)), rn(B, H, K), rn(B, H * D)
-    gemv = time_op(lambda: torch.mm(ho, wo.t()), flush)
-    wb = W * H * D * 2
-    add("latent absorb, decode", time_op(lambda: ops.latent_absorb(qd, uk, H, D, R, K + R), flush), "torch.mm wo", gemv,
+    uk, uv = rn(H * D, K), rn(H * D, K)
+    qd, o, ho = rn(B, H * (D + R)), rn(B, H, K), rn(B, K)
+    gemv = time_op(lambda: torch.mm(ho, uv.t()), flush)
+    wb = H * D * K * 2
+    add("latent absorb, decode", time_op(lambda: ops.latent_absorb(qd, uk, H, D, R, K + R), flush), "torch.mm, as many bytes", gemv,
         nbytes=H * D * K * 2, like_bytes=wb)
-    add("latent up, decode", time_op(lambda: ops.latent_up(o, uv, D), flush), "torch.mm wo", gemv, nbytes=H * D * K * 2, like_bytes=wb)
+    add("latent up, decode", time_op(lambda: ops.latent_up(o, uv, D), flush), "torch.mm, as many bytes", gemv, nbytes=H * D * K * 2, like_bytes=wb)
     # ---- residual stream
     x, y, w = torch.randn(S, W, device=dev), rn(S, W), rn(W)
     xb = rn(S, W)

@@ -26,6 +26,8 @@ def distance_bucket(n: int, rows: int, far: float) -> int:
     half = rows // 2
     if n < half:
         return n
+    if n >= far:
+        return rows - 1
     step = math.floor(math.log(n / half) / math.log(far / half) * (rows - half) + 1e-12)
     return min(rows - 1, half + step)
 

@@ -3,17 +3,18 @@
 // All query rows that share a key/value head (rep heads x S tokens) are worked on together, 16 or 32 rows per
 // CTA, so a key is read once for all of them; with one key/value head for every query head - attention on
 // latent rows - this is what makes the step read each cache row once.  A CTA walks its share of 64-key tiles
-// (cp.async, double buffer), computes the scores with m16n8k16 MMAs (rows are too few for the 128-row tensor
+// (bulk copies, double buffer), computes the scores with m16n8k16 MMAs (rows are too few for the 128-row tensor
 // core tiles), keeps the running maximum per row and accumulates P V with each warp owning a slice of the value columns.
 // When the values are a prefix of the key rows in memory, the key tile serves as the value tile.  A second kernel
 // merges the partial results of the splits.  The live length is read on the device; the grid is fixed.
 #include "blocks.cuh"
+#include "tcgen05.cuh"
 #include "warp_mma.cuh"
 
 namespace sk {
 namespace {
 
-constexpr int DM_THREADS = 256, DM_WARPS = 8, DM_KEYS = 64;
+constexpr int DM_WARPS = 8, DM_KEYS = 64;      // warps per 16-row tile, keys per tile
 constexpr float DM_LOG2E = 1.4426950408889634f;
 constexpr int DM_MAX_SPLITS = 160;
 
@@ -32,7 +33,7 @@ bool dm_plan(const sk_attn_params& p, DmPlan* d) {
     if (p.dtype != SK_BF16 || p.dqk % 8 || p.dv % 8 || p.dv > 512 || p.dqk > 640 || p.kv_rows >= (int64_t)1 << 30) return false;
     const int rows = p.S * (p.H / p.G);
     d->mt = rows <= 16 ? 1 : 2;
-    d->nvt = p.dv <= 128 ? 2 : (p.dv <= 256 ? 4 : 8);
+    d->nvt = p.dv <= 128 * d->mt ? 2 : (p.dv <= 256 * d->mt ? 4 : 8);
     d->groups = (rows + 16 * d->mt - 1) / (16 * d->mt);
     d->shared_v = p.v == p.k && p.v_ts == p.k_ts && p.v_bs == p.k_bs && (p.G == 1 || p.v_hs == p.k_hs) && p.dv <= p.dqk;
     d->k_stride = (p.dqk + 15) / 16 * 16 + 8;
@@ -40,7 +41,7 @@ bool dm_plan(const sk_attn_params& p, DmPlan* d) {
     const size_t kv = (size_t)2 * DM_KEYS * (d->k_stride + (d->shared_v ? 0 : d->v_stride)) * 2;
     d->smem = kv + (size_t)16 * d->mt * d->k_stride * 2 + (size_t)16 * d->mt * (DM_KEYS + 8) * 2;
     if (d->smem > 220 * 1024) return false;
-    const int per_sm = d->smem > 110 * 1024 ? 1 : (d->smem > 72 * 1024 ? 2 : 3);
+    const int per_sm = d->smem > 110 * 1024 ? 1 : (d->smem > 72 * 1024 || d->mt == 2 ? 2 : 3);
     const int64_t ctas = (int64_t)d->groups * p.G * p.B, tiles = (p.kv_rows + DM_KEYS - 1) / DM_KEYS;
     int64_t sp = ((int64_t)sm_count() * per_sm) / ctas;
     if (sp > tiles) sp = tiles;
@@ -70,14 +71,16 @@ __device__ __forceinline__ DmRange dm_range(const sk_attn_params& p, int splits)
     return r;
 }
 
+// MT: 16-row tiles per CTA (8 MT warps: one key group of 8 per warp and tile), NVT: 8-column value tiles per warp
 template <int MT, int NVT>
-__global__ void __launch_bounds__(DM_THREADS)
+__global__ void __launch_bounds__(DM_WARPS * 32 * MT)
 attn_decode_kernel(sk_attn_params p, int splits, int groups, int shared_v, int k_stride, int v_stride, size_t part_floats) {
     extern __shared__ __align__(16) char dm_raw[];
-    __shared__ float wmax[2][16 * MT][DM_WARPS];
-    __shared__ float row_sum[16 * MT][DM_WARPS];
+    constexpr int ROWS = 16 * MT, WARPS = DM_WARPS * MT, THREADS = WARPS * 32, KG = 8;
+    __shared__ __align__(16) float wmax[2][ROWS][KG];
+    __shared__ float row_sum[ROWS][KG];
+    __shared__ uint64_t full[2];
     using bf = __nv_bfloat16;
-    constexpr int ROWS = 16 * MT, KG = DM_WARPS / MT, NT = MT;  // key groups of 8 NT keys
     bf* ks = reinterpret_cast<bf*>(dm_raw);                     // [2][64][k_stride]
     bf* vs = shared_v ? ks : ks + 2 * DM_KEYS * k_stride;
     bf* qs = vs + 2 * DM_KEYS * v_stride;                       // [ROWS][k_stride]
@@ -96,38 +99,40 @@ attn_decode_kernel(sk_attn_params p, int splits, int groups, int shared_v, int k
 
     const bf* kb = (const bf*)p.k + (int64_t)b * p.k_bs + (int64_t)g * p.k_hs;
     const bf* vb = (const bf*)p.v + (int64_t)b * p.v_bs + (int64_t)g * p.v_hs;
-    const int kc = p.dqk / 8, vc = p.dv / 8;                    // 16-byte chunks of a row
+    const int kc = p.dqk / 8;                                   // 16-byte pieces of a row
+    const uint32_t k_bytes = p.dqk * 2, v_bytes = p.dv * 2;
+    // warp 0: one bulk copy per key row (and value row); rows past the end repeat the last one and are masked
     auto fetch = [&](int tile, int stage) {
-        const int r0 = rg.lo + tile * DM_KEYS;
-        for (int r = warp; r < DM_KEYS; r += DM_WARPS) {         // a warp per row, lanes along it
-            const bool live = r0 + r <= rg.hi;
-            const int64_t row = live ? r0 + r : rg.hi;
-            const bf* src = kb + row * p.k_ts;
-            const uint32_t dst = saddr(ks + (stage * DM_KEYS + r) * k_stride);
-            for (int c = lane; c < kc; c += 32) cp16(dst + c * 16, src + c * 8, live);
-            if (!shared_v) {
-                const bf* vsrc = vb + row * p.v_ts;
-                const uint32_t vdst = saddr(vs + (stage * DM_KEYS + r) * v_stride);
-                for (int c = lane; c < vc; c += 32) cp16(vdst + c * 16, vsrc + c * 8, live);
-            }
+        if (lane == 0) mbar_expect(&full[stage], DM_KEYS * (k_bytes + (shared_v ? 0u : v_bytes)));
+        __syncwarp();
+#pragma unroll
+        for (int r = lane; r < DM_KEYS; r += 32) {
+            const int64_t row = min(rg.lo + tile * DM_KEYS + r, rg.hi);
+            bulk_load(ks + (stage * DM_KEYS + r) * k_stride, kb + row * p.k_ts, k_bytes, &full[stage]);
+            if (!shared_v) bulk_load(vs + (stage * DM_KEYS + r) * v_stride, vb + row * p.v_ts, v_bytes, &full[stage]);
         }
-        asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    fetch(t_beg, 0);
+    if (tid == 0) {
+        mbar_init_count(&full[0], 1);
+        mbar_init_count(&full[1], 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 0) {
+        __syncwarp();
+        fetch(t_beg, 0);
+    }
     const int k16 = (p.dqk + 15) / 16;
     // queries, and the zero columns that round a row up to 16
-    for (int e = tid; e < ROWS * k16 * 2; e += DM_THREADS) {
-        const int r = e / (k16 * 2), c = e - r * (k16 * 2), row = r_first + r;
-        uint4 v = make_uint4(0, 0, 0, 0);
-        if (row < n_rows && c < kc) {
-            const int s = row / rep, hh = row - s * rep;
-            v = *reinterpret_cast<const uint4*>((const bf*)p.q + (int64_t)b * p.q_bs + (int64_t)s * p.q_ss +
-                                                (int64_t)(g * rep + hh) * p.q_hs + c * 8);
+    for (int r = warp; r < ROWS; r += WARPS) {
+        const int row = r_first + r, s = row / rep, hh = row - s * rep;
+        const bf* src = (const bf*)p.q + (int64_t)b * p.q_bs + (int64_t)s * p.q_ss + (int64_t)(g * rep + hh) * p.q_hs;
+        for (int c = lane; c < k16 * 2; c += 32) {
+            const uint4 v = row < n_rows && c < kc ? *reinterpret_cast<const uint4*>(src + c * 8) : make_uint4(0, 0, 0, 0);
+            *reinterpret_cast<uint4*>(qs + r * k_stride + c * 8) = v;
         }
-        *reinterpret_cast<uint4*>(qs + r * k_stride + c * 8) = v;
     }
     if (k16 * 2 > kc)
-        for (int e = tid; e < 2 * DM_KEYS; e += DM_THREADS) *reinterpret_cast<uint4*>(ks + e * k_stride + kc * 8) = make_uint4(0, 0, 0, 0);
+        for (int e = tid; e < 2 * DM_KEYS; e += THREADS) *reinterpret_cast<uint4*>(ks + e * k_stride + kc * 8) = make_uint4(0, 0, 0, 0);
 
     // rows of this thread: scores (one 16-row tile per warp) and accumulators (all tiles)
     const int mtile = MT == 1 ? 0 : (warp & 1), kg = MT == 1 ? warp : (warp >> 1);
@@ -156,71 +161,57 @@ attn_decode_kernel(sk_attn_params p, int splits, int groups, int shared_v, int k
             for (int e = 0; e < 4; ++e) acc[t][v][e] = 0.f;
     }
     const int col0 = warp * NVT * 8;
+    bool in_time = true;
 
     for (int t = t_beg; t < t_end; ++t) {
-        const int stage = (t - t_beg) & 1;
+        const int it = t - t_beg, stage = it & 1;
         __syncthreads();                                        // the other stage is free
-        if (t + 1 < t_end) {
-            fetch(t + 1, stage ^ 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();
+        if (warp == 0 && t + 1 < t_end) fetch(t + 1, stage ^ 1);
+        if (in_time) in_time = mbar_wait_bounded(&full[stage], (uint32_t)((it >> 1) & 1));
         const bf* kt = ks + stage * DM_KEYS * k_stride;
         const bf* vt = vs + stage * DM_KEYS * v_stride;
-        // ---- scores of 16 rows x 8 NT keys, two independent sums along the head dimension
-        float sc[2][NT][4];
+        // ---- scores of 16 rows x 8 keys, two independent sums along the head dimension
+        float sc[2][4];
 #pragma unroll
         for (int u = 0; u < 2; ++u)
 #pragma unroll
-            for (int n = 0; n < NT; ++n)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) sc[u][n][e] = 0.f;
+            for (int e = 0; e < 4; ++e) sc[u][e] = 0.f;
         const uint32_t qa = saddr(qs + (mtile * 16 + (lane & 15)) * k_stride + (lane >> 4) * 8);
-        const uint32_t ka = NT == 1 ? saddr(kt + (kg * 8 + (lane & 7)) * k_stride + ((lane >> 3) & 1) * 8)
-                                    : saddr(kt + (kg * 16 + (lane & 7) + (lane >> 4) * 8) * k_stride + ((lane >> 3) & 1) * 8);
-        auto along = [&](float (&d)[NT][4], int k) {
-            uint32_t a[4];
-            ldsm4(qa + k * 32, a);
-            if constexpr (NT == 1) {
-                uint32_t b0, b1;
-                ldsm2(ka + k * 32, b0, b1);
-                mma16816(d[0], a, b0, b1);
-            } else {
-                uint32_t bb[4];
-                ldsm4(ka + k * 32, bb);
-                mma16816(d[0], a, bb[0], bb[1]);
-                mma16816(d[1], a, bb[2], bb[3]);
-            }
-        };
+        const uint32_t ka = saddr(kt + (kg * 8 + (lane & 7)) * k_stride + (lane >> 3) * 8);
         int kk = 0;
-#pragma unroll 2
-        for (; kk + 2 <= k16; kk += 2) {
-            along(sc[0], kk);
-            along(sc[1], kk + 1);
+#pragma unroll 4
+        for (; kk + 2 <= k16; kk += 2) {                        // 32 head dimensions at a time
+            uint32_t a0[4], a1[4], bb[4];
+            ldsm4(ka + kk * 32, bb);
+            ldsm4(qa + kk * 32, a0);
+            ldsm4(qa + kk * 32 + 32, a1);
+            mma16816(sc[0], a0, bb[0], bb[1]);
+            mma16816(sc[1], a1, bb[2], bb[3]);
         }
-        if (kk < k16) along(sc[0], kk);
-        const int r0 = rg.lo + t * DM_KEYS + kg * 8 * NT;       // key row of column 0 of this warp
+        if (kk < k16) {
+            uint32_t a0[4], b0, b1;
+            ldsm2(saddr(kt + (kg * 8 + (lane & 7)) * k_stride + ((lane >> 3) & 1) * 8) + kk * 32, b0, b1);
+            ldsm4(qa + kk * 32, a0);
+            mma16816(sc[0], a0, b0, b1);
+        }
+        const int r0 = rg.lo + t * DM_KEYS + kg * 8;            // key row of column 0 of this warp
         float mt[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-        for (int n = 0; n < NT; ++n)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int k = e >> 1, r = r0 + n * 8 + fc + (e & 1);
-                float v = (sc[0][n][e] + sc[1][n][e]) * sl;
-                if (r <= qi[k] && r >= lo[k] && r <= rg.hi) {
-                    if (brow[k] != nullptr) {
-                        const int64_t d = qi[k] - r;
-                        v = fmaf(__ldg(brow[k] + (d < p.bias_len ? d : p.bias_len - 1)), DM_LOG2E, v);
-                    }
-                } else {
-                    v = -INFINITY;
+        for (int e = 0; e < 4; ++e) {
+            const int k = e >> 1, r = r0 + fc + (e & 1);
+            float v = (sc[0][e] + sc[1][e]) * sl;
+            if (r <= qi[k] && r >= lo[k] && r <= rg.hi) {
+                if (brow[k] != nullptr) {
+                    const int64_t d = qi[k] - r;
+                    v = fmaf(__ldg(brow[k] + (d < p.bias_len ? d : p.bias_len - 1)), DM_LOG2E, v);
                 }
-                sc[0][n][e] = v;
-                mt[k] = fmaxf(mt[k], v);
+            } else {
+                v = -INFINITY;
             }
-        float (*wm)[DM_WARPS] = wmax[t & 1];
+            sc[0][e] = v;
+            mt[k] = fmaxf(mt[k], v);
+        }
+        float (*wm)[KG] = wmax[it & 1];
 #pragma unroll
         for (int k = 0; k < 2; ++k) {
             mt[k] = fmaxf(mt[k], __shfl_xor_sync(FULL, mt[k], 1));
@@ -228,40 +219,33 @@ attn_decode_kernel(sk_attn_params p, int splits, int groups, int shared_v, int k
             if ((lane & 3) == 0) wm[mtile * 16 + fr + 8 * k][kg] = mt[k];
         }
         __syncthreads();
-        // ---- new maxima: of the score rows for the weights, of all rows for the accumulators
-#pragma unroll
-        for (int k = 0; k < 2; ++k) {
-            float mn = m_own[k];
-#pragma unroll
-            for (int w = 0; w < KG; ++w) mn = fmaxf(mn, wm[mtile * 16 + fr + 8 * k][w]);
-            l_own[k] *= mn == -INFINITY ? 1.f : exp2f(m_own[k] - mn);
-            m_own[k] = mn;
-            const float mc = mn == -INFINITY ? 0.f : mn;
-#pragma unroll
-            for (int n = 0; n < NT; ++n) {
-                const float x = exp2f(sc[0][n][2 * k] - mc), y = exp2f(sc[0][n][2 * k + 1] - mc);
-                l_own[k] += x + y;
-                *reinterpret_cast<__nv_bfloat162*>(ps + (mtile * 16 + fr + 8 * k) * PS + kg * 8 * NT + n * 8 + fc) =
-                    __floats2bfloat162_rn(x, y);
-            }
-        }
+        // ---- new maxima of all rows; accumulators follow them, score rows become weights
 #pragma unroll
         for (int tt = 0; tt < MT; ++tt)
 #pragma unroll
             for (int k = 0; k < 2; ++k) {
-                float mn = m_acc[tt][k];
-#pragma unroll
-                for (int w = 0; w < KG; ++w) mn = fmaxf(mn, wm[tt * 16 + fr + 8 * k][w]);
+                const float4* w4 = reinterpret_cast<const float4*>(wm[tt * 16 + fr + 8 * k]);
+                const float4 x = w4[0], y = w4[1];
+                const float mn = fmaxf(fmaxf(fmaxf(fmaxf(x.x, x.y), fmaxf(x.z, x.w)), fmaxf(fmaxf(y.x, y.y), fmaxf(y.z, y.w))), m_acc[tt][k]);
                 if (mn != m_acc[tt][k]) {
-                    const float f = exp2f(m_acc[tt][k] - mn);   // mn is finite here
+                    const float f = exp2_fast(m_acc[tt][k] - mn);   // mn is finite here
 #pragma unroll
                     for (int v = 0; v < NVT; ++v) {
                         acc[tt][v][2 * k] *= f;
                         acc[tt][v][2 * k + 1] *= f;
                     }
+                    if (tt == mtile) l_own[k] *= f;
                     m_acc[tt][k] = mn;
                 }
+                if (tt == mtile) m_own[k] = mn;
             }
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const float mc = m_own[k] == -INFINITY ? 0.f : m_own[k];
+            const float x = exp2_fast(sc[0][2 * k] - mc), y = exp2_fast(sc[0][2 * k + 1] - mc);
+            l_own[k] += x + y;
+            *reinterpret_cast<__nv_bfloat162*>(ps + (mtile * 16 + fr + 8 * k) * PS + kg * 8 + fc) = __floats2bfloat162_rn(x, y);
+        }
         __syncthreads();
         // ---- P V: every warp all rows, its own value columns
         if (col0 < p.dv) {
@@ -284,6 +268,11 @@ attn_decode_kernel(sk_attn_params p, int splits, int groups, int shared_v, int k
                 }
             }
         }
+    }
+    if (!in_time) {                                             // a copy did not land: reported, and none left in flight
+        if (p.status != nullptr) atomicOr(p.status, SK_DEV_WAIT_TIMEOUT);
+        mbar_wait_bounded(&full[(t_end - 1 - t_beg) & 1], (uint32_t)(((t_end - 1 - t_beg) >> 1) & 1));
+        if (t_end - t_beg > 1) mbar_wait_bounded(&full[(t_end - t_beg) & 1], (uint32_t)(((t_end - 2 - t_beg) >> 1) & 1));
     }
     // ---- partial result: rows x (dv sums | maximum | sum of weights)
 #pragma unroll
@@ -319,16 +308,16 @@ attn_decode_kernel(sk_attn_params p, int splits, int groups, int shared_v, int k
         }
 }
 
-// One CTA per query row: merge the splits that exist, add the sink, divide.  Groups of 128 threads take every
-// fourth split; a thread of a group owns four value columns at a time.
-constexpr int DG_THREADS = 512, DG_GROUPS = DG_THREADS / 128;
-__global__ void __launch_bounds__(DG_THREADS)
-attn_decode_merge_kernel(sk_attn_params p, int splits, int groups, int rows_per_group, size_t part_floats) {
+// One CTA per query row and 128 value columns: merge the splits that exist, add the sink, divide.  A warp takes
+// every sixteenth split, a lane four columns.
+constexpr int DG_WARPS = 16, DG_COLS = 128;
+__global__ void __launch_bounds__(DG_WARPS * 32)
+attn_decode_merge_kernel(sk_attn_params p, int splits, int groups, int rows_per_group, size_t part_floats, int col_blocks) {
     __shared__ float w_s[DM_MAX_SPLITS];
-    __shared__ float red[2][DG_THREADS / 32];
-    __shared__ float4 acc_s[DG_GROUPS - 1][128];
-    const int rep = p.H / p.G, row = blockIdx.x, g = blockIdx.y, b = blockIdx.z, t = threadIdx.x;
-    const int warp = t >> 5, lane = t & 31;
+    __shared__ float red[2][DG_WARPS];
+    __shared__ float4 acc_s[DG_WARPS][32];
+    const int rep = p.H / p.G, row = blockIdx.x / col_blocks, g = blockIdx.y, b = blockIdx.z, t = threadIdx.x;
+    const int warp = t >> 5, lane = t & 31, c = (blockIdx.x - row * col_blocks) * DG_COLS + 4 * lane;
     const int s = row / rep, h = g * rep + row - s * rep, grp = row / rows_per_group, r = row - grp * rows_per_group;
     const float sink = p.sink != nullptr ? p.sink[h] * DM_LOG2E : -INFINITY;
     const DmRange rg = dm_range(p, splits);
@@ -341,6 +330,14 @@ attn_decode_merge_kernel(sk_attn_params p, int splits, int groups, int rows_per_
         mk = __ldcg(stat + t * part_floats);
         lk = __ldcg(stat + t * part_floats + rows_per_group);
     }
+    constexpr int U = DM_MAX_SPLITS / DG_WARPS;                 // splits of a warp, all requested at once
+    float4 v[U];
+#pragma unroll
+    for (int k = 0; k < U; ++k) {
+        const int sp = warp + k * DG_WARPS;
+        v[k] = sp < n && c < p.dv ? __ldcg(reinterpret_cast<const float4*>(part + sp * part_floats + (int64_t)r * p.dv + c))
+                                  : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
     float m = fmaxf(mk, sink);
 #pragma unroll
     for (int o = 16; o >= 1; o >>= 1) m = fmaxf(m, __shfl_xor_sync(FULL, m, o));
@@ -348,50 +345,39 @@ attn_decode_merge_kernel(sk_attn_params p, int splits, int groups, int rows_per_
     __syncthreads();
     m = sink;
 #pragma unroll
-    for (int w = 0; w < DG_THREADS / 32; ++w) m = fmaxf(m, red[0][w]);
+    for (int w = 0; w < DG_WARPS; ++w) m = fmaxf(m, red[0][w]);
     const float mc = m == -INFINITY ? 0.f : m;
     const float wk = exp2f(mk - mc);
-    if (t < n) w_s[t] = wk;
+    if (t < DM_MAX_SPLITS) w_s[t] = t < n ? wk : 0.f;
     const float lw = warp_sum(t < n ? wk * lk : 0.f);
     if (lane == 0) red[1][warp] = lw;
     __syncthreads();
-    float l = exp2f(sink - mc);
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-    for (int w = 0; w < DG_THREADS / 32; ++w) l += red[1][w];
-    const float inv = l > 0.f ? 1.f / l : 0.f;
-    __nv_bfloat16* out = (__nv_bfloat16*)p.out + (int64_t)b * p.o_bs + (int64_t)s * p.o_ss + (int64_t)h * p.o_hs;
-    const int grp_t = t >> 7, tc = t & 127;
-    for (int c0 = 0; c0 < p.dv; c0 += 512) {
-        const int c = c0 + 4 * tc;
-        float a[4] = {0.f, 0.f, 0.f, 0.f};
-        if (c < p.dv) {
-            const float* src = part + (int64_t)r * p.dv + c;
-#pragma unroll 8
-            for (int k = grp_t; k < n; k += DG_GROUPS) {
-                const float4 v = __ldcg(reinterpret_cast<const float4*>(src + k * part_floats));
-                const float w = w_s[k];
-                a[0] = fmaf(w, v.x, a[0]);
-                a[1] = fmaf(w, v.y, a[1]);
-                a[2] = fmaf(w, v.z, a[2]);
-                a[3] = fmaf(w, v.w, a[3]);
-            }
+    for (int k = 0; k < U; ++k) {
+        const float w = w_s[warp + k * DG_WARPS];
+        a.x = fmaf(w, v[k].x, a.x);
+        a.y = fmaf(w, v[k].y, a.y);
+        a.z = fmaf(w, v[k].z, a.z);
+        a.w = fmaf(w, v[k].w, a.w);
+    }
+    acc_s[warp][lane] = a;
+    __syncthreads();
+    if (warp == 0 && c < p.dv) {
+        float l = exp2f(sink - mc), o[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int w = 0; w < DG_WARPS; ++w) {
+            const float4 x = acc_s[w][lane];
+            l += red[1][w];
+            o[0] += x.x;
+            o[1] += x.y;
+            o[2] += x.z;
+            o[3] += x.w;
         }
-        if (c0 > 0) __syncthreads();
-        if (grp_t > 0) acc_s[grp_t - 1][tc] = make_float4(a[0], a[1], a[2], a[3]);
-        __syncthreads();
-        if (grp_t == 0 && c < p.dv) {
+        const float inv = l > 0.f ? 1.f / l : 0.f;
 #pragma unroll
-            for (int k = 0; k < DG_GROUPS - 1; ++k) {
-                const float4 v = acc_s[k][tc];
-                a[0] += v.x;
-                a[1] += v.y;
-                a[2] += v.z;
-                a[3] += v.w;
-            }
-#pragma unroll
-            for (int e = 0; e < 4; ++e) a[e] *= inv;
-            store_vec<__nv_bfloat16, 4>(out + c, a);
-        }
+        for (int e = 0; e < 4; ++e) o[e] *= inv;
+        store_vec<__nv_bfloat16, 4>((__nv_bfloat16*)p.out + (int64_t)b * p.o_bs + (int64_t)s * p.o_ss + (int64_t)h * p.o_hs + c, o);
     }
 }
 
@@ -422,7 +408,7 @@ int launch_attn_decode_mma(const sk_attn_params& p, cudaStream_t st) {
         auto kern = attn_decode_kernel<MT, NVT>;                                                                         \
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)d.smem);      \
         if (e != cudaSuccess) return fail(SK_ERR_CUDA, "attn_decode_kernel smem attribute: %s", cudaGetErrorString(e));  \
-        kern<<<grid, DM_THREADS, d.smem, st>>>(p, d.splits, d.groups, (int)d.shared_v, d.k_stride, d.v_stride, d.part_floats); \
+        kern<<<grid, DM_WARPS * 32 * MT, d.smem, st>>>(p, d.splits, d.groups, (int)d.shared_v, d.k_stride, d.v_stride, d.part_floats); \
     } while (0)
     if (d.mt == 1) {
         if (d.nvt == 2) SK_DM(1, 2);
@@ -430,13 +416,13 @@ int launch_attn_decode_mma(const sk_attn_params& p, cudaStream_t st) {
         else SK_DM(1, 8);
     } else {
         if (d.nvt == 2) SK_DM(2, 2);
-        else if (d.nvt == 4) SK_DM(2, 4);
-        else SK_DM(2, 8);
+        else SK_DM(2, 4);
     }
 #undef SK_DM
     if (int rc = check_launch("attn_decode_kernel")) return rc;
-    const cudaError_t e = launch_after(attn_decode_merge_kernel, dim3((unsigned)(p.S * (p.H / p.G)), (unsigned)p.G, (unsigned)p.B),
-                                       dim3(DG_THREADS), 0, st, p, d.splits, d.groups, 16 * d.mt, d.part_floats);
+    const int col_blocks = (p.dv + DG_COLS - 1) / DG_COLS;
+    const cudaError_t e = launch_after(attn_decode_merge_kernel, dim3((unsigned)(p.S * (p.H / p.G) * col_blocks), (unsigned)p.G, (unsigned)p.B),
+                                       dim3(DG_WARPS * 32), 0, st, p, d.splits, d.groups, 16 * d.mt, d.part_floats, col_blocks);
     if (e != cudaSuccess) return fail(SK_ERR_CUDA, "attn_decode_merge_kernel: %s", cudaGetErrorString(e));
     return SK_OK;
 }

@@ -45,12 +45,6 @@ struct FpShape {            // what the kernel needs beside the tensor maps
     float scale_log2;
 };
 
-__device__ __forceinline__ float exp2_fast(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-
 template <bool BIAS>
 __global__ void __launch_bounds__(FP_THREADS, 1)
 attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,

@@ -65,7 +65,19 @@ template <typename T, int V> __device__ __forceinline__ void store_vec(T* p, con
     }
 }
 
-__device__ __forceinline__ float silu_f32(float x) { return x / (1.f + expf(-x)); }
+__device__ __forceinline__ float exp2_fast(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+// activations: full fp32 accuracy for fp32 models; for bf16 ones the hardware exponential and division,
+// whose error is far below the rounding of the result
+template <typename T> __device__ __forceinline__ float sigmoid_scaled(float x, float slope) {
+    if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-slope * x));
+    else return 1.f / (1.f + expf(-slope * x));
+}
+template <typename T> __device__ __forceinline__ float silu(float x) { return x * sigmoid_scaled<T>(x, 1.f); }
 __device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 // position of the first token of a portion: on the device (decode) or given by the host

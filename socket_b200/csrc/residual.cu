@@ -116,7 +116,7 @@ glu_clamped_kernel(const T* __restrict__ gu, int64_t rows, int ff, int64_t ld, f
 #pragma unroll
         for (int e = 0; e < V; ++e) {
             const float a = fminf(g[e], limit), b = fminf(fmaxf(u[e], -limit), limit);
-            r[e] = a / (1.f + expf(-slope * a)) * (b + 1.f);
+            r[e] = a * sigmoid_scaled<T>(a, slope) * (b + 1.f);
         }
         store_vec<T, V>(out + row * ff + i, r);
     }

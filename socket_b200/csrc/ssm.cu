@@ -45,21 +45,26 @@ ssm_conv_kernel(sk_ssm_params p) {
             for (int e = 0; e < V; ++e) wt[j][e] = to_f32(w[(int64_t)(ch + e) * K + j]);
 #pragma unroll
         for (int j = 1; j < K; ++j) conv_tap_input<T, V>(p, b, s0 - K + j, ch, fresh, channels, win[j]);
-        for (int s = s0; s < s1; ++s) {
-            float acc[V];
+        constexpr int U = 4;                                      // tokens requested together
+        for (int s = s0; s < s1; s += U) {
+            float in[U][V];
 #pragma unroll
-            for (int j = 0; j + 1 < K; ++j)
+            for (int u = 0; u < U; ++u) conv_tap_input<T, V>(p, b, s + u < s1 ? s + u : s1 - 1, ch, fresh, channels, in[u]);
 #pragma unroll
-                for (int e = 0; e < V; ++e) win[j][e] = win[j + 1][e];
-            conv_tap_input<T, V>(p, b, s, ch, fresh, channels, win[K - 1]);
+            for (int u = 0; u < U; ++u) {
+                float acc[V];
 #pragma unroll
-            for (int e = 0; e < V; ++e) {
-                acc[e] = bias[e];
+                for (int e = 0; e < V; ++e) {
 #pragma unroll
-                for (int j = 0; j < K; ++j) acc[e] = fmaf(wt[j][e], win[j][e], acc[e]);
-                acc[e] = silu_f32(acc[e]);
+                    for (int j = 0; j + 1 < K; ++j) win[j][e] = win[j + 1][e];
+                    win[K - 1][e] = in[u][e];
+                    acc[e] = bias[e];
+#pragma unroll
+                    for (int j = 0; j < K; ++j) acc[e] = fmaf(wt[j][e], win[j][e], acc[e]);
+                    acc[e] = silu<T>(acc[e]);
+                }
+                if (s + u < s1) store_vec<T, V>((T*)p.xbc + ((int64_t)b * p.S + s + u) * p.xbc_ld + ch, acc);
             }
-            store_vec<T, V>((T*)p.xbc + ((int64_t)b * p.S + s) * p.xbc_ld + ch, acc);
         }
     } else
     for (int s = s0; s < s1; ++s) {
@@ -73,7 +78,7 @@ ssm_conv_kernel(sk_ssm_params p) {
             for (int e = 0; e < V; ++e) acc[e] = fmaf(to_f32(w[(int64_t)(ch + e) * p.taps + j]), in[e], acc[e]);
         }
 #pragma unroll
-        for (int e = 0; e < V; ++e) acc[e] = silu_f32(acc[e]);
+        for (int e = 0; e < V; ++e) acc[e] = silu<T>(acc[e]);
         store_vec<T, V>((T*)p.xbc + ((int64_t)b * p.S + s) * p.xbc_ld + ch, acc);
     }
     // one token: this thread is the only reader of its channels' carried inputs, so it moves them on itself
@@ -180,7 +185,7 @@ gated_group_norm_kernel(const T* __restrict__ y, const T* __restrict__ z, int64_
             load_vec<T, V>(z + row * z_ld + c0 + i, zz);
 #pragma unroll
             for (int e = 0; e < V; ++e) {
-                v[n][e] *= silu_f32(zz[e]);
+                v[n][e] *= silu<T>(zz[e]);
                 ss = fmaf(v[n][e], v[n][e], ss);
             }
         }
@@ -195,48 +200,6 @@ gated_group_norm_kernel(const T* __restrict__ y, const T* __restrict__ z, int64_
 #pragma unroll
             for (int e = 0; e < V; ++e) v[n][e] *= inv * ww[e];
             store_vec<T, V>(out + row * inner + c0 + i, v[n]);
-        }
-    }
-}
-
-// The same with one warp per (row, part), 8-element vectors: parts of up to 256 NV elements (bf16)
-template <int NV>
-__global__ void __launch_bounds__(256)
-gated_group_norm_warp_kernel(const __nv_bfloat16* __restrict__ y, const __nv_bfloat16* __restrict__ z, int64_t z_ld,
-                             const __nv_bfloat16* __restrict__ w, int64_t rows, int inner, int part, float eps,
-                             __nv_bfloat16* __restrict__ out) {
-    using T = __nv_bfloat16;
-    const int lane = threadIdx.x & 31, parts = inner / part;
-    const int64_t u = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5), row = u / parts;
-    if (row >= rows) return;
-    const int c0 = (int)(u - row * parts) * part;
-    float v[NV][8], zz[NV][8], ss = 0.f;
-#pragma unroll
-    for (int n = 0; n < NV; ++n) {
-        const int i = (n * 32 + lane) * 8;
-        if (i < part) {
-            load_vec<T, 8>(y + row * inner + c0 + i, v[n]);
-            load_vec<T, 8>(z + row * z_ld + c0 + i, zz[n]);
-        }
-    }
-#pragma unroll
-    for (int n = 0; n < NV; ++n)
-        if ((n * 32 + lane) * 8 < part)
-#pragma unroll
-            for (int e = 0; e < 8; ++e) {
-                v[n][e] *= silu_f32(zz[n][e]);
-                ss = fmaf(v[n][e], v[n][e], ss);
-            }
-    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)part + eps);
-#pragma unroll
-    for (int n = 0; n < NV; ++n) {
-        const int i = (n * 32 + lane) * 8;
-        if (i < part) {
-            float ww[8];
-            load_vec<T, 8>(w + c0 + i, ww);
-#pragma unroll
-            for (int e = 0; e < 8; ++e) v[n][e] *= inv * ww[e];
-            store_vec<T, 8>(out + row * inner + c0 + i, v[n]);
         }
     }
 }
@@ -274,11 +237,15 @@ template <typename T> int steps_dispatch(const sk_ssm_params& p, cudaStream_t st
 template <typename T> int conv_dispatch(const sk_ssm_params& p, cudaStream_t st) {
     const int channels = p.H * p.P + 2 * p.G * p.N;
     // the first column of [x | B | C] sits behind the gate's H * P columns
-    const bool v4 = channels % 4 == 0 && p.in_ld % 4 == 0 && p.xbc_ld % 4 == 0 && (uintptr_t)p.xbc_in % (4 * sizeof(T)) == 0;
-    const int V = v4 ? 4 : 1;
+    auto vec = [&](int v) {
+        return channels % v == 0 && p.in_ld % v == 0 && p.xbc_ld % v == 0 && (uintptr_t)p.xbc_in % (v * sizeof(T)) == 0;
+    };
+    const int V = sizeof(T) == 2 && vec(8) && p.taps == 4 ? 8 : (vec(4) ? 4 : 1);
     dim3 grid((unsigned)((channels + 128 * V - 1) / (128 * V)), (unsigned)((p.S + CONV_TOK - 1) / CONV_TOK), (unsigned)p.B);
-    if (v4 && p.taps == 4) ssm_conv_kernel<T, 4, 4><<<grid, 128, 0, st>>>(p);
-    else if (v4) ssm_conv_kernel<T, 4, 0><<<grid, 128, 0, st>>>(p);
+    if (V == 8) {
+        if constexpr (sizeof(T) == 2) ssm_conv_kernel<T, 8, 4><<<grid, 128, 0, st>>>(p);
+    } else if (V == 4 && p.taps == 4) ssm_conv_kernel<T, 4, 4><<<grid, 128, 0, st>>>(p);
+    else if (V == 4) ssm_conv_kernel<T, 4, 0><<<grid, 128, 0, st>>>(p);
     else ssm_conv_kernel<T, 1, 0><<<grid, 128, 0, st>>>(p);
     if (int rc = check_launch("ssm_conv_kernel")) return rc;
     if (p.S > 1 && p.taps > 1) {
@@ -302,14 +269,8 @@ int launch_gated_group_norm(const void* y, const void* z, int64_t z_ld, const vo
                             int inner, int parts, float eps, void* out, cudaStream_t st) {
     const int part = inner / parts;
     const bool v4 = part % 4 == 0 && z_ld % 4 == 0;
-    if (dtype == SK_BF16 && part % 8 == 0 && z_ld % 8 == 0 && part <= 1024 && rows * parts >= 1024 && (uintptr_t)z % 16 == 0) {
-        const unsigned grid = (unsigned)((rows * parts + 7) / 8);
-        const __nv_bfloat16 *yb = (const __nv_bfloat16*)y, *zb = (const __nv_bfloat16*)z, *wb = (const __nv_bfloat16*)w;
-        if (part <= 256) gated_group_norm_warp_kernel<1><<<grid, 256, 0, st>>>(yb, zb, z_ld, wb, rows, inner, part, eps, (__nv_bfloat16*)out);
-        else if (part <= 512) gated_group_norm_warp_kernel<2><<<grid, 256, 0, st>>>(yb, zb, z_ld, wb, rows, inner, part, eps, (__nv_bfloat16*)out);
-        else gated_group_norm_warp_kernel<4><<<grid, 256, 0, st>>>(yb, zb, z_ld, wb, rows, inner, part, eps, (__nv_bfloat16*)out);
-        return check_launch("gated_group_norm_warp_kernel");
-    }
+    if (dtype == SK_BF16 && part % 8 == 0 && z_ld % 8 == 0 && (uintptr_t)z % 16 == 0)
+        return norm_dispatch<__nv_bfloat16, 8>(y, z, z_ld, w, rows, inner, parts, eps, out, st);
     if (dtype == SK_BF16)
         return v4 ? norm_dispatch<__nv_bfloat16, 4>(y, z, z_ld, w, rows, inner, parts, eps, out, st)
                   : norm_dispatch<__nv_bfloat16, 1>(y, z, z_ld, w, rows, inner, parts, eps, out, st);

@@ -87,7 +87,7 @@ class ChunkedAttention(nn.Module):
         self.wqkv = projection(padded_rows(sum(self.sizes)), width)
         self.wo = projection(width, heads * vdim)
         self.rel = nn.Parameter(torch.zeros(bias_rows, heads), requires_grad=False)
-        self.register_buffer("bias", torch.zeros(heads, math.ceil(bias_max) + 1), persistent=False)
+        self.register_buffer("bias", torch.zeros(heads, max(math.ceil(bias_max), bias_rows) + 1), persistent=False)
 
     def tensors(self) -> dict:
         q, k, v = self.wqkv[:sum(self.sizes)].split(self.sizes)

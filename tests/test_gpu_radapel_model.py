@@ -244,3 +244,17 @@ def test_trace_runner_as_a_process(dtype, tmp_path):
     wa, wb = _want(name, a), _want(name, b)
     dt = getattr(torch, dtype)
     _check(got[0], wa[[0, 39]], dt), _check(got[2], wa[60:], dt), _check(got[3], wb, dt)
+
+
+def test_generation_from_the_command_line(tmp_path):
+    """Same tokens as generate() in this process; two prompts as a batch."""
+    name = "looped"
+    (tmp_path / "config.json").write_text(json.dumps(CONFIGS[name]))
+    write_safetensors(str(tmp_path / "model.safetensors"), _weights(name))
+    prompts = [_tokens(name, 30, seed=1), _tokens(name, 30, seed=2)]
+    want, _ = generate(_model(name, F32), torch.tensor(prompts), 8)
+    text = ";".join(",".join(map(str, p)) for p in prompts)
+    r = subprocess.run([sys.executable, "-m", "socket_b200.generate", "--model", str(tmp_path), "--tokens", text, "--new", "8",
+                        "--dtype", "float32", "--prefill-chunk", "13"], capture_output=True, text=True, timeout=300, cwd=ROOT)
+    assert r.returncode == 0, r.stderr[-2000:]
+    assert [[int(t) for t in line.split(",")] for line in r.stdout.split()] == want[:, 30:].tolist()

@@ -155,16 +155,16 @@ def test_positions_outside_the_caches_are_refused():
 
 
 # ------------------------------------------------------------------------------- distance buckets, angles
-@pytest.mark.parametrize("rows,far", [(16, 50), (16, 128), (10, 160), (9, 77), (32, 1000), (6, 4.5), (8, 9)])
+@pytest.mark.parametrize("rows,far", [(16, 50), (16, 128), (10, 160), (9, 77), (32, 1000), (6, 4.5), (8, 9), (20, 6)])
 def test_distance_buckets(rows, far):
-    top = math.ceil(far)
+    top = max(math.ceil(far), rows)
     got = distance_buckets(top, rows, far).tolist()
     half = rows // 2
     assert got[:half] == list(range(half)) and got[-1] == rows - 1
     assert all(b - a >= 0 for a, b in zip(got, got[1:]))
     assert got == [orc.distance_bucket(n, rows, far) for n in range(top + 1)]
     for n in range(half, top + 1):                     # the edge rule in exact integers where it is one
-        if isinstance(far, int):
+        if isinstance(far, int) and far > half:
             k = 0
             while half + k < rows - 1 and n ** (rows - half) * half ** (k + 1) >= far ** (k + 1) * half ** (rows - half):
                 k += 1
@@ -221,3 +221,11 @@ def test_plain_latent_attention_depends_on_distance_only():
     q, k = torch.randn(8, dtype=torch.float64), torch.randn(8, dtype=torch.float64)
     at = lambda x, p: orc.rotate_pairs(x, p, m["rot"]["dims"], m["rot"]["base"])  # noqa: E731
     torch.testing.assert_close(at(q, 40) @ at(k, 33), at(q, 7) @ at(k, 0))
+
+
+def test_prompt_parsing_of_the_command_line():
+    from socket_b200.generate import parse_prompts
+    assert parse_prompts("5,17,3") == [[5, 17, 3]] and parse_prompts("1,2;3,4") == [[1, 2], [3, 4]]
+    for bad in ("", "1,2;3"):
+        with pytest.raises(ValueError):
+            parse_prompts(bad)
