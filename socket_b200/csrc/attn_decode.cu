@@ -3,18 +3,20 @@
 // All query rows that share a key/value head (rep heads x S tokens) are worked on together, 16 or 32 rows per
 // CTA, so a key is read once for all of them; with one key/value head for every query head - attention on
 // latent rows - this is what makes the step read each cache row once.  A CTA walks its share of 64-key tiles
-// (bulk copies, double buffer), computes the scores with m16n8k16 MMAs (rows are too few for the 128-row tensor
+// (TMA, 128-byte swizzle, double buffer), computes the scores with m16n8k16 MMAs (rows are too few for the 128-row tensor
 // core tiles), keeps the running maximum per row and accumulates P V with each warp owning a slice of the value columns.
 // When the values are a prefix of the key rows in memory, the key tile serves as the value tile.  A second kernel
 // merges the partial results of the splits.  The live length is read on the device; the grid is fixed.
 #include "blocks.cuh"
 #include "tcgen05.cuh"
+#include "tensor_map.cuh"
 #include "warp_mma.cuh"
 
 namespace sk {
 namespace {
 
 constexpr int DM_WARPS = 8, DM_KEYS = 64;      // warps per 16-row tile, keys per tile
+constexpr uint32_t DM_PANEL = DM_KEYS * 128;             // 64 keys x 64 columns
 constexpr float DM_LOG2E = 1.4426950408889634f;
 constexpr int DM_MAX_SPLITS = 160;
 
@@ -24,7 +26,8 @@ struct DmPlan {
     int groups;             // row groups per (batch, key/value head)
     int splits;
     bool shared_v;
-    int k_stride, v_stride; // elements per shared-memory row
+    int q_stride;           // elements per shared-memory row of the queries
+    int np, nvp;            // 64-column panels of a key and of a value tile (0: the key tile serves)
     size_t smem;
     size_t part_floats;     // per split: 16 mt rows x (dv + 2)
 };
@@ -36,10 +39,10 @@ bool dm_plan(const sk_attn_params& p, DmPlan* d) {
     d->nvt = p.dv <= 128 * d->mt ? 2 : (p.dv <= 256 * d->mt ? 4 : 8);
     d->groups = (rows + 16 * d->mt - 1) / (16 * d->mt);
     d->shared_v = p.v == p.k && p.v_ts == p.k_ts && p.v_bs == p.k_bs && (p.G == 1 || p.v_hs == p.k_hs) && p.dv <= p.dqk;
-    d->k_stride = (p.dqk + 15) / 16 * 16 + 8;
-    d->v_stride = d->shared_v ? d->k_stride : (p.dv + 15) / 16 * 16 + 8;
-    const size_t kv = (size_t)2 * DM_KEYS * (d->k_stride + (d->shared_v ? 0 : d->v_stride)) * 2;
-    d->smem = kv + (size_t)16 * d->mt * d->k_stride * 2 + (size_t)16 * d->mt * (DM_KEYS + 8) * 2;
+    d->q_stride = (p.dqk + 15) / 16 * 16 + 8;
+    d->np = (p.dqk + 63) / 64;
+    d->nvp = d->shared_v ? 0 : (p.dv + 63) / 64;
+    d->smem = 1024 + (size_t)2 * (d->np + d->nvp) * DM_PANEL + (size_t)16 * d->mt * d->q_stride * 2 + (size_t)16 * d->mt * (DM_KEYS + 8) * 2;
     if (d->smem > 220 * 1024) return false;
     const int per_sm = d->smem > 110 * 1024 ? 1 : (d->smem > 72 * 1024 || d->mt == 2 ? 2 : 3);
     const int64_t ctas = (int64_t)d->groups * p.G * p.B, tiles = (p.kv_rows + DM_KEYS - 1) / DM_KEYS;
@@ -74,18 +77,20 @@ __device__ __forceinline__ DmRange dm_range(const sk_attn_params& p, int splits)
 // MT: 16-row tiles per CTA (8 MT warps: one key group of 8 per warp and tile), NVT: 8-column value tiles per warp
 template <int MT, int NVT>
 __global__ void __launch_bounds__(DM_WARPS * 32 * MT)
-attn_decode_kernel(sk_attn_params p, int splits, int groups, int shared_v, int k_stride, int v_stride, size_t part_floats) {
-    extern __shared__ __align__(16) char dm_raw[];
+attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const __grid_constant__ sk_attn_params p,
+                   int splits, int groups, int np, int nvp, int q_stride, size_t part_floats) {
+    extern __shared__ char dm_raw[];
     constexpr int ROWS = 16 * MT, WARPS = DM_WARPS * MT, THREADS = WARPS * 32, KG = 8;
     __shared__ __align__(16) float wmax[2][ROWS][KG];
     __shared__ float row_sum[ROWS][KG];
     __shared__ uint64_t full[2];
     using bf = __nv_bfloat16;
-    bf* ks = reinterpret_cast<bf*>(dm_raw);                     // [2][64][k_stride]
-    bf* vs = shared_v ? ks : ks + 2 * DM_KEYS * k_stride;
-    bf* qs = vs + 2 * DM_KEYS * v_stride;                       // [ROWS][k_stride]
+    char* ks = reinterpret_cast<char*>((reinterpret_cast<uintptr_t>(dm_raw) + 1023) & ~(uintptr_t)1023);   // [2][panel][64][128 B]
+    char* vs = nvp > 0 ? ks + 2 * np * DM_PANEL : ks;
+    const int v_panels = nvp > 0 ? nvp : np;                    // stage stride of the value tiles
+    bf* qs = reinterpret_cast<bf*>(ks + 2 * (np + nvp) * DM_PANEL);   // [ROWS][q_stride]
     constexpr int PS = DM_KEYS + 8;
-    bf* ps = qs + ROWS * k_stride;                              // [ROWS][64 + 8]
+    bf* ps = qs + ROWS * q_stride;                              // [ROWS][64 + 8]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int split = blockIdx.x, g = blockIdx.y / groups, grp = blockIdx.y % groups, b = blockIdx.z;
     const int rep = p.H / p.G, n_rows = p.S * rep, r_first = grp * ROWS;
@@ -97,42 +102,30 @@ attn_decode_kernel(sk_attn_params p, int splits, int groups, int shared_v, int k
     const int t_end = t_beg + rg.per_split < rg.tiles ? t_beg + rg.per_split : rg.tiles;
     if (t_beg >= t_end) return;                                 // the merge knows which splits exist
 
-    const bf* kb = (const bf*)p.k + (int64_t)b * p.k_bs + (int64_t)g * p.k_hs;
-    const bf* vb = (const bf*)p.v + (int64_t)b * p.v_bs + (int64_t)g * p.v_hs;
-    const int kc = p.dqk / 8;                                   // 16-byte pieces of a row
-    const uint32_t k_bytes = p.dqk * 2, v_bytes = p.dv * 2;
-    // warp 0: one bulk copy per key row (and value row); rows past the end repeat the last one and are masked
+    // one thread: the 64-column panels of a tile; rows past the end of the tensor read as zero, rows past the live
+    // end are masked
     auto fetch = [&](int tile, int stage) {
-        if (lane == 0) mbar_expect(&full[stage], DM_KEYS * (k_bytes + (shared_v ? 0u : v_bytes)));
-        __syncwarp();
-#pragma unroll
-        for (int r = lane; r < DM_KEYS; r += 32) {
-            const int64_t row = min(rg.lo + tile * DM_KEYS + r, rg.hi);
-            bulk_load(ks + (stage * DM_KEYS + r) * k_stride, kb + row * p.k_ts, k_bytes, &full[stage]);
-            if (!shared_v) bulk_load(vs + (stage * DM_KEYS + r) * v_stride, vb + row * p.v_ts, v_bytes, &full[stage]);
-        }
+        const int row = rg.lo + tile * DM_KEYS;
+        mbar_expect(&full[stage], (uint32_t)(np + nvp) * DM_PANEL);
+        for (int c = 0; c < np; ++c) tma_load_4d(ks + (stage * np + c) * DM_PANEL, &map_k, c * 64, g, row, b, &full[stage]);
+        for (int c = 0; c < nvp; ++c) tma_load_4d(vs + (stage * nvp + c) * DM_PANEL, &map_v, c * 64, g, row, b, &full[stage]);
     };
     if (tid == 0) {
         mbar_init_count(&full[0], 1);
         mbar_init_count(&full[1], 1);
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
-    }
-    if (warp == 0) {
-        __syncwarp();
         fetch(t_beg, 0);
     }
-    const int k16 = (p.dqk + 15) / 16;
+    const int k16 = (p.dqk + 15) / 16, kc = p.dqk / 8;
     // queries, and the zero columns that round a row up to 16
     for (int r = warp; r < ROWS; r += WARPS) {
         const int row = r_first + r, s = row / rep, hh = row - s * rep;
         const bf* src = (const bf*)p.q + (int64_t)b * p.q_bs + (int64_t)s * p.q_ss + (int64_t)(g * rep + hh) * p.q_hs;
         for (int c = lane; c < k16 * 2; c += 32) {
             const uint4 v = row < n_rows && c < kc ? *reinterpret_cast<const uint4*>(src + c * 8) : make_uint4(0, 0, 0, 0);
-            *reinterpret_cast<uint4*>(qs + r * k_stride + c * 8) = v;
+            *reinterpret_cast<uint4*>(qs + r * q_stride + c * 8) = v;
         }
     }
-    if (k16 * 2 > kc)
-        for (int e = tid; e < 2 * DM_KEYS; e += THREADS) *reinterpret_cast<uint4*>(ks + e * k_stride + kc * 8) = make_uint4(0, 0, 0, 0);
 
     // rows of this thread: scores (one 16-row tile per warp) and accumulators (all tiles)
     const int mtile = MT == 1 ? 0 : (warp & 1), kg = MT == 1 ? warp : (warp >> 1);
@@ -166,23 +159,23 @@ attn_decode_kernel(sk_attn_params p, int splits, int groups, int shared_v, int k
     for (int t = t_beg; t < t_end; ++t) {
         const int it = t - t_beg, stage = it & 1;
         __syncthreads();                                        // the other stage is free
-        if (warp == 0 && t + 1 < t_end) fetch(t + 1, stage ^ 1);
+        if (tid == 0 && t + 1 < t_end) fetch(t + 1, stage ^ 1);
         if (in_time) in_time = mbar_wait_bounded(&full[stage], (uint32_t)((it >> 1) & 1));
-        const bf* kt = ks + stage * DM_KEYS * k_stride;
-        const bf* vt = vs + stage * DM_KEYS * v_stride;
         // ---- scores of 16 rows x 8 keys, two independent sums along the head dimension
         float sc[2][4];
 #pragma unroll
         for (int u = 0; u < 2; ++u)
 #pragma unroll
             for (int e = 0; e < 4; ++e) sc[u][e] = 0.f;
-        const uint32_t qa = saddr(qs + (mtile * 16 + (lane & 15)) * k_stride + (lane >> 4) * 8);
-        const uint32_t ka = saddr(kt + (kg * 8 + (lane & 7)) * k_stride + (lane >> 3) * 8);
+        // a lane reads row (lane & 7) of its 8-key group; 16-byte piece c of a row sits at piece c ^ (row & 7)
+        const uint32_t qa = saddr(qs + (mtile * 16 + (lane & 15)) * q_stride + (lane >> 4) * 8);
+        const uint32_t ka = saddr(ks + stage * np * DM_PANEL + (kg * 8 + (lane & 7)) * 128);
+        const int sw = lane & 7;
         int kk = 0;
 #pragma unroll 4
         for (; kk + 2 <= k16; kk += 2) {                        // 32 head dimensions at a time
             uint32_t a0[4], a1[4], bb[4];
-            ldsm4(ka + kk * 32, bb);
+            ldsm4(ka + (kk >> 2) * DM_PANEL + ((((kk & 2) * 2 + (lane >> 3)) ^ sw) << 4), bb);
             ldsm4(qa + kk * 32, a0);
             ldsm4(qa + kk * 32 + 32, a1);
             mma16816(sc[0], a0, bb[0], bb[1]);
@@ -190,7 +183,7 @@ attn_decode_kernel(sk_attn_params p, int splits, int groups, int shared_v, int k
         }
         if (kk < k16) {
             uint32_t a0[4], b0, b1;
-            ldsm2(saddr(kt + (kg * 8 + (lane & 7)) * k_stride + ((lane >> 3) & 1) * 8) + kk * 32, b0, b1);
+            ldsm2(ka + (kk >> 2) * DM_PANEL + ((((kk & 3) * 2 + ((lane >> 3) & 1)) ^ sw) << 4), b0, b1);
             ldsm4(qa + kk * 32, a0);
             mma16816(sc[0], a0, b0, b1);
         }
@@ -249,6 +242,7 @@ attn_decode_kernel(sk_attn_params p, int splits, int groups, int shared_v, int k
         __syncthreads();
         // ---- P V: every warp all rows, its own value columns
         if (col0 < p.dv) {
+            const uint32_t va = saddr(vs + stage * v_panels * DM_PANEL + (lane & 15) * 128);
 #pragma unroll
             for (int k = 0; k < DM_KEYS / 16; ++k) {
                 uint32_t a[MT][4];
@@ -258,7 +252,8 @@ attn_decode_kernel(sk_attn_params p, int splits, int groups, int shared_v, int k
                 for (int v = 0; v < NVT; v += 2) {
                     if (col0 + v * 8 < p.dv) {
                         uint32_t bb[4];
-                        ldsm4t(saddr(vt + (k * 16 + (lane & 15)) * v_stride + col0 + v * 8 + (lane >> 4) * 8), bb);
+                        const int c = (col0 >> 3) + v + (lane >> 4);
+                        ldsm4t(va + (c >> 3) * DM_PANEL + k * 2048 + (((c & 7) ^ sw) << 4), bb);
 #pragma unroll
                         for (int tt = 0; tt < MT; ++tt) {
                             mma16816(acc[tt][v], a[tt], bb[0], bb[1]);
@@ -381,16 +376,12 @@ attn_decode_merge_kernel(sk_attn_params p, int splits, int groups, int rows_per_
     }
 }
 
-bool rows_16b(const void* base, int64_t a, int64_t b, int64_t c) {
-    return (uintptr_t)base % 16 == 0 && a % 8 == 0 && b % 8 == 0 && c % 8 == 0;
-}
-
 }  // namespace
 
 bool attn_decode_mma_applicable(const sk_attn_params& p) {
     DmPlan d;
-    return dm_plan(p, &d) && rows_16b(p.q, p.q_bs, p.q_ss, p.q_hs) && rows_16b(p.k, p.k_bs, p.k_ts, p.k_hs) &&
-           rows_16b(p.v, p.v_bs, p.v_ts, p.v_hs) && rows_16b(p.out, p.o_bs, p.o_ss, p.o_hs);
+    return dm_plan(p, &d) && head_map_ok(p.q, p.dqk, p.q_hs, p.q_ss, p.q_bs) && head_map_ok(p.k, p.dqk, p.k_hs, p.k_ts, p.k_bs) &&
+           head_map_ok(p.v, p.dv, p.v_hs, p.v_ts, p.v_bs) && head_map_ok(p.out, p.dv, p.o_hs, p.o_ss, p.o_bs);
 }
 
 size_t attn_decode_mma_workspace(const sk_attn_params& p) {
@@ -402,13 +393,16 @@ size_t attn_decode_mma_workspace(const sk_attn_params& p) {
 int launch_attn_decode_mma(const sk_attn_params& p, cudaStream_t st) {
     DmPlan d;
     if (!dm_plan(p, &d)) return fail(SK_ERR_UNSUPPORTED, "skb_attn: shape outside the decode kernel");
+    CUtensorMap mk, mv;
+    if (int rc = make_head_map(&mk, p.k, p.dqk, p.G, p.kv_rows, p.B, p.k_hs, p.k_ts, p.k_bs, DM_KEYS)) return rc;
+    if (int rc = make_head_map(&mv, p.v, p.dv, p.G, p.kv_rows, p.B, p.v_hs, p.v_ts, p.v_bs, DM_KEYS)) return rc;
     dim3 grid((unsigned)d.splits, (unsigned)(p.G * d.groups), (unsigned)p.B);
 #define SK_DM(MT, NVT)                                                                                                   \
     do {                                                                                                                 \
         auto kern = attn_decode_kernel<MT, NVT>;                                                                         \
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)d.smem);      \
         if (e != cudaSuccess) return fail(SK_ERR_CUDA, "attn_decode_kernel smem attribute: %s", cudaGetErrorString(e));  \
-        kern<<<grid, DM_WARPS * 32 * MT, d.smem, st>>>(p, d.splits, d.groups, (int)d.shared_v, d.k_stride, d.v_stride, d.part_floats); \
+        kern<<<grid, DM_WARPS * 32 * MT, d.smem, st>>>(mk, mv, p, d.splits, d.groups, d.np, d.nvp, d.q_stride, d.part_floats); \
     } while (0)
     if (d.mt == 1) {
         if (d.nvt == 2) SK_DM(1, 2);

@@ -13,6 +13,7 @@
 // Every wait is bounded; one that runs out makes all roles leave, and is reported in the status word.
 #include "blocks.cuh"
 #include "tcgen05.cuh"
+#include "tensor_map.cuh"
 
 namespace sk {
 namespace {
@@ -314,44 +315,6 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512u) : "memory");
 }
 
-typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
-                                  const cuuint64_t*, const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave,
-                                  CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-EncodeTiledFn encode_tiled_fn() {
-    static EncodeTiledFn fn = nullptr;
-    if (fn == nullptr) {
-        void* f = nullptr;
-        cudaDriverEntryPointQueryResult q;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &f, cudaEnableDefault, &q) == cudaSuccess &&
-            q == cudaDriverEntryPointSuccess)
-            fn = reinterpret_cast<EncodeTiledFn>(f);
-    }
-    return fn;
-}
-
-// [batch, rows, heads, d] bf16 with a contiguous last dimension -> boxes of 128 rows x 64 columns of one head
-int make_head_map(CUtensorMap* map, const void* base, int d, int heads, int64_t rows, int batch, int64_t hs, int64_t rs,
-                  int64_t bs) {
-    EncodeTiledFn enc = encode_tiled_fn();
-    if (enc == nullptr) return fail(SK_ERR_CUDA, "skb_attn: cuTensorMapEncodeTiled is not available");
-    if (batch == 1) bs = rs;                                  // never stepped over
-    if (heads == 1) hs = rs;
-    const cuuint64_t dims[4] = {(cuuint64_t)d, (cuuint64_t)heads, (cuuint64_t)rows, (cuuint64_t)batch};
-    const cuuint64_t strides[3] = {(cuuint64_t)hs * 2, (cuuint64_t)rs * 2, (cuuint64_t)bs * 2};
-    const cuuint32_t box[4] = {64, 1, FP_TILE, 1};
-    const cuuint32_t estr[4] = {1, 1, 1, 1};
-    const CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base), dims, strides, box, estr,
-                           CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-                           CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-    if (r != CUDA_SUCCESS) return fail(SK_ERR_CUDA, "skb_attn: cuTensorMapEncodeTiled failed (%d)", (int)r);
-    return SK_OK;
-}
-
-bool map_ok(const void* base, int d, int64_t hs, int64_t rs, int64_t bs) {
-    return (uintptr_t)base % 16 == 0 && d % 8 == 0 && hs % 8 == 0 && rs % 8 == 0 && bs % 8 == 0;
-}
-
 // Stages of the two rings and the dynamic shared memory they take; 0 bytes when the shape does not fit
 uint32_t plan_smem(int dqk, int dv, bool bias, int* nk, int* nv) {
     const uint32_t np = (dqk + 63) / 64, nvp = (dv + 63) / 64, extra = bias ? FP_BIAS_BYTES : 0;
@@ -372,9 +335,9 @@ uint32_t plan_smem(int dqk, int dv, bool bias, int* nk, int* nv) {
 bool attn_prefill_tc_applicable(const sk_attn_params& p) {
     int nk, nv;
     return p.dtype == SK_BF16 && p.pos == nullptr && !p.ring && p.dv <= 128 && p.dqk <= 256 && p.scale > 0.f &&
-           p.start >= p.kv_start && p.kv_rows < (int64_t)1 << 30 && map_ok(p.q, p.dqk, p.q_hs, p.q_ss, p.q_bs) &&
-           map_ok(p.k, p.dqk, p.k_hs, p.k_ts, p.k_bs) && map_ok(p.v, p.dv, p.v_hs, p.v_ts, p.v_bs) &&
-           map_ok(p.out, p.dv, p.o_hs, p.o_ss, p.o_bs) && plan_smem(p.dqk, p.dv, p.bias != nullptr, &nk, &nv) > 0;
+           p.start >= p.kv_start && p.kv_rows < (int64_t)1 << 30 && head_map_ok(p.q, p.dqk, p.q_hs, p.q_ss, p.q_bs) &&
+           head_map_ok(p.k, p.dqk, p.k_hs, p.k_ts, p.k_bs) && head_map_ok(p.v, p.dv, p.v_hs, p.v_ts, p.v_bs) &&
+           head_map_ok(p.out, p.dv, p.o_hs, p.o_ss, p.o_bs) && plan_smem(p.dqk, p.dv, p.bias != nullptr, &nk, &nv) > 0;
 }
 
 int launch_attn_prefill_tc(const sk_attn_params& p, cudaStream_t st) {
@@ -398,9 +361,9 @@ int launch_attn_prefill_tc(const sk_attn_params& p, cudaStream_t st) {
     f.scale_log2 = p.scale * FP_LOG2E;
     const uint32_t smem = plan_smem(p.dqk, p.dv, p.bias != nullptr, &f.nk, &f.nv);
     CUtensorMap mq, mk, mv;
-    if (int rc = make_head_map(&mq, p.q, p.dqk, p.H, p.S, p.B, p.q_hs, p.q_ss, p.q_bs)) return rc;
-    if (int rc = make_head_map(&mk, p.k, p.dqk, p.G, p.kv_rows, p.B, p.k_hs, p.k_ts, p.k_bs)) return rc;
-    if (int rc = make_head_map(&mv, p.v, p.dv, p.G, p.kv_rows, p.B, p.v_hs, p.v_ts, p.v_bs)) return rc;
+    if (int rc = make_head_map(&mq, p.q, p.dqk, p.H, p.S, p.B, p.q_hs, p.q_ss, p.q_bs, FP_TILE)) return rc;
+    if (int rc = make_head_map(&mk, p.k, p.dqk, p.G, p.kv_rows, p.B, p.k_hs, p.k_ts, p.k_bs, FP_TILE)) return rc;
+    if (int rc = make_head_map(&mv, p.v, p.dv, p.G, p.kv_rows, p.B, p.v_hs, p.v_ts, p.v_bs, FP_TILE)) return rc;
     auto kern = p.bias != nullptr ? attn_prefill_kernel<true> : attn_prefill_kernel<false>;
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return fail(SK_ERR_CUDA, "attn_prefill_kernel smem attribute: %s", cudaGetErrorString(e));

@@ -6,19 +6,22 @@
 namespace sk {
 namespace {
 
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(256)
 embed_rows_kernel(const int64_t* __restrict__ tokens, const T* __restrict__ table, int64_t vocab, int width, float scale,
                   float* __restrict__ x, float* __restrict__ x_copy, int32_t* status) {
     const int64_t row = blockIdx.x;
+    const int i = (blockIdx.y * 256 + threadIdx.x) * V;
     const int64_t tok = tokens[row];
     const bool ok = tok >= 0 && tok < vocab;              // outside the table: flagged, the row reads zero
-    if (!ok && threadIdx.x == 0 && status != nullptr) atomicOr(status, SK_DEV_INDEX_OUT_OF_RANGE);
-    for (int i = threadIdx.x; i < width; i += blockDim.x) {
-        const float v = ok ? to_f32(table[tok * width + i]) * scale : 0.f;
-        x[row * width + i] = v;
-        if (x_copy != nullptr) x_copy[row * width + i] = v;
-    }
+    if (!ok && i == 0 && status != nullptr) atomicOr(status, SK_DEV_INDEX_OUT_OF_RANGE);
+    if (i >= width) return;
+    float v[V];
+    if (ok) load_vec<T, V>(table + tok * width + i, v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = ok ? v[e] * scale : 0.f;
+    store_vec<float, V>(x + row * width + i, v);
+    if (x_copy != nullptr) store_vec<float, V>(x_copy + row * width + i, v);
 }
 
 // One CTA per row; the row lives in registers (NV vectors of V elements per thread).
@@ -161,12 +164,12 @@ int residual_dispatch(const sk_residual_params& p, cudaStream_t st) {
 
 int launch_embed_rows(const int64_t* tokens, const void* table, int dtype, int64_t rows, int64_t vocab, int width,
                       float scale, float* x, float* x_copy, int32_t* status, cudaStream_t st) {
-    if (dtype == SK_BF16)
-        embed_rows_kernel<<<(unsigned)rows, 256, 0, st>>>(tokens, (const __nv_bfloat16*)table, vocab, width, scale, x,
-                                                          x_copy, status);
-    else
-        embed_rows_kernel<<<(unsigned)rows, 256, 0, st>>>(tokens, (const float*)table, vocab, width, scale, x, x_copy,
-                                                          status);
+    const int V = width % 4 == 0 ? 4 : 1;
+    dim3 grid((unsigned)rows, (unsigned)((width + 256 * V - 1) / (256 * V)));
+#define SK_EMBED(T, V) embed_rows_kernel<T, V><<<grid, 256, 0, st>>>(tokens, (const T*)table, vocab, width, scale, x, x_copy, status)
+    if (dtype == SK_BF16) { if (V == 4) SK_EMBED(__nv_bfloat16, 4); else SK_EMBED(__nv_bfloat16, 1); }
+    else { if (V == 4) SK_EMBED(float, 4); else SK_EMBED(float, 1); }
+#undef SK_EMBED
     return check_launch("embed_rows_kernel");
 }
 

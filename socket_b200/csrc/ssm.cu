@@ -240,7 +240,7 @@ template <typename T> int conv_dispatch(const sk_ssm_params& p, cudaStream_t st)
     auto vec = [&](int v) {
         return channels % v == 0 && p.in_ld % v == 0 && p.xbc_ld % v == 0 && (uintptr_t)p.xbc_in % (v * sizeof(T)) == 0;
     };
-    const int V = sizeof(T) == 2 && vec(8) && p.taps == 4 ? 8 : (vec(4) ? 4 : 1);
+    const int V = p.S == 1 ? 1 : sizeof(T) == 2 && vec(8) && p.taps == 4 ? 8 : (vec(4) ? 4 : 1);
     dim3 grid((unsigned)((channels + 128 * V - 1) / (128 * V)), (unsigned)((p.S + CONV_TOK - 1) / CONV_TOK), (unsigned)p.B);
     if (V == 8) {
         if constexpr (sizeof(T) == 2) ssm_conv_kernel<T, 8, 4><<<grid, 128, 0, st>>>(p);

@@ -132,13 +132,6 @@ __device__ __forceinline__ void tma_load_4d(void* dst, const CUtensorMap* map, i
         : "memory");
 }
 
-// plain bulk copy: both addresses and the size multiples of 16 bytes
-__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
-    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_addr(dst)),
-                 "l"(src), "r"(bytes), "r"(smem_addr(bar))
-                 : "memory");
-}
-
 // Operand whose K index runs over the rows of 128 bytes (64 elements of the other index each), 128-byte
 // swizzle: 8-row groups 1024 bytes apart, the next 64 elements of the other index `panel_bytes` away.
 __device__ __forceinline__ uint64_t umma_desc_sw128_mn(uint32_t saddr, uint32_t panel_bytes) {
