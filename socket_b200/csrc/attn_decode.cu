@@ -1,7 +1,7 @@
 // Softmax attention of one or a few query tokens against a long cache (bf16), split over the keys.
 //
-// All query rows that share a key/value head (rep heads x S tokens) are worked on together, 16 or 32 rows per
-// CTA, so a key is read once for all of them; with one key/value head for every query head - attention on
+// All query rows that share a key/value head (rep heads x S tokens) are worked on together, up to 16 or 32 rows
+// per CTA, so a key is read once for all of them; with one key/value head for every query head - attention on
 // latent rows - this is what makes the step read each cache row once.  A CTA walks its share of 64-key tiles
 // (TMA, 128-byte swizzle, double buffer), computes the scores with m16n8k16 MMAs (rows are too few for the 128-row tensor
 // core tiles), keeps the running maximum per row and accumulates P V with each warp owning a slice of the value columns.
@@ -36,13 +36,14 @@ bool dm_plan(const sk_attn_params& p, DmPlan* d) {
     if (p.dtype != SK_BF16 || p.dqk % 8 || p.dv % 8 || p.dv > 512 || p.dqk > 640 || p.kv_rows >= (int64_t)1 << 30) return false;
     const int rows = p.S * (p.H / p.G);
     d->mt = rows <= 16 ? 1 : 2;
-    d->nvt = p.dv <= 128 * d->mt ? 2 : (p.dv <= 256 * d->mt ? 4 : 8);
+    d->nvt = p.dv <= 128 ? 2 : (p.dv <= 256 ? 4 : 8);
     d->groups = (rows + 16 * d->mt - 1) / (16 * d->mt);
     d->shared_v = p.v == p.k && p.v_ts == p.k_ts && p.v_bs == p.k_bs && (p.G == 1 || p.v_hs == p.k_hs) && p.dv <= p.dqk;
     d->q_stride = (p.dqk + 15) / 16 * 16 + 8;
     d->np = (p.dqk + 63) / 64;
     d->nvp = d->shared_v ? 0 : (p.dv + 63) / 64;
-    d->smem = 1024 + (size_t)2 * (d->np + d->nvp) * DM_PANEL + (size_t)16 * d->mt * d->q_stride * 2 + (size_t)16 * d->mt * (DM_KEYS + 8) * 2;
+    d->smem = 1024 + (size_t)2 * (d->np + d->nvp) * DM_PANEL + (size_t)16 * d->mt * (DM_KEYS + 8) * 2 +
+              (d->mt == 1 ? (size_t)16 * d->q_stride * 2 : (size_t)4 * 32 * (DM_KEYS + 8) * 4);   // queries / partial scores
     if (d->smem > 220 * 1024) return false;
     const int per_sm = d->smem > 110 * 1024 ? 1 : (d->smem > 72 * 1024 || d->mt == 2 ? 2 : 3);
     const int64_t ctas = (int64_t)d->groups * p.G * p.B, tiles = (p.kv_rows + DM_KEYS - 1) / DM_KEYS;
@@ -74,13 +75,13 @@ __device__ __forceinline__ DmRange dm_range(const sk_attn_params& p, int splits)
     return r;
 }
 
-// MT: 16-row tiles per CTA (8 MT warps: one key group of 8 per warp and tile), NVT: 8-column value tiles per warp
-template <int MT, int NVT>
-__global__ void __launch_bounds__(DM_WARPS * 32 * MT)
+// Up to 16 query rows: a warp computes the scores of 8 keys of a tile.  NVT: 8-column value tiles per warp
+template <int NVT>
+__global__ void __launch_bounds__(DM_WARPS * 32)
 attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const __grid_constant__ sk_attn_params p,
                    int splits, int groups, int np, int nvp, int q_stride, size_t part_floats) {
     extern __shared__ char dm_raw[];
-    constexpr int ROWS = 16 * MT, WARPS = DM_WARPS * MT, THREADS = WARPS * 32, KG = 8;
+    constexpr int ROWS = 16, WARPS = DM_WARPS, KG = 8;
     __shared__ __align__(16) float wmax[2][ROWS][KG];
     __shared__ float row_sum[ROWS][KG];
     __shared__ uint64_t full[2];
@@ -127,32 +128,27 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
         }
     }
 
-    // rows of this thread: scores (one 16-row tile per warp) and accumulators (all tiles)
-    const int mtile = MT == 1 ? 0 : (warp & 1), kg = MT == 1 ? warp : (warp >> 1);
+    // rows of this thread
+    const int kg = warp;                                        // key group
     const int fr = lane >> 2, fc = (lane & 3) * 2;              // fragment row and first column
     int64_t qi[2];                                              // query's own key row
     int lo[2];
     const float* brow[2];
 #pragma unroll
     for (int k = 0; k < 2; ++k) {
-        const int row = r_first + mtile * 16 + fr + 8 * k, s = row / rep;
+        const int row = r_first + fr + 8 * k, s = row / rep;
         const int64_t i = rg.i_first + s;
         qi[k] = row < n_rows ? i - rg.base : -1;                // absent row: sees nothing
         lo[k] = p.chunk > 0 ? (int)max((int64_t)0, i / p.chunk * p.chunk - rg.base) : 0;
         brow[k] = p.bias != nullptr && row < n_rows ? p.bias + (int64_t)(g * rep + row - s * rep) * p.bias_len : nullptr;
     }
     const float sl = p.scale * DM_LOG2E;
-    float m_own[2] = {-INFINITY, -INFINITY};                    // of the two score rows
-    float m_acc[MT][2], l_own[2] = {0.f, 0.f};
-    float acc[MT][NVT][4];
+    float m_own[2] = {-INFINITY, -INFINITY}, l_own[2] = {0.f, 0.f};
+    float acc[NVT][4];
 #pragma unroll
-    for (int t = 0; t < MT; ++t) {
-        m_acc[t][0] = m_acc[t][1] = -INFINITY;
+    for (int v = 0; v < NVT; ++v)
 #pragma unroll
-        for (int v = 0; v < NVT; ++v)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) acc[t][v][e] = 0.f;
-    }
+        for (int e = 0; e < 4; ++e) acc[v][e] = 0.f;
     const int col0 = warp * NVT * 8;
     bool in_time = true;
 
@@ -168,7 +164,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
 #pragma unroll
             for (int e = 0; e < 4; ++e) sc[u][e] = 0.f;
         // a lane reads row (lane & 7) of its 8-key group; 16-byte piece c of a row sits at piece c ^ (row & 7)
-        const uint32_t qa = saddr(qs + (mtile * 16 + (lane & 15)) * q_stride + (lane >> 4) * 8);
+        const uint32_t qa = saddr(qs + ((lane & 15)) * q_stride + (lane >> 4) * 8);
         const uint32_t ka = saddr(ks + stage * np * DM_PANEL + (kg * 8 + (lane & 7)) * 128);
         const int sw = lane & 7;
         int kk = 0;
@@ -209,56 +205,49 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
         for (int k = 0; k < 2; ++k) {
             mt[k] = fmaxf(mt[k], __shfl_xor_sync(FULL, mt[k], 1));
             mt[k] = fmaxf(mt[k], __shfl_xor_sync(FULL, mt[k], 2));
-            if ((lane & 3) == 0) wm[mtile * 16 + fr + 8 * k][kg] = mt[k];
+            if ((lane & 3) == 0) wm[fr + 8 * k][kg] = mt[k];
         }
         __syncthreads();
-        // ---- new maxima of all rows; accumulators follow them, score rows become weights
+        // ---- new maxima: accumulators follow them, scores become weights
 #pragma unroll
-        for (int tt = 0; tt < MT; ++tt)
+        for (int k = 0; k < 2; ++k) {
+            const float4* w4 = reinterpret_cast<const float4*>(wm[fr + 8 * k]);
+            const float4 x = w4[0], y = w4[1];
+            const float mn = fmaxf(fmaxf(fmaxf(fmaxf(x.x, x.y), fmaxf(x.z, x.w)), fmaxf(fmaxf(y.x, y.y), fmaxf(y.z, y.w))), m_own[k]);
+            if (mn != m_own[k]) {
+                const float f = exp2_fast(m_own[k] - mn);       // mn is finite here
 #pragma unroll
-            for (int k = 0; k < 2; ++k) {
-                const float4* w4 = reinterpret_cast<const float4*>(wm[tt * 16 + fr + 8 * k]);
-                const float4 x = w4[0], y = w4[1];
-                const float mn = fmaxf(fmaxf(fmaxf(fmaxf(x.x, x.y), fmaxf(x.z, x.w)), fmaxf(fmaxf(y.x, y.y), fmaxf(y.z, y.w))), m_acc[tt][k]);
-                if (mn != m_acc[tt][k]) {
-                    const float f = exp2_fast(m_acc[tt][k] - mn);   // mn is finite here
-#pragma unroll
-                    for (int v = 0; v < NVT; ++v) {
-                        acc[tt][v][2 * k] *= f;
-                        acc[tt][v][2 * k + 1] *= f;
-                    }
-                    if (tt == mtile) l_own[k] *= f;
-                    m_acc[tt][k] = mn;
+                for (int v = 0; v < NVT; ++v) {
+                    acc[v][2 * k] *= f;
+                    acc[v][2 * k + 1] *= f;
                 }
-                if (tt == mtile) m_own[k] = mn;
+                l_own[k] *= f;
+                m_own[k] = mn;
             }
+        }
 #pragma unroll
         for (int k = 0; k < 2; ++k) {
             const float mc = m_own[k] == -INFINITY ? 0.f : m_own[k];
             const float x = exp2_fast(sc[0][2 * k] - mc), y = exp2_fast(sc[0][2 * k + 1] - mc);
             l_own[k] += x + y;
-            *reinterpret_cast<__nv_bfloat162*>(ps + (mtile * 16 + fr + 8 * k) * PS + kg * 8 + fc) = __floats2bfloat162_rn(x, y);
+            *reinterpret_cast<__nv_bfloat162*>(ps + (fr + 8 * k) * PS + kg * 8 + fc) = __floats2bfloat162_rn(x, y);
         }
         __syncthreads();
-        // ---- P V: every warp all rows, its own value columns
+        // ---- P V: every warp its own value columns
         if (col0 < p.dv) {
             const uint32_t va = saddr(vs + stage * v_panels * DM_PANEL + (lane & 15) * 128);
 #pragma unroll
             for (int k = 0; k < DM_KEYS / 16; ++k) {
-                uint32_t a[MT][4];
-#pragma unroll
-                for (int tt = 0; tt < MT; ++tt) ldsm4(saddr(ps + (tt * 16 + (lane & 15)) * PS + k * 16 + (lane >> 4) * 8), a[tt]);
+                uint32_t a[4];
+                ldsm4(saddr(ps + (lane & 15) * PS + k * 16 + (lane >> 4) * 8), a);
 #pragma unroll
                 for (int v = 0; v < NVT; v += 2) {
                     if (col0 + v * 8 < p.dv) {
                         uint32_t bb[4];
                         const int c = (col0 >> 3) + v + (lane >> 4);
                         ldsm4t(va + (c >> 3) * DM_PANEL + k * 2048 + (((c & 7) ^ sw) << 4), bb);
-#pragma unroll
-                        for (int tt = 0; tt < MT; ++tt) {
-                            mma16816(acc[tt][v], a[tt], bb[0], bb[1]);
-                            mma16816(acc[tt][v + 1], a[tt], bb[2], bb[3]);
-                        }
+                        mma16816(acc[v], a, bb[0], bb[1]);
+                        mma16816(acc[v + 1], a, bb[2], bb[3]);
                     }
                 }
             }
@@ -274,7 +263,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
     for (int k = 0; k < 2; ++k) {
         l_own[k] += __shfl_xor_sync(FULL, l_own[k], 1);
         l_own[k] += __shfl_xor_sync(FULL, l_own[k], 2);
-        if ((lane & 3) == 0) row_sum[mtile * 16 + fr + 8 * k][kg] = l_own[k];
+        if ((lane & 3) == 0) row_sum[fr + 8 * k][kg] = l_own[k];
     }
     __syncthreads();
     float* part = (float*)p.workspace + ((((int64_t)b * p.G + g) * groups + grp) * splits + split) * part_floats;
@@ -286,11 +275,251 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
     }
     if (warp == 0 && (lane & 3) == 0)
 #pragma unroll
-        for (int tt = 0; tt < MT; ++tt)
+        for (int k = 0; k < 2; ++k) part[(int64_t)ROWS * p.dv + fr + 8 * k] = m_own[k];
 #pragma unroll
-            for (int k = 0; k < 2; ++k) part[(int64_t)ROWS * p.dv + tt * 16 + fr + 8 * k] = m_acc[tt][k];
+    for (int v = 0; v < NVT; ++v) {
+        const int c = col0 + v * 8 + fc;
+        if (c < p.dv) {
 #pragma unroll
-    for (int tt = 0; tt < MT; ++tt)
+            for (int k = 0; k < 2; ++k)
+                *reinterpret_cast<float2*>(part + (int64_t)(fr + 8 * k) * p.dv + c) = make_float2(acc[v][2 * k], acc[v][2 * k + 1]);
+        }
+    }
+}
+
+// The form for more than 16 query rows (latent attention with many heads): 32 rows per CTA, 8 warps.  Four warps
+// split the head dimension and two the keys of a tile, so that every warp keeps its share of the queries in
+// registers and no key is read from shared memory twice; the partial scores meet in shared memory, where eight
+// lanes own a row: they sum, mask, keep its maximum and sum of weights, and write the weights for P V.
+// KS: 16-column steps of the head dimension per warp, NVT: 8-column value tiles per warp
+template <int KS, int NVT>
+__global__ void __launch_bounds__(DM_WARPS * 32)
+attn_decode_wide_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
+                        const __grid_constant__ sk_attn_params p, int splits, int groups, int np, int nvp, size_t part_floats) {
+    extern __shared__ char dm_raw[];
+    constexpr int ROWS = 32, PS = DM_KEYS + 8, RS = DM_KEYS + 8;
+    __shared__ float f_s[ROWS];
+    __shared__ uint64_t full[2];
+    using bf = __nv_bfloat16;
+    char* ks = reinterpret_cast<char*>((reinterpret_cast<uintptr_t>(dm_raw) + 1023) & ~(uintptr_t)1023);   // [2][panel][64][128 B]
+    char* vs = nvp > 0 ? ks + 2 * np * DM_PANEL : ks;
+    const int v_panels = nvp > 0 ? nvp : np;
+    float* red = reinterpret_cast<float*>(ks + 2 * (np + nvp) * DM_PANEL);   // [4][ROWS][RS]
+    bf* ps = reinterpret_cast<bf*>(red + 4 * ROWS * RS);                     // [ROWS][PS]
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int split = blockIdx.x, g = blockIdx.y / groups, grp = blockIdx.y % groups, b = blockIdx.z;
+    const int rep = p.H / p.G, n_rows = p.S * rep, r_first = grp * ROWS;
+    pdl_launch_dependents();
+    const DmRange rg = dm_range(p, splits);
+    if (split == 0 && grp == 0 && tid == 0 && p.status != nullptr && rg.i_first + p.S - 1 - rg.base >= p.kv_rows)
+        atomicOr(p.status, SK_DEV_POS_OUT_OF_RANGE);
+    const int t_beg = split * rg.per_split;
+    const int t_end = t_beg + rg.per_split < rg.tiles ? t_beg + rg.per_split : rg.tiles;
+    if (t_beg >= t_end) return;
+    auto fetch = [&](int tile, int stage) {                     // one thread, as in the narrow form
+        const int row = rg.lo + tile * DM_KEYS;
+        mbar_expect(&full[stage], (uint32_t)(np + nvp) * DM_PANEL);
+        for (int c = 0; c < np; ++c) tma_load_4d(ks + (stage * np + c) * DM_PANEL, &map_k, c * 64, g, row, b, &full[stage]);
+        for (int c = 0; c < nvp; ++c) tma_load_4d(vs + (stage * nvp + c) * DM_PANEL, &map_v, c * 64, g, row, b, &full[stage]);
+    };
+    if (tid == 0) {
+        mbar_init_count(&full[0], 1);
+        mbar_init_count(&full[1], 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        fetch(t_beg, 0);
+    }
+    // ---- this warp's slice of the queries, as MMA fragments
+    const int fr = lane >> 2, fc = (lane & 3) * 2;
+    const int k16 = (p.dqk + 15) / 16, per = (k16 + 3) / 4, kq = warp & 3, kg = warp >> 2;
+    const int k_lo = kq * per, k_n = k_lo + per < k16 ? per : k16 - k_lo;    // <= KS steps, none for a short head
+    uint32_t qf[2][KS][4];
+#pragma unroll
+    for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int row = r_first + mt * 16 + fr + 8 * e, s = row / rep, hh = row - s * rep;
+            const bf* src = (const bf*)p.q + (int64_t)b * p.q_bs + (int64_t)s * p.q_ss + (int64_t)(g * rep + hh) * p.q_hs;
+#pragma unroll
+            for (int k = 0; k < KS; ++k)
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    const int c = (k_lo + k) * 16 + half * 8 + fc;
+                    qf[mt][k][half * 2 + e] = row < n_rows && k < k_n && c < p.dqk ? *reinterpret_cast<const uint32_t*>(src + c) : 0u;
+                }
+        }
+    // ---- the row this lane helps to own, and the positions it may see
+    const int own = warp * 4 + (lane >> 3), own_row = r_first + own, own_s = own_row / rep;
+    const bool live_row = own_row < n_rows;
+    const int64_t i = rg.i_first + own_s;
+    const int64_t qi = live_row ? i - rg.base : -1;
+    const int lo = p.chunk > 0 ? (int)max((int64_t)0, i / p.chunk * p.chunk - rg.base) : 0;
+    const int hi = (int)min(qi, (int64_t)rg.hi);
+    const float* brow = p.bias != nullptr && live_row ? p.bias + (int64_t)(g * rep + own_row - own_s * rep) * p.bias_len : nullptr;
+    const float sl = p.scale * DM_LOG2E;
+    float m = -INFINITY, l = 0.f;
+    float acc[2][NVT][4];
+#pragma unroll
+    for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int v = 0; v < NVT; ++v)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[t][v][e] = 0.f;
+    const int col0 = warp * NVT * 8, sw = lane & 7;
+    bool in_time = true;
+
+    for (int t = t_beg; t < t_end; ++t) {
+        const int it = t - t_beg, stage = it & 1;
+        __syncthreads();                                        // the other stage is free
+        if (tid == 0 && t + 1 < t_end) fetch(t + 1, stage ^ 1);
+        if (in_time) in_time = mbar_wait_bounded(&full[stage], (uint32_t)((it >> 1) & 1));
+        // ---- 32 rows x 32 keys over this warp's slice of the head dimension
+        {
+            float sc[2][4][4];
+#pragma unroll
+            for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+                for (int n = 0; n < 4; ++n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) sc[mt][n][e] = 0.f;
+            const uint32_t ka = saddr(ks + stage * np * DM_PANEL + (kg * 32 + (lane & 7) + (lane >> 4) * 8) * 128);
+#pragma unroll
+            for (int k = 0; k < KS; ++k) {
+                if (k < k_n) {
+                    const int kk = k_lo + k;
+                    const uint32_t at = ka + (kk >> 2) * DM_PANEL + ((((kk & 3) * 2 + ((lane >> 3) & 1)) ^ sw) << 4);
+                    uint32_t b0[4], b1[4];
+                    ldsm4(at, b0);
+                    ldsm4(at + 16 * 128, b1);
+#pragma unroll
+                    for (int mt = 0; mt < 2; ++mt) {
+                        mma16816(sc[mt][0], qf[mt][k], b0[0], b0[1]);
+                        mma16816(sc[mt][1], qf[mt][k], b0[2], b0[3]);
+                        mma16816(sc[mt][2], qf[mt][k], b1[0], b1[1]);
+                        mma16816(sc[mt][3], qf[mt][k], b1[2], b1[3]);
+                    }
+                }
+            }
+            float* rd = red + kq * ROWS * RS + kg * 32 + fc;
+#pragma unroll
+            for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+                for (int n = 0; n < 4; ++n)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e)
+                        *reinterpret_cast<float2*>(rd + (mt * 16 + fr + 8 * e) * RS + n * 8) =
+                            make_float2(sc[mt][n][2 * e], sc[mt][n][2 * e + 1]);
+        }
+        __syncthreads();
+        // ---- the owned row: keys 4 (lane % 8) .. + 3 and 32 more
+        {
+            float v[8];
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const float* src = red + own * RS + u * 32 + (lane & 7) * 4;
+                float4 x = *reinterpret_cast<const float4*>(src);
+#pragma unroll
+                for (int q = 1; q < 4; ++q) {
+                    const float4 y = *reinterpret_cast<const float4*>(src + q * ROWS * RS);
+                    x.x += y.x;
+                    x.y += y.y;
+                    x.z += y.z;
+                    x.w += y.w;
+                }
+                v[4 * u] = x.x;
+                v[4 * u + 1] = x.y;
+                v[4 * u + 2] = x.z;
+                v[4 * u + 3] = x.w;
+            }
+            float mn = m;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                const int r = rg.lo + t * DM_KEYS + (e >> 2) * 32 + (lane & 7) * 4 + (e & 3);
+                float x = v[e] * sl;
+                if (r >= lo && r <= hi) {
+                    if (brow != nullptr) {
+                        const int64_t d = qi - r;
+                        x = fmaf(__ldg(brow + (d < p.bias_len ? d : p.bias_len - 1)), DM_LOG2E, x);
+                    }
+                } else {
+                    x = -INFINITY;
+                }
+                v[e] = x;
+                mn = fmaxf(mn, x);
+            }
+#pragma unroll
+            for (int o = 4; o >= 1; o >>= 1) mn = fmaxf(mn, __shfl_xor_sync(FULL, mn, o));
+            const float mc = mn == -INFINITY ? 0.f : mn;
+            const float f = mn == m ? 1.f : exp2_fast(m - mc);
+            m = mn;
+            l *= f;
+            if ((lane & 7) == 0) f_s[own] = f;
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                float w[4];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    w[e] = exp2_fast(v[4 * u + e] - mc);
+                    l += w[e];
+                }
+                store_vec<bf, 4>(ps + own * PS + u * 32 + (lane & 7) * 4, w);
+            }
+        }
+        __syncthreads();
+        // ---- P V: every warp all rows, its own value columns
+        if (col0 < p.dv) {
+            float f[2][2];
+            bool any = false;
+#pragma unroll
+            for (int tt = 0; tt < 2; ++tt)
+#pragma unroll
+                for (int k = 0; k < 2; ++k) {
+                    f[tt][k] = f_s[tt * 16 + fr + 8 * k];
+                    any |= f[tt][k] != 1.f;
+                }
+            if (__any_sync(FULL, any)) {
+#pragma unroll
+                for (int tt = 0; tt < 2; ++tt)
+#pragma unroll
+                    for (int v = 0; v < NVT; ++v)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) acc[tt][v][e] *= f[tt][e >> 1];
+            }
+            const uint32_t va = saddr(vs + stage * v_panels * DM_PANEL + (lane & 15) * 128);
+#pragma unroll
+            for (int k = 0; k < DM_KEYS / 16; ++k) {
+                uint32_t a[2][4];
+#pragma unroll
+                for (int tt = 0; tt < 2; ++tt) ldsm4(saddr(ps + (tt * 16 + (lane & 15)) * PS + k * 16 + (lane >> 4) * 8), a[tt]);
+#pragma unroll
+                for (int v = 0; v < NVT; v += 2) {
+                    if (col0 + v * 8 < p.dv) {
+                        uint32_t bb[4];
+                        const int c = (col0 >> 3) + v + (lane >> 4);
+                        ldsm4t(va + (c >> 3) * DM_PANEL + k * 2048 + (((c & 7) ^ sw) << 4), bb);
+#pragma unroll
+                        for (int tt = 0; tt < 2; ++tt) {
+                            mma16816(acc[tt][v], a[tt], bb[0], bb[1]);
+                            mma16816(acc[tt][v + 1], a[tt], bb[2], bb[3]);
+                        }
+                    }
+                }
+            }
+        }
+    }
+    if (!in_time) {
+        if (p.status != nullptr) atomicOr(p.status, SK_DEV_WAIT_TIMEOUT);
+        mbar_wait_bounded(&full[(t_end - 1 - t_beg) & 1], (uint32_t)(((t_end - 1 - t_beg) >> 1) & 1));
+        if (t_end - t_beg > 1) mbar_wait_bounded(&full[(t_end - t_beg) & 1], (uint32_t)(((t_end - 2 - t_beg) >> 1) & 1));
+    }
+    float* part = (float*)p.workspace + ((((int64_t)b * p.G + g) * groups + grp) * splits + split) * part_floats;
+#pragma unroll
+    for (int o = 4; o >= 1; o >>= 1) l += __shfl_xor_sync(FULL, l, o);
+    if ((lane & 7) == 0) {
+        part[(int64_t)ROWS * p.dv + own] = m;
+        part[(int64_t)ROWS * p.dv + ROWS + own] = l;
+    }
+#pragma unroll
+    for (int tt = 0; tt < 2; ++tt)
 #pragma unroll
         for (int v = 0; v < NVT; ++v) {
             const int c = col0 + v * 8 + fc;
@@ -397,21 +626,29 @@ int launch_attn_decode_mma(const sk_attn_params& p, cudaStream_t st) {
     if (int rc = make_head_map(&mk, p.k, p.dqk, p.G, p.kv_rows, p.B, p.k_hs, p.k_ts, p.k_bs, DM_KEYS)) return rc;
     if (int rc = make_head_map(&mv, p.v, p.dv, p.G, p.kv_rows, p.B, p.v_hs, p.v_ts, p.v_bs, DM_KEYS)) return rc;
     dim3 grid((unsigned)d.splits, (unsigned)(p.G * d.groups), (unsigned)p.B);
-#define SK_DM(MT, NVT)                                                                                                   \
+#define SK_DM(kernel, ...)                                                                                               \
     do {                                                                                                                 \
-        auto kern = attn_decode_kernel<MT, NVT>;                                                                         \
+        auto kern = kernel;                                                                                              \
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)d.smem);      \
-        if (e != cudaSuccess) return fail(SK_ERR_CUDA, "attn_decode_kernel smem attribute: %s", cudaGetErrorString(e));  \
-        kern<<<grid, DM_WARPS * 32 * MT, d.smem, st>>>(mk, mv, p, d.splits, d.groups, d.np, d.nvp, d.q_stride, d.part_floats); \
+        if (e != cudaSuccess) return fail(SK_ERR_CUDA, "attn_decode kernel smem attribute: %s", cudaGetErrorString(e));  \
+        kern<<<grid, DM_WARPS * 32, d.smem, st>>>(mk, mv, p, d.splits, d.groups, d.np, d.nvp, __VA_ARGS__);              \
+    } while (0)
+#define SK_DM_WIDE(KS)                                                                                    \
+    do {                                                                                                  \
+        if (d.nvt == 2) SK_DM((attn_decode_wide_kernel<KS, 2>), d.part_floats);                           \
+        else if (d.nvt == 4) SK_DM((attn_decode_wide_kernel<KS, 4>), d.part_floats);                      \
+        else SK_DM((attn_decode_wide_kernel<KS, 8>), d.part_floats);                                      \
     } while (0)
     if (d.mt == 1) {
-        if (d.nvt == 2) SK_DM(1, 2);
-        else if (d.nvt == 4) SK_DM(1, 4);
-        else SK_DM(1, 8);
+        if (d.nvt == 2) SK_DM((attn_decode_kernel<2>), d.q_stride, d.part_floats);
+        else if (d.nvt == 4) SK_DM((attn_decode_kernel<4>), d.q_stride, d.part_floats);
+        else SK_DM((attn_decode_kernel<8>), d.q_stride, d.part_floats);
+    } else if (p.dqk <= 256) {
+        SK_DM_WIDE(4);
     } else {
-        if (d.nvt == 2) SK_DM(2, 2);
-        else SK_DM(2, 4);
+        SK_DM_WIDE(10);
     }
+#undef SK_DM_WIDE
 #undef SK_DM
     if (int rc = check_launch("attn_decode_kernel")) return rc;
     const int col_blocks = (p.dv + DG_COLS - 1) / DG_COLS;
