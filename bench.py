@@ -1,6 +1,6 @@
 """Benchmark of the sparse-attention decode path (one layer, one decode step per "step").
 
-    python bench.py [--gpus N] [--steps K] [--warmup W] [--workload c3|c2] [--impl reference]
+    python bench.py [--gpus N] [--steps K] [--warmup W] [--workload c3|c2|c4|radapel] [--impl reference]
 
 Default workload: the 128K long-context configuration (`c3`: batch 4, 32 query / 8 KV heads,
 context 131072, top-k 2048 + 64 + 256).  With N > 1 GPUs its 8 KV heads are split over the ranks
@@ -65,7 +65,8 @@ def parse_args():
     ap.add_argument("--warmup", type=int, default=20)
     ap.add_argument("--workload", default="c3", choices=sorted(PRESETS) + ["c4", "c4-128k", "c4-128k-b4", "c5", "radapel"],
                     help="c1-c3: one attention layer (op level); c4 / c5: whole-model greedy decode, "
-                         "Llama-3-8B / Llama-3-70B shape with random weights")
+                         "Llama-3-8B / Llama-3-70B shape with random weights; radapel: the Radapel decoder "
+                         "beside the Transformer, and its kernels one by one")
     ap.add_argument("--model-record", default="auto", choices=["auto", "on", "off"],
                     help="also run the whole-model decode comparison (c4) and attach it to the line; "
                          "auto = on a single GPU only")
