@@ -112,7 +112,16 @@ class AttnParams(C.Structure):
         ("v_bs", _i64), ("v_ts", _i64), ("v_hs", _i64), ("o_bs", _i64), ("o_ss", _i64), ("o_hs", _i64),
         ("start", _i64), ("kv_start", _i64), ("kv_rows", _i64), ("bias_len", _i64),
         ("dtype", _i), ("B", _i), ("S", _i), ("H", _i), ("G", _i), ("dqk", _i), ("dv", _i), ("chunk", _i),
-        ("ring", _i), ("path", _i), ("scale", _f),
+        ("window", _i), ("ring", _i), ("path", _i), ("scale", _f), ("softcap", _f),
+    ]
+
+
+class RotaryRowsParams(C.Structure):
+    """Mirror of `sk_rotary_rows_params`."""
+    _fields_ = [
+        ("q_in", _p), ("k_in", _p), ("ring", _p), ("q_out", _p), ("rows_out", _p), ("angles", _p), ("pos", _p),
+        ("status", _p), ("in_ld", _i64), ("start", _i64), ("n_pos", _i64), ("rows_cap", _i64), ("ring_rows", _i64),
+        ("dtype", _i), ("B", _i), ("S", _i), ("H", _i), ("G", _i), ("dim", _i), ("rot_dims", _i), ("prev", _i),
     ]
 
 
@@ -136,6 +145,17 @@ class SsmParams(C.Structure):
     ]
 
 
+class MlstmParams(C.Structure):
+    """Mirror of `sk_mlstm_params`."""
+    _fields_ = [
+        ("q", _p), ("k", _p), ("v", _p), ("z", _p), ("norm_w", _p), ("gates", _p), ("i_bias", _p), ("f_bias", _p),
+        ("S_state", _p), ("n_state", _p), ("m_state", _p), ("num", _p), ("den", _p), ("m_next", _p), ("out", _p),
+        ("pos", _p), ("workspace", _p), ("workspace_bytes", _sz), ("in_ld", _i64), ("gates_ld", _i64),
+        ("out_ld", _i64), ("start", _i64), ("dtype", _i), ("B", _i), ("S", _i), ("H", _i), ("N", _i), ("P", _i),
+        ("path", _i), ("cap", _f), ("q_scale", _f), ("eps", _f),
+    ]
+
+
 # the building-block library, in the order of include/socket_b200_blocks.h
 BLOCK_SIGNATURES = {
     "skb_abi_version": (_i, []),
@@ -143,8 +163,9 @@ BLOCK_SIGNATURES = {
     "skb_last_error": (C.c_char_p, []),
     "skb_embed_rows": (_i, [_p, _p, _i, _i64, _i64, _i, _f, _p, _p, _p, _p]),
     "skb_residual_norm": (_i, [C.POINTER(ResidualParams), _p]),
-    "skb_glu_clamped": (_i, [_p, _i, _i64, _i, _i64, _f, _f, _p, _p]),
-    "skb_ring_append": (_i, [_p, _p, _i, _i, _i, _i64, _i64, _i64, _i64, _i, _i, _i, _p, _i64, _p, _p, _p]),
+    "skb_glu": (_i, [_p, _p, _i, _i64, _i, _i64, _i, _f, _f, _p, _i64, _p]),
+    "skb_ring_append": (_i, [_p, _p, _i, _i, _i, _i64, _i64, _i64, _i64, _i, _i, _i, _i, _p, _i64, _p, _p, _p]),
+    "skb_rotary_rows": (_i, [C.POINTER(RotaryRowsParams), _p]),
     "skb_attn_workspace_bytes": (_sz, [C.POINTER(AttnParams)]),
     "skb_attn": (_i, [C.POINTER(AttnParams), _p]),
     "skb_attn_path": (_i, [C.POINTER(AttnParams)]),
@@ -155,6 +176,9 @@ BLOCK_SIGNATURES = {
     "skb_ssm_workspace_bytes": (_sz, [C.POINTER(SsmParams)]),
     "skb_ssm_scan": (_i, [C.POINTER(SsmParams), _p]),
     "skb_ssm_path": (_i, [C.POINTER(SsmParams)]),
+    "skb_mlstm_workspace_bytes": (_sz, [C.POINTER(MlstmParams)]),
+    "skb_mlstm": (_i, [C.POINTER(MlstmParams), _p]),
+    "skb_mlstm_path": (_i, [C.POINTER(MlstmParams)]),
     "skb_gated_group_norm": (_i, [_p, _p, _i64, _p, _i, _i64, _i, _i, _f, _p, _p]),
 }
 

@@ -15,8 +15,10 @@ from .ops import _require_cuda
 
 ATTN_PATHS = {"auto": 0, "rows": 1, "prefill_tc": 2, "decode": 3}
 SSM_PATHS = {"auto": 0, "steps": 1, "chunks": 2}
-IN_NONE, IN_ADD_NORM, IN_REPLACE = 0, 1, 2
-OUT_NONE, OUT_NORM, OUT_CONCAT = 0, 1, 2
+IN_NONE, IN_ADD_NORM, IN_REPLACE, IN_ADD = 0, 1, 2, 3
+OUT_NONE, OUT_NORM, OUT_CONCAT, OUT_LAYER_NORM = 0, 1, 2, 3
+GLU_CLAMPED, GLU_SILU = 0, 1
+RING_KEEP = {"chunk": 0, "window": 1}
 GLU_SLOPE = 1.702
 
 
@@ -36,10 +38,11 @@ def embed_rows(tokens: Tensor, table: Tensor, scale: float, keep_copy: bool = Fa
 
 def residual_norm(x: Tensor, eps: float, *, y: Optional[Tensor] = None, w_in: Optional[Tensor] = None,
                   replace: bool = False, w_out: Optional[Tensor] = None, x0: Optional[Tensor] = None,
-                  dtype: Optional[torch.dtype] = None) -> Optional[Tensor]:
-    """The residual stream x [rows, width] (fp32, updated in place): x += rms_norm(y) * w_in, or x = y + w_in
-    with `replace`; then returns rms_norm(x) * w_out, or [x ; x0], or nothing.  `dtype`: element type of the
-    weights and of the result (taken from the weights when there are any)."""
+                  dtype: Optional[torch.dtype] = None, centred: bool = False) -> Optional[Tensor]:
+    """The residual stream x [rows, width] (fp32, updated in place): x += rms_norm(y) * w_in, x = y + w_in with
+    `replace`, or x += y without w_in; then returns rms_norm(x) * w_out (with `centred`: the layer norm), or
+    [x ; x0], or nothing.  `dtype`: element type of the weights and of the result (taken from the weights when
+    there are any)."""
     _require_cuda(x, y, w_in, w_out, x0)
     rows, width = x.shape
     assert x.dtype == torch.float32 and x.is_contiguous()
@@ -49,16 +52,18 @@ def residual_norm(x: Tensor, eps: float, *, y: Optional[Tensor] = None, w_in: Op
             dtype = w.dtype
     p = _lib.ResidualParams()
     p.x, p.rows, p.width, p.eps = ptr(x), rows, width, float(eps)
+    if dtype is None:                              # nothing but x and y: the element type does not matter
+        dtype = torch.float32 if y is None else y.dtype
     p.dtype = p.y_dtype = _lib.DTYPE_CODE[dtype]
     p.y_ld = width
     if y is not None:
         assert y.shape == (rows, width) and y.stride(1) == 1
         p.y, p.y_ld, p.y_dtype, p.w_in = ptr(y), y.stride(0), dtype_code(y), ptr(w_in)
-        p.in_mode = IN_REPLACE if replace else IN_ADD_NORM
+        p.in_mode = IN_REPLACE if replace else (IN_ADD if w_in is None else IN_ADD_NORM)
     out = None
     if w_out is not None:
         out = torch.empty(rows, width, dtype=dtype, device=x.device)
-        p.w_out, p.out_mode = ptr(w_out), OUT_NORM
+        p.w_out, p.out_mode = ptr(w_out), OUT_LAYER_NORM if centred else OUT_NORM
     elif x0 is not None:
         assert x0.shape == x.shape and x0.dtype == torch.float32 and x0.is_contiguous()
         out = torch.empty(rows, 2 * width, dtype=dtype, device=x.device)
@@ -68,36 +73,80 @@ def residual_norm(x: Tensor, eps: float, *, y: Optional[Tensor] = None, w_in: Op
     return out
 
 
-def glu_clamped(gate_up: Tensor, ff: int, limit: float, slope: float = GLU_SLOPE) -> Tensor:
-    """gate_up [rows, >= 2 ff] = [gate | up] -> [rows, ff]."""
-    _require_cuda(gate_up)
-    assert gate_up.stride(1) == 1 and gate_up.shape[1] >= 2 * ff
-    out = torch.empty(gate_up.shape[0], ff, dtype=gate_up.dtype, device=gate_up.device)
-    check_blocks(blocks().skb_glu_clamped(ptr(gate_up), dtype_code(gate_up), gate_up.shape[0], ff, gate_up.stride(0),
-                                          float(limit), float(slope), ptr(out), stream_ptr(out.device)), "skb_glu_clamped")
+def _glu(gate: Tensor, up: Tensor, kind: int, limit: float, slope: float, out: Optional[Tensor]) -> Tensor:
+    _require_cuda(gate, up, out)
+    rows, ff = gate.shape
+    if out is None:
+        out = torch.empty(rows, ff, dtype=gate.dtype, device=gate.device)
+    assert gate.stride(1) == up.stride(1) == out.stride(1) == 1 and gate.stride(0) == up.stride(0) and up.shape == gate.shape
+    assert out.shape == gate.shape and out.dtype == up.dtype == gate.dtype
+    check_blocks(blocks().skb_glu(ptr(gate), ptr(up), dtype_code(gate), rows, ff, gate.stride(0), kind, float(limit), float(slope),
+                                  ptr(out), out.stride(0), stream_ptr(out.device)), "skb_glu")
     return out
 
 
-def ring_append(k: Tensor, v: Tensor, k_cache: Tensor, v_cache: Tensor, start: int = 0,
-                pos: Optional[Tensor] = None) -> None:
-    """k [B,S,G,D], v [B,S,G,E] (token rows may be strided) -> k_cache [B,ring,G,D], v_cache [B,ring,G,E]."""
+def glu_clamped(gate_up: Tensor, ff: int, limit: float, slope: float = GLU_SLOPE) -> Tensor:
+    """gate_up [rows, >= 2 ff] = [gate | up] -> g * sigmoid(slope * g) * (u + 1) of the clamped halves, [rows, ff]."""
+    assert gate_up.shape[1] >= 2 * ff
+    return _glu(gate_up[:, :ff], gate_up[:, ff:2 * ff], GLU_CLAMPED, limit, slope, None)
+
+
+def glu_silu(gate: Tensor, up: Tensor, out: Optional[Tensor] = None) -> Tensor:
+    """silu(gate) * up of rows [rows, ff] that may be slices of wider ones; `out` too."""
+    return _glu(gate, up, GLU_SILU, 0.0, 1.0, out)
+
+
+def ring_append(k: Tensor, v: Optional[Tensor], k_cache: Tensor, v_cache: Optional[Tensor], start: int = 0,
+                pos: Optional[Tensor] = None, keep: str = "chunk") -> None:
+    """k [B,S,G,D], v [B,S,G,E] (token rows may be strided) -> k_cache [B,ring,G,D], v_cache [B,ring,G,E]; v and
+    v_cache may be None.  `keep`: of a portion longer than the ring, the tokens of its last chunk of `ring`
+    positions, or its last `ring` tokens ("window")."""
     _require_cuda(k, v, k_cache, v_cache, pos)
     B, S, G, D = k.shape
-    E = v.shape[3]
     ring = k_cache.shape[1]
-    assert k.stride(3) == 1 and (G == 1 or k.stride(2) == D) and v.stride(3) == 1 and (G == 1 or v.stride(2) == E)
-    assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.shape[2:] == (G, D)
-    assert v_cache.shape[1:] == (ring, G, E)
-    check_blocks(blocks().skb_ring_append(ptr(k), ptr(v), dtype_code(k), B, S, k.stride(0), k.stride(1), v.stride(0),
-                                          v.stride(1), G * D, G * E, ring, ptr(pos), start, ptr(k_cache), ptr(v_cache),
+    assert k.stride(3) == 1 and (G == 1 or k.stride(2) == D)
+    assert k_cache.is_contiguous() and k_cache.shape[2:] == (G, D) and (v is None) == (v_cache is None)
+    E = vbs = vss = 0
+    if v is not None:
+        E, vbs, vss = v.shape[3], v.stride(0), v.stride(1)
+        assert v.stride(3) == 1 and (G == 1 or v.stride(2) == E) and v_cache.is_contiguous() and v_cache.shape[1:] == (ring, G, E)
+    check_blocks(blocks().skb_ring_append(ptr(k), ptr(v), dtype_code(k), B, S, k.stride(0), k.stride(1), vbs, vss, G * D, G * E,
+                                          ring, RING_KEEP[keep], ptr(pos), start, ptr(k_cache), ptr(v_cache),
                                           stream_ptr(k.device)), "skb_ring_append")
 
 
+def rotary_rows(q: Tensor, k: Tensor, angles: Tensor, rot_dims: int, rows: Tensor, *, B: int, S: int, start: int = 0,
+                pos: Optional[Tensor] = None, ring: Optional[Tensor] = None, prev: int = 0,
+                status: Optional[Tensor] = None) -> Tensor:
+    """q [B*S, H, dim], k [B*S, G, dim]: slices of the same projection rows.  Fills rows [B, cap, G, dim + rot_dims]
+    (value = [..., :dim], key = [..., rot_dims:]) with the last `prev` positions before `start` out of `ring`,
+    then the new tokens; with `pos`, row pos % cap with the one new token.  Returns the queries [B, S, H, dim]
+    in the keys' element order.  angles [positions, rot_dims / 2, 2] fp32."""
+    _require_cuda(q, k, angles, rows, ring)
+    n, H, dim = q.shape
+    G = k.shape[1]
+    assert n == B * S == k.shape[0] and k.shape[2] == dim and q.stride(0) == k.stride(0) or n == 1
+    assert q.stride()[1:] == (dim, 1) and k.stride()[1:] == (dim, 1)
+    assert rows.is_contiguous() and rows.shape[2:] == (G, dim + rot_dims) and rows.shape[0] >= B
+    assert angles.dtype == torch.float32 and angles.is_contiguous() and angles.shape[1:] == (rot_dims // 2, 2)
+    assert ring is None or (ring.is_contiguous() and ring.shape[2:] == rows.shape[2:])
+    out = torch.empty(B, S, H, dim, dtype=q.dtype, device=q.device)
+    p = _lib.RotaryRowsParams()
+    p.q_in, p.k_in, p.ring, p.q_out, p.rows_out = ptr(q), ptr(k), ptr(ring), ptr(out), ptr(rows)
+    p.angles, p.pos, p.status = ptr(angles), ptr(pos), ptr(status)
+    p.in_ld, p.start, p.n_pos, p.rows_cap = q.stride(0), start, angles.shape[0], rows.shape[1]
+    p.ring_rows = 0 if ring is None else ring.shape[1]
+    p.dtype, p.B, p.S, p.H, p.G, p.dim, p.rot_dims, p.prev = dtype_code(q), B, S, H, G, dim, rot_dims, prev
+    check_blocks(blocks().skb_rotary_rows(C.byref(p), stream_ptr(q.device)), "skb_rotary_rows")
+    return out
+
+
 def attn_params(q: Tensor, k: Tensor, v: Tensor, out: Tensor, *, scale: float, start: int = 0,
-                pos: Optional[Tensor] = None, kv_start: int = 0, chunk: int = 0, ring: bool = False,
-                bias: Optional[Tensor] = None, sink: Optional[Tensor] = None, status: Optional[Tensor] = None,
+                pos: Optional[Tensor] = None, kv_start: int = 0, chunk: int = 0, window: int = 0, ring: bool = False,
+                softcap: float = 0.0, bias: Optional[Tensor] = None, sink: Optional[Tensor] = None, status: Optional[Tensor] = None,
                 workspace: Optional[Tensor] = None, path: str = "auto", meta: bool = False) -> _lib.AttnParams:
-    """The parameter block of one call.  With `meta` q and out are shapes only (for a size query)."""
+    """The parameter block of one call.  With `meta` q and out are shapes only (for a size query).  A window of 0
+    or a cap of 0 is none."""
     B, S, H, dqk = q.shape
     G, dv = k.shape[2], v.shape[3]
     assert k.shape[3] == dqk and v.shape[:3] == k.shape[:3] and out.shape == (B, S, H, dv)
@@ -105,14 +154,16 @@ def attn_params(q: Tensor, k: Tensor, v: Tensor, out: Tensor, *, scale: float, s
     for t in (q, k, v, out):
         assert t.stride(3) == 1
     p = _lib.AttnParams()
-    p.q, p.k, p.v, p.out = (0, 0, 0, 0) if meta else (ptr(q), ptr(k), ptr(v), ptr(out))
+    p.k, p.v = ptr(k), ptr(v)
+    p.q, p.out = (0, 0) if meta else (ptr(q), ptr(out))
     p.q_bs, p.q_ss, p.q_hs = q.stride()[:3]
     p.k_bs, p.k_ts, p.k_hs = k.stride()[:3]
     p.v_bs, p.v_ts, p.v_hs = v.stride()[:3]
     p.o_bs, p.o_ss, p.o_hs = out.stride()[:3]
     p.dtype, p.B, p.S, p.H, p.G, p.dqk, p.dv = dtype_code(q), B, S, H, G, dqk, dv
     p.start, p.pos, p.kv_start, p.kv_rows = start, ptr(pos), kv_start, k.shape[1]
-    p.chunk, p.ring, p.scale, p.path = chunk, int(ring), float(scale), ATTN_PATHS[path]
+    p.chunk, p.window, p.ring, p.path = chunk, window, int(ring), ATTN_PATHS[path]
+    p.scale, p.softcap = float(scale), float(softcap)
     if bias is not None:
         assert bias.dtype == torch.float32 and bias.is_contiguous() and bias.shape[0] == H
         p.bias, p.bias_len = ptr(bias), bias.shape[1]
@@ -125,11 +176,19 @@ def attn_params(q: Tensor, k: Tensor, v: Tensor, out: Tensor, *, scale: float, s
     return p
 
 
-def attn(q: Tensor, k: Tensor, v: Tensor, **kw) -> Tensor:
-    """Softmax attention of a portion: q [B,S,H,dqk], k [B,rows,G,dqk], v [B,rows,G,dv] -> [B,S,H,dv].
-    Keyword arguments as in `attn_params`; a workspace that is absent or too small is allocated when the kernel needs one."""
+def attn_workspace(q_shape, k: Tensor, v: Tensor, **kw) -> int:
+    """Scratch bytes of `attn` for queries of shape [B,S,H,dqk]; keyword arguments as there."""
+    q = torch.empty(q_shape, dtype=k.dtype, device="meta")
+    o = torch.empty(*q_shape[:3], v.shape[3], dtype=k.dtype, device="meta")
+    return int(blocks().skb_attn_workspace_bytes(C.byref(attn_params(q, k, v, o, meta=True, **kw))))
+
+
+def attn(q: Tensor, k: Tensor, v: Tensor, out: Optional[Tensor] = None, **kw) -> Tensor:
+    """Softmax attention of a portion: q [B,S,H,dqk], k [B,rows,G,dqk], v [B,rows,G,dv] -> [B,S,H,dv] (`out`: rows may be
+    slices of wider ones).  Keyword arguments as in `attn_params`; a workspace that is absent or too small is allocated when the kernel needs one."""
     _require_cuda(q, k, v)
-    out = torch.empty(*q.shape[:3], v.shape[3], dtype=q.dtype, device=q.device)
+    if out is None:
+        out = torch.empty(*q.shape[:3], v.shape[3], dtype=q.dtype, device=q.device)
     p = attn_params(q, k, v, out, **kw)
     need = int(blocks().skb_attn_workspace_bytes(C.byref(p)))
     if need > p.workspace_bytes:
@@ -211,6 +270,39 @@ def ssm(proj: Tensor, inner: int, conv_w: Tensor, conv_b: Tensor, dt_bias: Tenso
     check_blocks(blocks().skb_ssm_conv(C.byref(p), st), "skb_ssm_conv")
     check_blocks(blocks().skb_ssm_scan(C.byref(p), st), "skb_ssm_scan")
     return y
+
+
+def mlstm(q: Tensor, k: Tensor, v: Tensor, z: Tensor, gates: Tensor, i_bias: Tensor, f_bias: Tensor, norm_w: Tensor,
+          S_state: Tensor, n_state: Tensor, m_state: Tensor, out: Tensor, *, S: int, cap: float, q_scale: float, eps: float,
+          start: int = 0, pos: Optional[Tensor] = None, path: str = "auto") -> Tensor:
+    """Matrix memory of B * S tokens: q, k [rows, H * N], v, z [rows, H * P] are slices of the same projection rows;
+    gates [rows, >= 2 H] = [input | forget] fp32 before their biases.  S_state [B, H, N, P], n_state [B, H, N] and
+    m_state [B, H] (fp32) are advanced by the portion; out [rows, H * P] (may be a slice) is normed per head and gated."""
+    _require_cuda(q, k, v, z, gates, i_bias, f_bias, norm_w, S_state, n_state, m_state, out)
+    B, H, N, P = S_state.shape
+    rows = q.shape[0]
+    assert rows == B * S and q.shape[1] == k.shape[1] == H * N and v.shape[1] == z.shape[1] == out.shape[1] == H * P
+    assert all(t.stride(1) == 1 and t.stride(0) == q.stride(0) and t.dtype == q.dtype for t in (q, k, v, z))
+    assert out.stride(1) == 1 and out.dtype == q.dtype and gates.dtype == torch.float32 and gates.stride(1) == 1
+    assert gates.shape[0] == rows and gates.shape[1] >= 2 * H and norm_w.shape == (H * P,) and norm_w.dtype == q.dtype
+    for t, shape in ((S_state, (B, H, N, P)), (n_state, (B, H, N)), (m_state, (B, H)), (i_bias, (H,)), (f_bias, (H,))):
+        assert t.dtype == torch.float32 and t.is_contiguous() and t.shape == shape
+    dev = q.device
+    num = torch.empty(rows, H * P, dtype=q.dtype, device=dev)
+    den = torch.empty(rows, H, dtype=torch.float32, device=dev)
+    m_next = torch.empty(B, H, dtype=torch.float32, device=dev)
+    p = _lib.MlstmParams()
+    p.q, p.k, p.v, p.z, p.norm_w, p.gates, p.i_bias, p.f_bias = (ptr(t) for t in (q, k, v, z, norm_w, gates, i_bias, f_bias))
+    p.S_state, p.n_state, p.m_state, p.num, p.den, p.m_next, p.out = (ptr(t) for t in (S_state, n_state, m_state, num, den,
+                                                                                       m_next, out))
+    p.pos, p.start, p.in_ld, p.gates_ld, p.out_ld = ptr(pos), start, q.stride(0), gates.stride(0), out.stride(0)
+    p.dtype, p.B, p.S, p.H, p.N, p.P, p.path = dtype_code(q), B, S, H, N, P, SSM_PATHS[path]
+    p.cap, p.q_scale, p.eps = float(cap), float(q_scale), float(eps)
+    need = int(blocks().skb_mlstm_workspace_bytes(C.byref(p)))
+    ws = torch.empty(need, dtype=torch.uint8, device=dev) if need else None
+    p.workspace, p.workspace_bytes = ptr(ws), need
+    check_blocks(blocks().skb_mlstm(C.byref(p), stream_ptr(dev)), "skb_mlstm")
+    return out
 
 
 def gated_group_norm(y: Tensor, z: Tensor, w: Tensor, parts: int, eps: float) -> Tensor:

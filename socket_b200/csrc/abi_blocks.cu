@@ -14,9 +14,11 @@ int check_attn(const sk_attn_params* p) {
     SK_REQUIRE(block_dtype(p->dtype), "skb_attn: bad dtype");
     SK_REQUIRE(p->B > 0 && p->S > 0 && p->H > 0 && p->G > 0 && p->dqk > 0 && p->dv > 0, "skb_attn: sizes must be positive");
     SK_REQUIRE(p->H % p->G == 0, "skb_attn: %d query heads are not a multiple of %d key/value heads", p->H, p->G);
-    SK_REQUIRE(p->kv_rows > 0 && p->start >= 0 && p->kv_start >= 0 && p->chunk >= 0, "skb_attn: bad positions");
+    SK_REQUIRE(p->kv_rows > 0 && p->start >= 0 && p->kv_start >= 0 && p->chunk >= 0 && p->window >= 0, "skb_attn: bad positions");
+    SK_REQUIRE(p->softcap >= 0.f, "skb_attn: a score cap is positive (0: none)");
     SK_REQUIRE(p->bias == nullptr || p->bias_len > 0, "skb_attn: empty bias table");
-    SK_REQUIRE(!p->ring || (p->chunk > 0 && p->S == 1), "skb_attn: a ring serves one token under a chunk mask");
+    SK_REQUIRE(!p->ring || ((p->chunk > 0 || (p->window > 0 && p->kv_rows <= p->window)) && p->S == 1),
+               "skb_attn: a ring serves one token under a chunk mask, or one of a window that is no smaller than the ring");
     SK_REQUIRE(p->pos != nullptr || p->ring || p->start + p->S - 1 - p->kv_start < p->kv_rows,
                "skb_attn: keys of positions up to %lld are needed, %lld rows from %lld exist",
                (long long)(p->start + p->S - 1), (long long)p->kv_rows, (long long)p->kv_start);
@@ -48,6 +50,23 @@ int ssm_path(const sk_ssm_params& p) {
     return p.S >= 16 && ssm_chunks_applicable(p) ? SKB_SSM_CHUNKS : SKB_SSM_STEPS;
 }
 
+int check_mlstm(const sk_mlstm_params* p) {
+    SK_REQUIRE(p != nullptr, "skb_mlstm: null parameter block");
+    SK_REQUIRE(p->q && p->k && p->v && p->z && p->norm_w && p->gates && p->i_bias && p->f_bias && p->S_state && p->n_state &&
+                   p->m_state && p->num && p->den && p->m_next && p->out, "skb_mlstm: null pointer");
+    SK_REQUIRE(block_dtype(p->dtype), "skb_mlstm: bad dtype");
+    SK_REQUIRE(p->B > 0 && p->S > 0 && p->H > 0 && p->N > 0 && p->P > 0 && p->start >= 0 && p->cap > 0.f,
+               "skb_mlstm: sizes and the gates' cap must be positive");
+    SK_REQUIRE(p->gates_ld >= 2 * p->H && p->out_ld >= (int64_t)p->H * p->P && p->in_ld >= (int64_t)p->H * (p->N > p->P ? p->N : p->P),
+               "skb_mlstm: row stride smaller than row");
+    return SK_OK;
+}
+
+int mlstm_path(const sk_mlstm_params& p) {
+    if (p.path != SKB_SSM_AUTO) return p.path;
+    return p.S >= 16 && mlstm_chunks_applicable(p) ? SKB_SSM_CHUNKS : SKB_SSM_STEPS;
+}
+
 }  // namespace
 
 extern "C" {
@@ -66,29 +85,46 @@ int skb_embed_rows(const int64_t* tokens, const void* table, int dtype, int64_t 
 int skb_residual_norm(const sk_residual_params* p, void* stream) {
     SK_REQUIRE(p && p->x && p->rows > 0 && p->width > 0, "skb_residual_norm: null pointer or empty stream");
     SK_REQUIRE(block_dtype(p->dtype) && (p->y_dtype == p->dtype || p->y_dtype == SK_F32), "skb_residual_norm: bad dtype");
-    SK_REQUIRE(p->in_mode >= 0 && p->in_mode <= 2 && p->out_mode >= 0 && p->out_mode <= 2, "skb_residual_norm: bad mode");
-    SK_REQUIRE(p->in_mode == SKB_IN_NONE || (p->y && p->w_in && p->y_ld >= p->width), "skb_residual_norm: input missing");
+    SK_REQUIRE(p->in_mode >= 0 && p->in_mode <= 3 && p->out_mode >= 0 && p->out_mode <= 3, "skb_residual_norm: bad mode");
+    SK_REQUIRE(p->in_mode == SKB_IN_NONE || (p->y && (p->w_in || p->in_mode == SKB_IN_ADD) && p->y_ld >= p->width),
+               "skb_residual_norm: input missing");
     SK_REQUIRE(p->out_mode == SKB_OUT_NONE || p->out, "skb_residual_norm: output missing");
-    SK_REQUIRE(p->out_mode != SKB_OUT_NORM || p->w_out, "skb_residual_norm: norm weight missing");
+    SK_REQUIRE((p->out_mode != SKB_OUT_NORM && p->out_mode != SKB_OUT_LAYER_NORM) || p->w_out,
+               "skb_residual_norm: norm weight missing");
     SK_REQUIRE(p->out_mode != SKB_OUT_CONCAT || p->x0, "skb_residual_norm: second stream missing");
     return launch_residual_norm(*p, (cudaStream_t)stream);
 }
 
-int skb_glu_clamped(const void* gate_up, int dtype, int64_t rows, int ff, int64_t ld, float limit, float slope, void* out,
-                    void* stream) {
-    SK_REQUIRE(gate_up && out && block_dtype(dtype) && rows > 0 && ff > 0 && ld >= 2 * (int64_t)ff,
-               "skb_glu_clamped: null pointer, bad sizes or dtype");
-    return launch_glu_clamped(gate_up, dtype, rows, ff, ld, limit, slope, out, (cudaStream_t)stream);
+int skb_glu(const void* gate, const void* up, int dtype, int64_t rows, int ff, int64_t ld, int kind, float limit, float slope,
+            void* out, int64_t out_ld, void* stream) {
+    SK_REQUIRE(gate && up && out && block_dtype(dtype) && rows > 0 && ff > 0 && ld >= ff && out_ld >= ff,
+               "skb_glu: null pointer, bad sizes or dtype");
+    SK_REQUIRE(kind == SKB_GLU_CLAMPED || kind == SKB_GLU_SILU, "skb_glu: unknown unit %d", kind);
+    return launch_glu(gate, up, dtype, rows, ff, ld, kind, limit, slope, out, out_ld, (cudaStream_t)stream);
 }
 
 int skb_ring_append(const void* k, const void* v, int dtype, int B, int S, int64_t k_bs, int64_t k_ss, int64_t v_bs,
-                    int64_t v_ss, int k_row, int v_row, int ring, const int64_t* pos, int64_t start, void* k_cache,
+                    int64_t v_ss, int k_row, int v_row, int ring, int keep, const int64_t* pos, int64_t start, void* k_cache,
                     void* v_cache, void* stream) {
-    SK_REQUIRE(k && v && k_cache && v_cache && block_dtype(dtype), "skb_ring_append: null pointer or bad dtype");
-    SK_REQUIRE(B > 0 && S > 0 && k_row > 0 && v_row > 0 && ring > 0 && start >= 0, "skb_ring_append: sizes must be positive");
+    SK_REQUIRE(k && k_cache && (v == nullptr) == (v_cache == nullptr) && block_dtype(dtype), "skb_ring_append: null pointer or bad dtype");
+    SK_REQUIRE(B > 0 && S > 0 && k_row > 0 && (v == nullptr || v_row > 0) && ring > 0 && start >= 0,
+               "skb_ring_append: sizes must be positive");
+    SK_REQUIRE(keep == SKB_RING_CHUNK || keep == SKB_RING_WINDOW, "skb_ring_append: unknown rule %d", keep);
     SK_REQUIRE(pos == nullptr || S == 1, "skb_ring_append: a device position serves one token");
-    return launch_ring_append(k, v, dtype, B, S, k_bs, k_ss, v_bs, v_ss, k_row, v_row, ring, pos, start, k_cache, v_cache,
+    return launch_ring_append(k, v, dtype, B, S, k_bs, k_ss, v_bs, v_ss, k_row, v_row, ring, keep, pos, start, k_cache, v_cache,
                               (cudaStream_t)stream);
+}
+
+int skb_rotary_rows(const sk_rotary_rows_params* p, void* stream) {
+    SK_REQUIRE(p && p->q_in && p->k_in && p->q_out && p->rows_out && p->angles, "skb_rotary_rows: null pointer");
+    SK_REQUIRE(block_dtype(p->dtype) && p->B > 0 && p->S > 0 && p->H > 0 && p->G > 0 && p->dim > 0 && p->start >= 0,
+               "skb_rotary_rows: sizes must be positive");
+    SK_REQUIRE(p->rot_dims >= 0 && p->rot_dims % 2 == 0 && p->rot_dims <= p->dim, "skb_rotary_rows: %d rotated of %d dimensions",
+               p->rot_dims, p->dim);
+    SK_REQUIRE(p->prev >= 0 && (p->prev == 0 || (p->ring && p->prev <= p->ring_rows && p->prev <= p->start && p->pos == nullptr)),
+               "skb_rotary_rows: %d earlier rows cannot be had", p->prev);
+    SK_REQUIRE(p->pos ? p->S == 1 && p->rows_cap > 0 : p->rows_cap >= p->prev + p->S, "skb_rotary_rows: rows do not fit");
+    return launch_rotary_rows(*p, (cudaStream_t)stream);
 }
 
 size_t skb_attn_workspace_bytes(const sk_attn_params* p) {
@@ -159,6 +195,27 @@ int skb_ssm_scan(const sk_ssm_params* p, void* stream) {
         return launch_ssm_chunks(*p, (cudaStream_t)stream);
     }
     return launch_ssm_steps(*p, (cudaStream_t)stream);
+}
+
+size_t skb_mlstm_workspace_bytes(const sk_mlstm_params* p) {
+    return p != nullptr && mlstm_path(*p) == SKB_SSM_CHUNKS ? mlstm_chunks_workspace(*p) : 0;
+}
+
+int skb_mlstm_path(const sk_mlstm_params* p) { return p != nullptr ? mlstm_path(*p) : SKB_SSM_STEPS; }
+
+int skb_mlstm(const sk_mlstm_params* p, void* stream) {
+    if (int rc = check_mlstm(p)) return rc;
+    const cudaStream_t st = (cudaStream_t)stream;
+    if (mlstm_path(*p) == SKB_SSM_CHUNKS) {
+        if (!mlstm_chunks_applicable(*p)) return fail(SK_ERR_UNSUPPORTED, "skb_mlstm: shape outside the block kernel");
+        if (p->workspace == nullptr || p->workspace_bytes < mlstm_chunks_workspace(*p))
+            return fail(SK_ERR_WORKSPACE, "skb_mlstm: workspace of %zu bytes needed, %zu given", mlstm_chunks_workspace(*p),
+                        p->workspace_bytes);
+        if (int rc = launch_mlstm_chunks(*p, st)) return rc;
+    } else if (int rc = launch_mlstm_steps(*p, st)) {
+        return rc;
+    }
+    return launch_mlstm_finish(*p, st);
 }
 
 int skb_gated_group_norm(const void* y, const void* z, int64_t z_ld, const void* w, int dtype, int64_t rows, int inner,

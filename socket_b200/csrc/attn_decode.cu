@@ -5,7 +5,8 @@
 // latent rows - this is what makes the step read each cache row once.  A CTA walks its share of 64-key tiles
 // (TMA, 128-byte swizzle, double buffer), computes the scores with m16n8k16 MMAs (rows are too few for the 128-row tensor
 // core tiles), keeps the running maximum per row and accumulates P V with each warp owning a slice of the value columns.
-// When the values are a prefix of the key rows in memory, the key tile serves as the value tile.  A second kernel
+// When keys and values are slices of the same rows in memory (values a prefix of latent rows; rotary keys that share
+// all but their turned elements with the values), one tile of the whole rows serves both.  A second kernel
 // merges the partial results of the splits.  The live length is read on the device; the grid is fixed.
 #include "blocks.cuh"
 #include "tcgen05.cuh"
@@ -26,6 +27,7 @@ struct DmPlan {
     int groups;             // row groups per (batch, key/value head)
     int splits;
     bool shared_v;
+    int k_off;              // first key column of a shared tile, whose column 0 is the first value column
     int q_stride;           // elements per shared-memory row of the queries
     int np, nvp;            // 64-column panels of a key and of a value tile (0: the key tile serves)
     size_t smem;
@@ -38,9 +40,12 @@ bool dm_plan(const sk_attn_params& p, DmPlan* d) {
     d->mt = rows <= 16 ? 1 : 2;
     d->nvt = p.dv <= 128 ? 2 : (p.dv <= 256 ? 4 : 8);
     d->groups = (rows + 16 * d->mt - 1) / (16 * d->mt);
-    d->shared_v = p.v == p.k && p.v_ts == p.k_ts && p.v_bs == p.k_bs && (p.G == 1 || p.v_hs == p.k_hs) && p.dv <= p.dqk;
+    const int64_t delta = ((intptr_t)p.k - (intptr_t)p.v) / 2;
+    d->shared_v = p.v_ts == p.k_ts && p.v_bs == p.k_bs && (p.G == 1 || p.v_hs == p.k_hs) && delta >= 0 && delta % 8 == 0 &&
+                  delta + p.dqk <= 640 && p.dv <= delta + p.dqk && delta + p.dqk <= p.k_ts && (p.G == 1 || delta + p.dqk <= p.k_hs);
+    d->k_off = d->shared_v ? (int)delta : 0;
     d->q_stride = (p.dqk + 15) / 16 * 16 + 8;
-    d->np = (p.dqk + 63) / 64;
+    d->np = (d->k_off + (p.dqk + 15) / 16 * 16 + 63) / 64;
     d->nvp = d->shared_v ? 0 : (p.dv + 63) / 64;
     d->smem = 1024 + (size_t)2 * (d->np + d->nvp) * DM_PANEL + (size_t)16 * d->mt * (DM_KEYS + 8) * 2 +
               (d->mt == 1 ? (size_t)16 * d->q_stride * 2 : (size_t)4 * 32 * (DM_KEYS + 8) * 4);   // queries / partial scores
@@ -60,26 +65,52 @@ struct DmRange {
     int64_t i_first, base;      // position of token 0, position of key row 0
     int lo, hi;                 // rows any query of the call sees: [lo, hi]
     int tiles, per_split;
+    int wrap;                   // rows of a ring that holds the latest positions (0: rows are in order)
+    bool outside;               // a token lies beyond the cache
 };
 __device__ __forceinline__ DmRange dm_range(const sk_attn_params& p, int splits) {
     DmRange r;
     r.i_first = first_position(p.pos, p.start);
     const int64_t chunk_lo = p.chunk > 0 ? r.i_first / p.chunk * p.chunk : 0;
-    r.base = p.ring ? chunk_lo : p.kv_start;
-    r.lo = (int)(chunk_lo > r.base ? chunk_lo - r.base : 0);
+    r.wrap = p.ring && p.chunk == 0 ? (int)p.kv_rows : 0;
+    r.base = r.wrap ? 0 : (p.ring ? chunk_lo : p.kv_start);
+    int64_t lo = chunk_lo;
+    if (p.window > 0 && !r.wrap && r.i_first - p.window + 1 > lo) lo = r.i_first - p.window + 1;
+    r.lo = (int)(lo > r.base ? lo - r.base : 0);
     int64_t hi = r.i_first + p.S - 1 - r.base;
-    if (hi >= p.kv_rows) hi = p.kv_rows - 1;                     // flagged by the first CTA
+    r.outside = hi >= p.kv_rows && !r.wrap;                      // flagged by the first CTA
+    if (hi >= p.kv_rows) hi = p.kv_rows - 1;
     r.hi = (int)hi;
     r.tiles = r.hi >= r.lo ? (r.hi - r.lo) / DM_KEYS + 1 : 0;
     r.per_split = (r.tiles + splits - 1) / splits;
     return r;
 }
 
+// What one query row (token s of the call) sees: key rows [lo, hi], at the distance origin - row (+ wrap if negative)
+struct DmRow {
+    int lo, hi;
+    int64_t origin;
+};
+__device__ __forceinline__ DmRow dm_row(const sk_attn_params& p, const DmRange& rg, int s, bool live) {
+    const int64_t i = rg.i_first + s;
+    DmRow r;
+    r.origin = rg.wrap ? i % rg.wrap : i - rg.base;
+    int64_t lo = p.chunk > 0 ? i / p.chunk * p.chunk - rg.base : 0;
+    if (p.window > 0 && !rg.wrap) lo = max(lo, i - p.window + 1 - rg.base);
+    r.lo = (int)max((int64_t)0, lo);
+    r.hi = !live ? -1 : rg.wrap ? rg.hi : (int)min(r.origin, (int64_t)rg.hi);      // an absent row sees nothing
+    return r;
+}
+// scaled score in log2 units, without bias
+__device__ __forceinline__ float dm_score(const sk_attn_params& p, float dot) {
+    return p.softcap > 0.f ? p.softcap * DM_LOG2E * tanh_exp2(dot * (p.scale / p.softcap)) : dot * (p.scale * DM_LOG2E);
+}
+
 // Up to 16 query rows: a warp computes the scores of 8 keys of a tile.  NVT: 8-column value tiles per warp
 template <int NVT>
 __global__ void __launch_bounds__(DM_WARPS * 32)
 attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const __grid_constant__ sk_attn_params p,
-                   int splits, int groups, int np, int nvp, int q_stride, size_t part_floats) {
+                   int splits, int groups, int np, int nvp, int k_off, int q_stride, size_t part_floats) {
     extern __shared__ char dm_raw[];
     constexpr int ROWS = 16, WARPS = DM_WARPS, KG = 8;
     __shared__ __align__(16) float wmax[2][ROWS][KG];
@@ -97,7 +128,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
     const int rep = p.H / p.G, n_rows = p.S * rep, r_first = grp * ROWS;
     pdl_launch_dependents();
     const DmRange rg = dm_range(p, splits);
-    if (split == 0 && grp == 0 && tid == 0 && p.status != nullptr && rg.i_first + p.S - 1 - rg.base >= p.kv_rows)
+    if (split == 0 && grp == 0 && tid == 0 && p.status != nullptr && rg.outside)
         atomicOr(p.status, SK_DEV_POS_OUT_OF_RANGE);
     const int t_beg = split * rg.per_split;
     const int t_end = t_beg + rg.per_split < rg.tiles ? t_beg + rg.per_split : rg.tiles;
@@ -131,18 +162,14 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
     // rows of this thread
     const int kg = warp;                                        // key group
     const int fr = lane >> 2, fc = (lane & 3) * 2;              // fragment row and first column
-    int64_t qi[2];                                              // query's own key row
-    int lo[2];
+    DmRow see[2];
     const float* brow[2];
 #pragma unroll
     for (int k = 0; k < 2; ++k) {
         const int row = r_first + fr + 8 * k, s = row / rep;
-        const int64_t i = rg.i_first + s;
-        qi[k] = row < n_rows ? i - rg.base : -1;                // absent row: sees nothing
-        lo[k] = p.chunk > 0 ? (int)max((int64_t)0, i / p.chunk * p.chunk - rg.base) : 0;
+        see[k] = dm_row(p, rg, s, row < n_rows);
         brow[k] = p.bias != nullptr && row < n_rows ? p.bias + (int64_t)(g * rep + row - s * rep) * p.bias_len : nullptr;
     }
-    const float sl = p.scale * DM_LOG2E;
     float m_own[2] = {-INFINITY, -INFINITY}, l_own[2] = {0.f, 0.f};
     float acc[NVT][4];
 #pragma unroll
@@ -166,12 +193,13 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
         // a lane reads row (lane & 7) of its 8-key group; 16-byte piece c of a row sits at piece c ^ (row & 7)
         const uint32_t qa = saddr(qs + ((lane & 15)) * q_stride + (lane >> 4) * 8);
         const uint32_t ka = saddr(ks + stage * np * DM_PANEL + (kg * 8 + (lane & 7)) * 128);
-        const int sw = lane & 7;
+        const int sw = lane & 7, kp = k_off / 8;                // the keys begin at 16-byte piece kp of a row
         int kk = 0;
 #pragma unroll 4
         for (; kk + 2 <= k16; kk += 2) {                        // 32 head dimensions at a time
             uint32_t a0[4], a1[4], bb[4];
-            ldsm4(ka + (kk >> 2) * DM_PANEL + ((((kk & 2) * 2 + (lane >> 3)) ^ sw) << 4), bb);
+            const int c = kk * 2 + (lane >> 3) + kp;
+            ldsm4(ka + (c >> 3) * DM_PANEL + (((c & 7) ^ sw) << 4), bb);
             ldsm4(qa + kk * 32, a0);
             ldsm4(qa + kk * 32 + 32, a1);
             mma16816(sc[0], a0, bb[0], bb[1]);
@@ -179,7 +207,8 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
         }
         if (kk < k16) {
             uint32_t a0[4], b0, b1;
-            ldsm2(ka + (kk >> 2) * DM_PANEL + ((((kk & 3) * 2 + ((lane >> 3) & 1)) ^ sw) << 4), b0, b1);
+            const int c = kk * 2 + ((lane >> 3) & 1) + kp;
+            ldsm2(ka + (c >> 3) * DM_PANEL + (((c & 7) ^ sw) << 4), b0, b1);
             ldsm4(qa + kk * 32, a0);
             mma16816(sc[0], a0, b0, b1);
         }
@@ -188,10 +217,11 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const int k = e >> 1, r = r0 + fc + (e & 1);
-            float v = (sc[0][e] + sc[1][e]) * sl;
-            if (r <= qi[k] && r >= lo[k] && r <= rg.hi) {
+            float v = dm_score(p, sc[0][e] + sc[1][e]);
+            if (r >= see[k].lo && r <= see[k].hi) {
                 if (brow[k] != nullptr) {
-                    const int64_t d = qi[k] - r;
+                    int64_t d = see[k].origin - r;
+                    if (d < 0) d += rg.wrap;
                     v = fmaf(__ldg(brow[k] + (d < p.bias_len ? d : p.bias_len - 1)), DM_LOG2E, v);
                 }
             } else {
@@ -295,7 +325,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
 template <int KS, int NVT>
 __global__ void __launch_bounds__(DM_WARPS * 32)
 attn_decode_wide_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
-                        const __grid_constant__ sk_attn_params p, int splits, int groups, int np, int nvp, size_t part_floats) {
+                        const __grid_constant__ sk_attn_params p, int splits, int groups, int np, int nvp, int k_off, size_t part_floats) {
     extern __shared__ char dm_raw[];
     constexpr int ROWS = 32, PS = DM_KEYS + 8, RS = DM_KEYS + 8;
     __shared__ float f_s[ROWS];
@@ -311,7 +341,7 @@ attn_decode_wide_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     const int rep = p.H / p.G, n_rows = p.S * rep, r_first = grp * ROWS;
     pdl_launch_dependents();
     const DmRange rg = dm_range(p, splits);
-    if (split == 0 && grp == 0 && tid == 0 && p.status != nullptr && rg.i_first + p.S - 1 - rg.base >= p.kv_rows)
+    if (split == 0 && grp == 0 && tid == 0 && p.status != nullptr && rg.outside)
         atomicOr(p.status, SK_DEV_POS_OUT_OF_RANGE);
     const int t_beg = split * rg.per_split;
     const int t_end = t_beg + rg.per_split < rg.tiles ? t_beg + rg.per_split : rg.tiles;
@@ -350,12 +380,8 @@ attn_decode_wide_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     // ---- the row this lane helps to own, and the positions it may see
     const int own = warp * 4 + (lane >> 3), own_row = r_first + own, own_s = own_row / rep;
     const bool live_row = own_row < n_rows;
-    const int64_t i = rg.i_first + own_s;
-    const int64_t qi = live_row ? i - rg.base : -1;
-    const int lo = p.chunk > 0 ? (int)max((int64_t)0, i / p.chunk * p.chunk - rg.base) : 0;
-    const int hi = (int)min(qi, (int64_t)rg.hi);
+    const DmRow see = dm_row(p, rg, own_s, live_row);
     const float* brow = p.bias != nullptr && live_row ? p.bias + (int64_t)(g * rep + own_row - own_s * rep) * p.bias_len : nullptr;
-    const float sl = p.scale * DM_LOG2E;
     float m = -INFINITY, l = 0.f;
     float acc[2][NVT][4];
 #pragma unroll
@@ -364,7 +390,7 @@ attn_decode_wide_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         for (int v = 0; v < NVT; ++v)
 #pragma unroll
             for (int e = 0; e < 4; ++e) acc[t][v][e] = 0.f;
-    const int col0 = warp * NVT * 8, sw = lane & 7;
+    const int col0 = warp * NVT * 8, sw = lane & 7, kp = k_off / 8;
     bool in_time = true;
 
     for (int t = t_beg; t < t_end; ++t) {
@@ -386,7 +412,8 @@ attn_decode_wide_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             for (int k = 0; k < KS; ++k) {
                 if (k < k_n) {
                     const int kk = k_lo + k;
-                    const uint32_t at = ka + (kk >> 2) * DM_PANEL + ((((kk & 3) * 2 + ((lane >> 3) & 1)) ^ sw) << 4);
+                    const int c = kk * 2 + ((lane >> 3) & 1) + kp;
+                    const uint32_t at = ka + (c >> 3) * DM_PANEL + (((c & 7) ^ sw) << 4);
                     uint32_t b0[4], b1[4];
                     ldsm4(at, b0);
                     ldsm4(at + 16 * 128, b1);
@@ -434,10 +461,11 @@ attn_decode_wide_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 #pragma unroll
             for (int e = 0; e < 8; ++e) {
                 const int r = rg.lo + t * DM_KEYS + (e >> 2) * 32 + (lane & 7) * 4 + (e & 3);
-                float x = v[e] * sl;
-                if (r >= lo && r <= hi) {
+                float x = dm_score(p, v[e]);
+                if (r >= see.lo && r <= see.hi) {
                     if (brow != nullptr) {
-                        const int64_t d = qi - r;
+                        int64_t d = see.origin - r;
+                        if (d < 0) d += rg.wrap;
                         x = fmaf(__ldg(brow + (d < p.bias_len ? d : p.bias_len - 1)), DM_LOG2E, x);
                     }
                 } else {
@@ -623,7 +651,7 @@ int launch_attn_decode_mma(const sk_attn_params& p, cudaStream_t st) {
     DmPlan d;
     if (!dm_plan(p, &d)) return fail(SK_ERR_UNSUPPORTED, "skb_attn: shape outside the decode kernel");
     CUtensorMap mk, mv;
-    if (int rc = make_head_map(&mk, p.k, p.dqk, p.G, p.kv_rows, p.B, p.k_hs, p.k_ts, p.k_bs, DM_KEYS)) return rc;
+    if (int rc = make_head_map(&mk, d.shared_v ? p.v : p.k, d.k_off + p.dqk, p.G, p.kv_rows, p.B, p.k_hs, p.k_ts, p.k_bs, DM_KEYS)) return rc;
     if (int rc = make_head_map(&mv, p.v, p.dv, p.G, p.kv_rows, p.B, p.v_hs, p.v_ts, p.v_bs, DM_KEYS)) return rc;
     dim3 grid((unsigned)d.splits, (unsigned)(p.G * d.groups), (unsigned)p.B);
 #define SK_DM(kernel, ...)                                                                                               \
@@ -631,7 +659,7 @@ int launch_attn_decode_mma(const sk_attn_params& p, cudaStream_t st) {
         auto kern = kernel;                                                                                              \
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)d.smem);      \
         if (e != cudaSuccess) return fail(SK_ERR_CUDA, "attn_decode kernel smem attribute: %s", cudaGetErrorString(e));  \
-        kern<<<grid, DM_WARPS * 32, d.smem, st>>>(mk, mv, p, d.splits, d.groups, d.np, d.nvp, __VA_ARGS__);              \
+        kern<<<grid, DM_WARPS * 32, d.smem, st>>>(mk, mv, p, d.splits, d.groups, d.np, d.nvp, d.k_off, __VA_ARGS__);     \
     } while (0)
 #define SK_DM_WIDE(KS)                                                                                    \
     do {                                                                                                  \

@@ -8,8 +8,8 @@
 // core works on the other.  The accumulator is rescaled only when a row's maximum has grown by more than
 // 2^8 since the last time (the final division by the sum makes the choice of reference invisible).
 //
-// Visibility is causal, optionally restricted to the query's own chunk of positions; tiles that no row of
-// a query tile can see are not visited.  Out-of-range rows and columns of a tile are zero-filled by TMA.
+// Visibility is causal, optionally restricted to the query's own chunk of positions or to a sliding window; tiles
+// that no row of a query tile can see are not visited.  Out-of-range rows and columns of a tile are zero-filled by TMA.
 // Every wait is bounded; one that runs out makes all roles leave, and is reported in the status word.
 #include "blocks.cuh"
 #include "tcgen05.cuh"
@@ -42,11 +42,19 @@ struct FpShape {            // what the kernel needs beside the tensor maps
     const float *bias, *sink;
     int32_t* status;
     int64_t o_bs, o_ss, o_hs, start, kv_start, bias_len;
-    int S, H, G, dqk, dv, chunk, nk, nv;      // nk, nv: stages of the K and V rings
-    float scale_log2;
+    int S, H, G, dqk, dv, chunk, window, nk, nv;      // nk, nv: stages of the K and V rings
+    float scale_log2, cap_in, cap_out;        // softcap: s <- cap_out tanh(s cap_in), log2 units
 };
 
-template <bool BIAS>
+// first key row (in key-row coordinates, may be negative) that query row i sees
+__device__ __forceinline__ int64_t fp_first_row(const FpShape& p, int64_t i) {
+    int64_t lo = -p.kv_start;
+    if (p.chunk > 0) lo = (i + p.kv_start) / p.chunk * p.chunk - p.kv_start;
+    if (p.window > 0 && i - p.window + 1 > lo) lo = i - p.window + 1;
+    return lo;
+}
+
+template <bool BIAS, bool CAP>
 __global__ void __launch_bounds__(FP_THREADS, 1)
 attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_v, const FpShape p) {
@@ -70,11 +78,8 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     for (int t = 0; t < 2; ++t) {
         const int first = q0 + t * FP_TILE;
         i0[t] = p.start + first - p.kv_start;
-        int64_t lo = 0;
-        if (p.chunk > 0) {
-            lo = (i0[t] + p.kv_start) / p.chunk * p.chunk - p.kv_start;
-            if (lo < 0) lo = 0;
-        }
+        int64_t lo = fp_first_row(p, i0[t]);
+        if (lo < 0) lo = 0;
         if (t == 0) base = lo;
         const int rows = p.S - first < FP_TILE ? p.S - first : FP_TILE;
         beg[t] = (int)((lo - base) / FP_TILE);
@@ -196,12 +201,8 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         const uint32_t lane_base = (uint32_t)(quad * 32) << 16;
         const uint32_t s_addr = tmem + lane_base + t * FP_TILE, o_addr = tmem + lane_base + 2 * FP_TILE + t * FP_TILE;
         const int64_t i = i0[t] + a;                          // query row in key-row coordinates
-        const float cc = BIAS ? 1.f : p.scale_log2;           // log2 units per unit of s below
-        int64_t lo_row = -1, lo_last = -1;
-        if (p.chunk > 0) {
-            lo_row = (i + p.kv_start) / p.chunk * p.chunk - p.kv_start;
-            lo_last = (i0[t] + FP_TILE - 1 + p.kv_start) / p.chunk * p.chunk - p.kv_start;
-        }
+        const float cc = BIAS || CAP ? 1.f : p.scale_log2;    // log2 units per unit of s below
+        const int64_t lo_row = fp_first_row(p, i), lo_last = fp_first_row(p, i0[t] + FP_TILE - 1);
         float* bt = bias_s + (warp - FP_SOFTMAX_WARP0) * FP_BIAS_SPAN;
         const float* bias_h = BIAS ? p.bias + (int64_t)h * p.bias_len : nullptr;
         float m = -INFINITY, l = 0.f;
@@ -226,9 +227,25 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             tc_fence_after();
             float s[FP_TILE];
             tmem_ld128(s_addr, reinterpret_cast<uint32_t(&)[FP_TILE]>(s));
+            if (CAP) {                                        // small scores: a polynomial, off the exponential's unit
+                float top[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                for (int c = 0; c < FP_TILE; ++c) top[c & 3] = fmaxf(top[c & 3], fabsf(s[c]));
+                const float t4 = fmaxf(fmaxf(top[0], top[1]), fmaxf(top[2], top[3]));
+                if (__any_sync(FULL, !(t4 * p.cap_in <= TANH_POLY_RANGE))) {
+#pragma unroll
+                    for (int c = 0; c < FP_TILE; ++c) s[c] = p.cap_out * tanh_exp2(s[c] * p.cap_in);
+                } else {
+#pragma unroll
+                    for (int c = 0; c < FP_TILE; ++c) {
+                        const float x = s[c] * p.cap_in;
+                        s[c] = (s[c] * p.scale_log2) * tanh_over_x(x * x);
+                    }
+                }
+            }
             if (BIAS) {
 #pragma unroll
-                for (int c = 0; c < FP_TILE; ++c) s[c] = fmaf(s[c], p.scale_log2, bt[lane + FP_TILE - 1 - c]);
+                for (int c = 0; c < FP_TILE; ++c) s[c] = fmaf(s[c], CAP ? 1.f : p.scale_log2, bt[lane + FP_TILE - 1 - c]);
             }
             if (r0 + FP_TILE - 1 > i0[t] || r0 < lo_last) {   // some row does not see the whole tile
                 const int hi_c = (int)(i - r0 < FP_TILE ? i - r0 : FP_TILE), lo_c = (int)(lo_row - r0 > 0 ? lo_row - r0 : 0);
@@ -358,13 +375,17 @@ int launch_attn_prefill_tc(const sk_attn_params& p, cudaStream_t st) {
     f.dqk = p.dqk;
     f.dv = p.dv;
     f.chunk = p.chunk;
+    f.window = p.window;
     f.scale_log2 = p.scale * FP_LOG2E;
+    f.cap_in = p.softcap > 0.f ? p.scale / p.softcap : 0.f;
+    f.cap_out = p.softcap * FP_LOG2E;
     const uint32_t smem = plan_smem(p.dqk, p.dv, p.bias != nullptr, &f.nk, &f.nv);
     CUtensorMap mq, mk, mv;
     if (int rc = make_head_map(&mq, p.q, p.dqk, p.H, p.S, p.B, p.q_hs, p.q_ss, p.q_bs, FP_TILE)) return rc;
     if (int rc = make_head_map(&mk, p.k, p.dqk, p.G, p.kv_rows, p.B, p.k_hs, p.k_ts, p.k_bs, FP_TILE)) return rc;
     if (int rc = make_head_map(&mv, p.v, p.dv, p.G, p.kv_rows, p.B, p.v_hs, p.v_ts, p.v_bs, FP_TILE)) return rc;
-    auto kern = p.bias != nullptr ? attn_prefill_kernel<true> : attn_prefill_kernel<false>;
+    auto kern = p.softcap > 0.f ? (p.bias != nullptr ? attn_prefill_kernel<true, true> : attn_prefill_kernel<false, true>)
+                                : (p.bias != nullptr ? attn_prefill_kernel<true, false> : attn_prefill_kernel<false, false>);
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return fail(SK_ERR_CUDA, "attn_prefill_kernel smem attribute: %s", cudaGetErrorString(e));
     dim3 grid((unsigned)((p.S + 2 * FP_TILE - 1) / (2 * FP_TILE)), (unsigned)p.H, (unsigned)p.B);

@@ -18,8 +18,11 @@ attn_rows_kernel(sk_attn_params p) {
     const int g = h / (p.H / p.G);
     const int64_t i = first_position(p.pos, p.start) + s;
     const int64_t chunk_lo = p.chunk > 0 ? i / p.chunk * p.chunk : 0;
-    const int64_t base = p.ring ? chunk_lo : p.kv_start;         // position of key row 0
-    const int64_t row_lo = chunk_lo > base ? chunk_lo - base : 0, row_hi = i - base;   // visible rows [row_lo, row_hi]
+    const bool wrap = p.ring && p.chunk == 0;                    // row r: the latest position that is r modulo kv_rows
+    const int64_t base = wrap ? 0 : (p.ring ? chunk_lo : p.kv_start);    // position of key row 0
+    const int64_t lo = p.window > 0 && !wrap && i - p.window + 1 > chunk_lo ? i - p.window + 1 : chunk_lo;
+    const int64_t row_lo = lo > base ? lo - base : 0;            // visible rows [row_lo, row_hi]
+    const int64_t row_hi = wrap && i >= p.kv_rows ? p.kv_rows - 1 : i - base;
     T* out = (T*)p.out + b * p.o_bs + s * p.o_ss + h * p.o_hs;
     if (row_hi < 0 || row_hi >= p.kv_rows) {                     // outside the cache: flagged, the row reads zero
         if (t == 0 && p.status != nullptr) atomicOr(p.status, SK_DEV_POS_OUT_OF_RANGE);
@@ -49,8 +52,10 @@ attn_rows_kernel(sk_attn_params p) {
             }
             for (; d < p.dqk; ++d) d0 = fmaf(q_s[d], to_f32(k[d]), d0);
             sc = ((d0 + d1) + (d2 + d3)) * p.scale;
+            if (p.softcap > 0.f) sc = soft_cap_f32(sc, p.softcap);
             if (p.bias != nullptr) {
-                const int64_t n = i - (base + r);
+                int64_t n = i - (base + r);
+                if (wrap) n %= p.kv_rows;
                 sc += p.bias[(int64_t)h * p.bias_len + (n < p.bias_len ? n : p.bias_len - 1)];
             }
         }

@@ -78,6 +78,21 @@ template <typename T> __device__ __forceinline__ float sigmoid_scaled(float x, f
     else return 1.f / (1.f + expf(-slope * x));
 }
 template <typename T> __device__ __forceinline__ float silu(float x) { return x * sigmoid_scaled<T>(x, 1.f); }
+// cap * tanh(x / cap) in full fp32 accuracy
+__device__ __forceinline__ float soft_cap_f32(float x, float cap) { return cap * tanhf(x / cap); }
+__device__ __forceinline__ float log_sigmoid_f32(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
+// tanh(x) with an absolute error of about 1e-7, from one hardware exponential and one division
+__device__ __forceinline__ float tanh_exp2(float x) {
+    return 1.f - __fdividef(2.f, 1.f + exp2_fast(x * 2.8853900817779268f));        // 2 log2(e)
+}
+// tanh(x) / x for |x| <= 1/2 as a polynomial in x^2: interpolation at Chebyshev nodes, error 1.3e-8
+constexpr float TANH_POLY_RANGE = 0.5f;
+__device__ __forceinline__ float tanh_over_x(float x2) {
+    float r = fmaf(x2, 0.017141319f, -0.0529892412f);
+    r = fmaf(x2, r, 0.13324829f);
+    r = fmaf(x2, r, -0.333330719f);
+    return fmaf(x2, r, 0.999999987f);
+}
 __device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 // position of the first token of a portion: on the device (decode) or given by the host
@@ -87,11 +102,12 @@ __device__ __forceinline__ int64_t first_position(const int64_t* pos, int64_t st
 int launch_embed_rows(const int64_t* tokens, const void* table, int dtype, int64_t rows, int64_t vocab, int width,
                       float scale, float* x, float* x_copy, int32_t* status, cudaStream_t st);
 int launch_residual_norm(const sk_residual_params& p, cudaStream_t st);
-int launch_glu_clamped(const void* gate_up, int dtype, int64_t rows, int ff, int64_t ld, float limit, float slope,
-                       void* out, cudaStream_t st);
+int launch_glu(const void* gate, const void* up, int dtype, int64_t rows, int ff, int64_t ld, int kind, float limit, float slope,
+               void* out, int64_t out_ld, cudaStream_t st);
 int launch_ring_append(const void* k, const void* v, int dtype, int B, int S, int64_t k_bs, int64_t k_ss, int64_t v_bs,
-                       int64_t v_ss, int k_row, int v_row, int ring, const int64_t* pos, int64_t start, void* k_cache,
+                       int64_t v_ss, int k_row, int v_row, int ring, int keep, const int64_t* pos, int64_t start, void* k_cache,
                        void* v_cache, cudaStream_t st);
+int launch_rotary_rows(const sk_rotary_rows_params& p, cudaStream_t st);
 int launch_attn_rows(const sk_attn_params& p, cudaStream_t st);
 bool attn_prefill_tc_applicable(const sk_attn_params& p);
 int launch_attn_prefill_tc(const sk_attn_params& p, cudaStream_t st);
@@ -110,5 +126,10 @@ size_t ssm_chunks_workspace(const sk_ssm_params& p);
 int launch_ssm_chunks(const sk_ssm_params& p, cudaStream_t st);
 int launch_gated_group_norm(const void* y, const void* z, int64_t z_ld, const void* w, int dtype, int64_t rows,
                             int inner, int parts, float eps, void* out, cudaStream_t st);
+bool mlstm_chunks_applicable(const sk_mlstm_params& p);
+size_t mlstm_chunks_workspace(const sk_mlstm_params& p);
+int launch_mlstm_chunks(const sk_mlstm_params& p, cudaStream_t st);
+int launch_mlstm_steps(const sk_mlstm_params& p, cudaStream_t st);
+int launch_mlstm_finish(const sk_mlstm_params& p, cudaStream_t st);
 
 }  // namespace sk

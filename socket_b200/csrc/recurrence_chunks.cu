@@ -1,11 +1,17 @@
-// Selective state-space recurrence over a prompt portion as matrix products per block of 64 tokens (bf16
-// inputs).  With cum_t the running sum of the log decays inside a block,
-//   y_t = exp(cum_t) C_t^T S_in + sum_{s <= t} (C_t . B_s) exp(cum_t - cum_s) dt_s x_s + D x_t
-//   S_out = exp(cum_end) S_in + sum_s B_s (exp(cum_end - cum_s) dt_s x_s)^T
-// A first kernel computes the step sizes and running decays (base-2 logarithms) of all blocks.  Then a CTA owns
+// Linear recurrences with a scalar decay per head and token, over a prompt portion, as matrix products per block of
+// 64 tokens (bf16 inputs): the state-space mixer and the matrix memory.  In both, with weights W that depend on the
+// head's gates only,
+//   y_t   = W_in(t) q_t^T S_in + sum_{s <= t} (q_t . k_s) W(t, s) v_s        S_out = W_in(end) S_in + sum_s W(end, s) k_s v_s^T
+// State space (k = B, q = C, v = x; cum_t the running sum of the log decays inside a block):
+//   W(t, s) = exp(cum_t - cum_s) dt_s,  W_in(t) = exp(cum_t),  and D x_t is added to y_t.
+// Matrix memory (f, i the log gates, b_t the running sum of f, a_s = i_s - b_s, A_t = max_{s <= t} a_s, M_t = max(m_in, A_t),
+// so that the stabiliser is m_t = b_t + M_t):
+//   W(t, s) = exp(a_s - M_t),  W_in(t) = exp(m_in - M_t);  m_in of the next block is b_end + M_end.
+// Its normaliser is one more value column whose value is 1; that column's results become the denominators.
+// A first kernel computes the per-token quantities (base-2 logarithms) of all blocks.  Then a CTA owns
 // 32 value columns of one head and walks the blocks in order, two CTAs per SM; the state stays in fp32
-// accumulator registers.  B, C and x are bf16 as the convolution leaves them, products accumulate in fp32,
-// and every factor that carries a decay, a step size or the state enters a product as two bf16 numbers
+// accumulator registers.  q, k and v are bf16 as they come, products accumulate in fp32,
+// and every factor that carries a decay, a gate, a step size or the state enters a product as two bf16 numbers
 // (value and remainder, 16 significant bits together), so that nothing of the recurrence is rounded to
 // 8 bits.
 #include "blocks.cuh"
@@ -56,13 +62,70 @@ ssm_decay_kernel(sk_ssm_params p, int blocks, float* __restrict__ dt, float* __r
     }
 }
 
-// NM: 16-row tiles of the state per warp (8 warps x 16 NM >= N)
-template <int NM>
+// a[b][h][t] = i - b_t, top[b][h][t] = running maximum of a, sum[b][h][t] = b_t inside t's block, all in log2 units;
+// tokens past the portion's end add nothing (a = -inf) and leave the sum as it is.  A CTA: 64 tokens of 32 heads.
+__global__ void __launch_bounds__(256)
+mlstm_gates_kernel(sk_mlstm_params p, int blocks, float* __restrict__ a, float* __restrict__ top, float* __restrict__ sum) {
+    __shared__ float in_s[32][SC_TOK + 1], fo_s[32][SC_TOK + 1];
+    const int blk = blockIdx.x, h0 = blockIdx.y * 32, b = blockIdx.z, t = threadIdx.x, lane = t & 31, warp = t >> 5;
+    const int h = h0 + lane;
+    const float ib = h < p.H ? p.i_bias[h] : 0.f, fb = h < p.H ? p.f_bias[h] : 0.f;
+    for (int s = warp; s < SC_TOK; s += 8) {
+        const int tok = blk * SC_TOK + s;
+        float gi = -INFINITY, gf = 0.f;
+        if (h < p.H && tok < p.S) {
+            const float* g = p.gates + ((int64_t)b * p.S + tok) * p.gates_ld;
+            gi = soft_cap_f32(g[h] + ib, p.cap) * SC_LOG2E;
+            gf = log_sigmoid_f32(soft_cap_f32(g[p.H + h] + fb, p.cap)) * SC_LOG2E;
+        }
+        in_s[lane][s] = gi;
+        fo_s[lane][s] = gf;
+    }
+    __syncthreads();
+    for (int k = warp; k < 32 && h0 + k < p.H; k += 8) {
+        const float f1 = fo_s[k][2 * lane + 1];
+        float acc = fo_s[k][2 * lane] + f1;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float x = __shfl_up_sync(FULL, acc, o);
+            if (lane >= o) acc += x;
+        }
+        const float b0 = acc - f1, a0 = in_s[k][2 * lane] - b0, a1 = in_s[k][2 * lane + 1] - acc;
+        float mx = fmaxf(a0, a1);
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float x = __shfl_up_sync(FULL, mx, o);
+            if (lane >= o) mx = fmaxf(mx, x);
+        }
+        const float before = __shfl_up_sync(FULL, mx, 1);
+        const int64_t at = (((int64_t)b * p.H + h0 + k) * blocks + blk) * SC_TOK + 2 * lane;
+        *reinterpret_cast<float2*>(a + at) = make_float2(a0, a1);
+        *reinterpret_cast<float2*>(top + at) = make_float2(lane > 0 ? fmaxf(before, a0) : a0, mx);
+        *reinterpret_cast<float2*>(sum + at) = make_float2(b0, acc);
+    }
+}
+
+struct RecurrenceParams {
+    const __nv_bfloat16 *q, *k, *v;          // token 0: q and k [H / rep, N], v [H, P]
+    __nv_bfloat16* y;                        // [B S, H P]
+    float *state, *n_state, *den, *m_next;   // n_state, den, m_state, m_next: matrix memory only
+    const float *m_state, *skip;
+    const float *e0, *e1, *e2;               // [B, H, blocks, 64]: running decay, step size | a, its running maximum, b
+    const int64_t* pos;
+    int64_t q_ld, k_ld, v_ld, start;
+    int S, H, P, N, rep, ns, blocks;
+    float q_scale;
+};
+
+// NM: 16-row tiles of the state per warp (8 warps x 16 NM >= N).  MEMORY: the matrix memory, else the state space
+template <int NM, bool MEMORY>
 __global__ void __launch_bounds__(SC_THR, NM == 1 ? 2 : 1)
-ssm_chunks_kernel(sk_ssm_params p, int ns, int blocks, const float* __restrict__ dt_g, const float* __restrict__ cum_g) {
+recurrence_chunks_kernel(const __grid_constant__ RecurrenceParams p) {
     extern __shared__ __align__(16) char sc_raw[];
-    __shared__ __align__(16) float cum_sh[2][SC_TOK], dt_sh[2][SC_TOK];
+    constexpr int NE = MEMORY ? 3 : 2;
+    __shared__ __align__(16) float e_sh[NE][2][SC_TOK];
     __shared__ float w_sh[SC_TOK];
+    const int ns = p.ns, blocks = p.blocks;
     using bf = __nv_bfloat16;
     const int n16 = (p.N + 15) / 16 * 16;
     bf* b_s = reinterpret_cast<bf*>(sc_raw);                  // [2][64][ns]
@@ -72,21 +135,26 @@ ssm_chunks_kernel(sk_ssm_params p, int ns, int blocks, const float* __restrict__
     float4* ex_s = reinterpret_cast<float4*>(st_s + 2 * n16 * SC_PS);   // [warp][2][lane]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, fr = lane >> 2, fc = (lane & 3) * 2;
     const int p0 = blockIdx.x * SC_P, h = blockIdx.y, b = blockIdx.z;
-    const int g = h / (p.H / p.G), I = p.H * p.P, pc = p.P - p0 < SC_P ? p.P - p0 : SC_P;
+    const int g = h / p.rep, I = p.H * p.P;
+    const int pc = p.P - p0 < SC_P ? p.P - p0 : SC_P;         // value columns of this CTA; the normaliser, if it has it, is column pc
     const bool fresh = first_position(p.pos, p.start) == 0;
-    const float skip = p.D[h];
-    const bf* rows = (const bf*)p.xbc + (int64_t)b * p.S * p.xbc_ld;
+    const int64_t head = (int64_t)b * p.H + h;
+    const float skip = MEMORY ? 0.f : p.skip[h];
+    float m_in = MEMORY && !fresh ? p.m_state[head] * SC_LOG2E : 0.f;
+    const bf* q_rows = p.q + (int64_t)b * p.S * p.q_ld + (int64_t)g * p.N;
+    const bf* k_rows = p.k + (int64_t)b * p.S * p.k_ld + (int64_t)g * p.N;
+    const bf* v_rows = p.v + (int64_t)b * p.S * p.v_ld + (int64_t)h * p.P + p0;
     const int nc = p.N / 8, xc = pc / 8;
-    const float* dt_h = dt_g + ((int64_t)b * p.H + h) * blocks * SC_TOK;
-    const float* cum_h = cum_g + ((int64_t)b * p.H + h) * blocks * SC_TOK;
+    const int64_t e_at = head * blocks * SC_TOK;
+    const float* e_h[3] = {p.e0 + e_at, p.e1 + e_at, MEMORY ? p.e2 + e_at : nullptr};
 
     auto fetch = [&](int blk, int stage) {
         const int t0 = blk * SC_TOK;
         for (int r = warp; r < SC_TOK; r += SC_THR / 32) {    // a warp per token, lanes along its row
             const bool live = t0 + r < p.S;
-            const bf* row = rows + (int64_t)(live ? t0 + r : p.S - 1) * p.xbc_ld;
-            const bf* bsrc = row + I + g * p.N;
-            const bf* csrc = bsrc + p.G * p.N;
+            const int64_t tok = live ? t0 + r : p.S - 1;
+            const bf* bsrc = k_rows + tok * p.k_ld;
+            const bf* csrc = q_rows + tok * p.q_ld;
             const uint32_t bd = saddr(b_s + (stage * SC_TOK + r) * ns), cd = saddr(c_s + (stage * SC_TOK + r) * ns);
             for (int c = lane; c < 2 * nc; c += 32) {
                 if (c < nc) cp16(bd + c * 16, bsrc + c * 8, live);
@@ -97,10 +165,13 @@ ssm_chunks_kernel(sk_ssm_params p, int ns, int blocks, const float* __restrict__
             const bool live = t0 + r < p.S;
             if ((tid & 3) < xc)
                 cp16(saddr(x_s + (stage * SC_TOK + r) * SC_PS + (tid & 3) * 8),
-                     rows + (int64_t)(live ? t0 + r : p.S - 1) * p.xbc_ld + h * p.P + p0 + (tid & 3) * 8, live);
+                     v_rows + (int64_t)(live ? t0 + r : p.S - 1) * p.v_ld + (tid & 3) * 8, live);
         }
-        if (tid < SC_TOK / 4) cp16(saddr(&dt_sh[stage][tid * 4]), dt_h + t0 + tid * 4, true);
-        else if (tid < SC_TOK / 2) cp16(saddr(&cum_sh[stage][(tid - SC_TOK / 4) * 4]), cum_h + t0 + (tid - SC_TOK / 4) * 4, true);
+#pragma unroll
+        for (int e = 0; e < NE; ++e) {
+            const int piece = tid - e * (SC_TOK / 4);
+            if (piece >= 0 && piece < SC_TOK / 4) cp16(saddr(&e_sh[e][stage][piece * 4]), e_h[e] + t0 + piece * 4, true);
+        }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     fetch(0, 0);
@@ -111,20 +182,24 @@ ssm_chunks_kernel(sk_ssm_params p, int ns, int blocks, const float* __restrict__
     }
     for (int e = tid; e < 2 * SC_TOK * (SC_PS - pc); e += SC_THR) {
         const int w = SC_PS - pc, r = e / w;
-        x_s[r * SC_PS + pc + (e - r * w)] = __float2bfloat16_rn(0.f);
+        x_s[r * SC_PS + pc + (e - r * w)] = __float2bfloat16_rn(MEMORY && e == r * w && pc < SC_P ? 1.f : 0.f);
     }
 
     // state rows of this warp: tiles warp, warp + 8 of 16 rows each
     float st[NM][4][4];
-    float* gst = p.state + ((int64_t)(b * p.H + h) * p.N) * p.P + p0;
+    float* gst = p.state + head * p.N * p.P + p0;
+    auto state_at = [&](int n, int c) -> float* {             // element (n, c) of this CTA's columns, or none
+        if (n < p.N && c < pc) return gst + (int64_t)n * p.P + c;
+        return MEMORY && n < p.N && c == pc && pc < SC_P ? p.n_state + head * p.N + n : nullptr;
+    };
 #pragma unroll
     for (int u = 0; u < NM; ++u)
 #pragma unroll
         for (int v = 0; v < 4; ++v)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                const int n = (warp + 8 * u) * 16 + fr + 8 * (e >> 1), c = v * 8 + fc + (e & 1);
-                st[u][v][e] = (!fresh && n < p.N && c < pc) ? gst[(int64_t)n * p.P + c] : 0.f;
+                const float* at = state_at((warp + 8 * u) * 16 + fr + 8 * (e >> 1), v * 8 + fc + (e & 1));
+                st[u][v][e] = !fresh && at != nullptr ? *at : 0.f;
             }
     auto publish_state = [&]() {                              // the state as two bf16 parts, for C . S
 #pragma unroll
@@ -157,10 +232,13 @@ ssm_chunks_kernel(sk_ssm_params p, int ns, int blocks, const float* __restrict__
         const bf* bt = b_s + stage * SC_TOK * ns;
         const bf* ct = c_s + stage * SC_TOK * ns;
         const bf* xt = x_s + stage * SC_TOK * SC_PS;
-        const float* cum = cum_sh[stage];
-        const float* dt = dt_sh[stage];
-        const float total = cum[SC_TOK - 1];
-        if (tid < SC_TOK) w_sh[tid] = dt[tid] * exp2f(total - cum[tid]);
+        const float* e0 = e_sh[0][stage];
+        const float* e1 = e_sh[1][stage];
+        // exponent of a token's row factor, without the state's; of the last token: the state's own
+        auto row_exp = [&](int t) { return MEMORY ? -fmaxf(m_in, e1[t]) : e0[t]; };
+        auto weight = [&](float row, int s) { return MEMORY ? exp2f(e0[s] + row) : exp2f(row - e0[s]) * e1[s]; };
+        const float total = row_exp(SC_TOK - 1);
+        if (tid < SC_TOK) w_sh[tid] = weight(total, tid);
         // ---- C . B of 16 tokens x 32 keys, C . S of 16 tokens x 16 value columns
         float gacc[4][4], y[2][4];
 #pragma unroll
@@ -194,10 +272,10 @@ ssm_chunks_kernel(sk_ssm_params p, int ns, int blocks, const float* __restrict__
             }
         }
         const int tr[2] = {mt * 16 + fr, mt * 16 + fr + 8};
-        const float ct_r[2] = {cum[tr[0]], cum[tr[1]]};
+        const float row_r[2] = {row_exp(tr[0]), row_exp(tr[1])};
 #pragma unroll
         for (int k = 0; k < 2; ++k) {
-            const float f = exp2f(ct_r[k]);
+            const float f = exp2f(row_r[k] + m_in);
 #pragma unroll
             for (int v = 0; v < 2; ++v) {
                 y[v][2 * k] *= f;
@@ -219,11 +297,10 @@ ssm_chunks_kernel(sk_ssm_params p, int ns, int blocks, const float* __restrict__
 #pragma unroll
                 for (int v = 0; v < 2; ++v) {
                     const int s = s0 + v * 8 + fc;
-                    const float c0 = cum[s], c1 = cum[s + 1], d0 = dt[s], d1 = dt[s + 1];
 #pragma unroll
                     for (int r = 0; r < 2; ++r) {
-                        const float w0 = s <= tr[r] ? gacc[2 * k + v][2 * r] * (exp2f(ct_r[r] - c0) * d0) : 0.f;
-                        const float w1 = s + 1 <= tr[r] ? gacc[2 * k + v][2 * r + 1] * (exp2f(ct_r[r] - c1) * d1) : 0.f;
+                        const float w0 = s <= tr[r] ? gacc[2 * k + v][2 * r] * weight(row_r[r], s) : 0.f;
+                        const float w1 = s + 1 <= tr[r] ? gacc[2 * k + v][2 * r + 1] * weight(row_r[r], s + 1) : 0.f;
                         split_bf16(w0, w1, a[0][2 * v + r], a[1][2 * v + r]);
                     }
                 }
@@ -269,15 +346,20 @@ ssm_chunks_kernel(sk_ssm_params p, int ns, int blocks, const float* __restrict__
                     const int c = half * 16 + v * 8 + fc;
                     if (c < pc) {
                         const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(xt + tr[k] * SC_PS + c);
-                        *reinterpret_cast<__nv_bfloat162*>((bf*)p.y + ((int64_t)b * p.S + t0 + tr[k]) * I + h * p.P + p0 + c) =
-                            __floats2bfloat162_rn(fmaf(skip, __low2float(x), y[v][2 * k]),
-                                                  fmaf(skip, __high2float(x), y[v][2 * k + 1]));
+                        *reinterpret_cast<__nv_bfloat162*>(p.y + ((int64_t)b * p.S + t0 + tr[k]) * I + h * p.P + p0 + c) =
+                            MEMORY ? __floats2bfloat162_rn(y[v][2 * k] * p.q_scale, y[v][2 * k + 1] * p.q_scale)
+                                   : __floats2bfloat162_rn(fmaf(skip, __low2float(x), y[v][2 * k]),
+                                                           fmaf(skip, __high2float(x), y[v][2 * k + 1]));
+                    } else if (MEMORY && c == pc) {           // n . q; m_t = b_t + M_t
+                        const float m = e_sh[NE - 1][stage][tr[k]] - row_r[k];
+                        p.den[((int64_t)b * p.S + t0 + tr[k]) * p.H + h] =
+                            fmaxf(fabsf(y[v][2 * k] * p.q_scale), exp2f(-m)) + 1e-6f;
                     }
                 }
             }
         }
         // ---- state: (weighted B)^T . x on top of the decayed state
-        const float f = exp2f(total);
+        const float f = exp2f(total + m_in);
 #pragma unroll
         for (int u = 0; u < NM; ++u) {
             const int n0 = (warp + 8 * u) * 16;
@@ -310,7 +392,8 @@ ssm_chunks_kernel(sk_ssm_params p, int ns, int blocks, const float* __restrict__
                 }
             }
         }
-        publish_state();                                      // C . S of this block was read before the last barrier
+        publish_state();                                      // q . S of this block was read before the last barrier
+        if (MEMORY) m_in = e_sh[NE - 1][stage][SC_TOK - 1] - total;
     }
 #pragma unroll
     for (int u = 0; u < NM; ++u)
@@ -318,9 +401,10 @@ ssm_chunks_kernel(sk_ssm_params p, int ns, int blocks, const float* __restrict__
         for (int v = 0; v < 4; ++v)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                const int n = (warp + 8 * u) * 16 + fr + 8 * (e >> 1), c = v * 8 + fc + (e & 1);
-                if (n < p.N && c < pc) gst[(int64_t)n * p.P + c] = st[u][v][e];
+                float* at = state_at((warp + 8 * u) * 16 + fr + 8 * (e >> 1), v * 8 + fc + (e & 1));
+                if (at != nullptr) *at = st[u][v][e];
             }
+    if (MEMORY && pc < SC_P && tid == 0) p.m_next[head] = m_in * (1.f / SC_LOG2E);
 }
 
 size_t chunks_smem(int N, int* ns) {
@@ -329,32 +413,98 @@ size_t chunks_smem(int N, int* ns) {
     return ((size_t)4 * SC_TOK * *ns + 2 * SC_TOK * SC_PS + (size_t)2 * n16 * SC_PS) * 2 + (size_t)(SC_THR / 32) * 2 * 32 * 16;
 }
 
-int chunk_blocks(const sk_ssm_params& p) { return (p.S + SC_TOK - 1) / SC_TOK; }
+int chunk_blocks(int S) { return (S + SC_TOK - 1) / SC_TOK; }
+
+template <bool MEMORY> int launch_blocks(RecurrenceParams& r, int B, cudaStream_t st) {
+    const size_t smem = chunks_smem(r.N, &r.ns);
+    auto kern = r.N <= 128 ? recurrence_chunks_kernel<1, MEMORY> : recurrence_chunks_kernel<2, MEMORY>;
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return fail(SK_ERR_CUDA, "recurrence_chunks_kernel smem attribute: %s", cudaGetErrorString(e));
+    const int cols = r.P + (MEMORY ? 1 : 0);
+    kern<<<dim3((unsigned)((cols + SC_P - 1) / SC_P), (unsigned)r.H, (unsigned)B), SC_THR, smem, st>>>(r);
+    return check_launch("recurrence_chunks_kernel");
+}
 
 }  // namespace
 
+// ---------------------------------------------------------------- state space
 bool ssm_chunks_applicable(const sk_ssm_params& p) {
     return p.dtype == SK_BF16 && p.pos == nullptr && p.N % 8 == 0 && p.N <= 256 && p.P % 8 == 0 && p.xbc_ld % 8 == 0 &&
            (uintptr_t)p.xbc % 16 == 0;
 }
 
 size_t ssm_chunks_workspace(const sk_ssm_params& p) {         // step sizes and running decays
-    return (size_t)2 * p.B * p.H * chunk_blocks(p) * SC_TOK * sizeof(float);
+    return (size_t)2 * p.B * p.H * chunk_blocks(p.S) * SC_TOK * sizeof(float);
 }
 
 int launch_ssm_chunks(const sk_ssm_params& p, cudaStream_t st) {
-    int ns;
-    const size_t smem = chunks_smem(p.N, &ns);
-    const int blocks = chunk_blocks(p);
+    const int blocks = chunk_blocks(p.S), I = p.H * p.P;
     float* dt = (float*)p.workspace;
     float* cum = dt + (size_t)p.B * p.H * blocks * SC_TOK;
     ssm_decay_kernel<<<dim3((unsigned)blocks, (unsigned)((p.H + 31) / 32), (unsigned)p.B), 256, 0, st>>>(p, blocks, dt, cum);
     if (int rc = check_launch("ssm_decay_kernel")) return rc;
-    auto kern = p.N <= 128 ? ssm_chunks_kernel<1> : ssm_chunks_kernel<2>;
-    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return fail(SK_ERR_CUDA, "ssm_chunks_kernel smem attribute: %s", cudaGetErrorString(e));
-    kern<<<dim3((unsigned)((p.P + SC_P - 1) / SC_P), (unsigned)p.H, (unsigned)p.B), SC_THR, smem, st>>>(p, ns, blocks, dt, cum);
-    return check_launch("ssm_chunks_kernel");
+    RecurrenceParams r{};
+    const __nv_bfloat16* x = (const __nv_bfloat16*)p.xbc;     // row: [x (H P) | B (G N) | C (G N)]
+    r.v = x;
+    r.k = x + I;
+    r.q = r.k + p.G * p.N;
+    r.q_ld = r.k_ld = r.v_ld = p.xbc_ld;
+    r.y = (__nv_bfloat16*)p.y;
+    r.state = p.state;
+    r.skip = p.D;
+    r.e0 = cum;
+    r.e1 = dt;
+    r.pos = p.pos;
+    r.start = p.start;
+    r.S = p.S;
+    r.H = p.H;
+    r.P = p.P;
+    r.N = p.N;
+    r.rep = p.H / p.G;
+    r.blocks = blocks;
+    return launch_blocks<false>(r, p.B, st);
+}
+
+// ---------------------------------------------------------------- matrix memory
+bool mlstm_chunks_applicable(const sk_mlstm_params& p) {
+    return p.dtype == SK_BF16 && p.pos == nullptr && p.N % 8 == 0 && p.N <= 256 && p.P % 8 == 0 && p.in_ld % 8 == 0 &&
+           ((uintptr_t)p.q | (uintptr_t)p.k | (uintptr_t)p.v) % 16 == 0;
+}
+
+size_t mlstm_chunks_workspace(const sk_mlstm_params& p) {     // a, its running maximum, b
+    return (size_t)3 * p.B * p.H * chunk_blocks(p.S) * SC_TOK * sizeof(float);
+}
+
+int launch_mlstm_chunks(const sk_mlstm_params& p, cudaStream_t st) {
+    const int blocks = chunk_blocks(p.S);
+    const size_t n = (size_t)p.B * p.H * blocks * SC_TOK;
+    float *a = (float*)p.workspace, *top = a + n, *sum = top + n;
+    mlstm_gates_kernel<<<dim3((unsigned)blocks, (unsigned)((p.H + 31) / 32), (unsigned)p.B), 256, 0, st>>>(p, blocks, a, top, sum);
+    if (int rc = check_launch("mlstm_gates_kernel")) return rc;
+    RecurrenceParams r{};
+    r.q = (const __nv_bfloat16*)p.q;
+    r.k = (const __nv_bfloat16*)p.k;
+    r.v = (const __nv_bfloat16*)p.v;
+    r.q_ld = r.k_ld = r.v_ld = p.in_ld;
+    r.y = (__nv_bfloat16*)p.num;
+    r.state = p.S_state;
+    r.n_state = p.n_state;
+    r.den = p.den;
+    r.m_state = p.m_state;
+    r.m_next = p.m_next;
+    r.e0 = a;
+    r.e1 = top;
+    r.e2 = sum;
+    r.pos = p.pos;
+    r.start = p.start;
+    r.S = p.S;
+    r.H = p.H;
+    r.P = p.P;
+    r.N = p.N;
+    r.rep = 1;
+    r.blocks = blocks;
+    r.q_scale = p.q_scale;
+    return launch_blocks<true>(r, p.B, st);
 }
 
 }  // namespace sk

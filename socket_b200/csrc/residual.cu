@@ -1,6 +1,6 @@
 // Everything between two matrix products that touches the fp32 residual stream: the scaled embedding,
 // the residual update with a norm on the sublayer's output fused with the norm of the next sublayer's
-// input, and the clamped gated unit of the feed-forward.
+// input, and the gated units of the feed-forwards.
 #include "blocks.cuh"
 
 namespace sk {
@@ -25,12 +25,12 @@ embed_rows_kernel(const int64_t* __restrict__ tokens, const T* __restrict__ tabl
 }
 
 // One CTA per row; the row lives in registers (NV vectors of V elements per thread).
-//   in_mode  0: x stays; 1: x += rms(y) * w_in; 2: x = y + w_in
-//   out_mode 0: nothing; 1: out = rms(x) * w_out; 2: out = [x ; x0]
+//   in_mode  0: x stays; 1: x += rms(y) * w_in; 2: x = y + w_in; 3: x += y
+//   out_mode 0: nothing; 1: out = rms(x) * w_out; 2: out = [x ; x0]; 3: out = layer norm of x * w_out
 template <typename T, typename TY, int V, int NV>
 __global__ void __launch_bounds__(1024)
 residual_norm_kernel(sk_residual_params p) {
-    __shared__ float red[2][32];
+    __shared__ float red[3][32];
     const int64_t row = blockIdx.x;
     const int W = p.width, nt = blockDim.x, t = threadIdx.x;
     float* xr = p.x + row * W;
@@ -45,7 +45,7 @@ residual_norm_kernel(sk_residual_params p) {
             const int i = (n * nt + t) * V;
             if (i < W) {
                 load_vec<TY, V>(yr + i, yv[n]);
-                if (p.in_mode == 1) load_vec<float, V>(xr + i, xv[n]);
+                if (p.in_mode != 2) load_vec<float, V>(xr + i, xv[n]);
 #pragma unroll
                 for (int e = 0; e < V; ++e) ss = fmaf(yv[n][e], yv[n][e], ss);
             }
@@ -57,10 +57,11 @@ residual_norm_kernel(sk_residual_params p) {
             const int i = (n * nt + t) * V;
             if (i < W) {
                 float w[V];
-                load_vec<T, V>(w_in + i, w);
+                if (p.in_mode != 3) load_vec<T, V>(w_in + i, w);
 #pragma unroll
                 for (int e = 0; e < V; ++e)
-                    xv[n][e] = p.in_mode == 1 ? xv[n][e] + yv[n][e] * inv * w[e] : yv[n][e] + w[e];
+                    xv[n][e] = p.in_mode == 1 ? xv[n][e] + yv[n][e] * inv * w[e]
+                                              : (p.in_mode == 2 ? yv[n][e] + w[e] : xv[n][e] + yv[n][e]);
                 store_vec<float, V>(xr + i, xv[n]);
             }
         }
@@ -71,13 +72,26 @@ residual_norm_kernel(sk_residual_params p) {
             if (i < W) load_vec<float, V>(xr + i, xv[n]);
         }
     }
-    if (p.out_mode == 1) {
+    if (p.out_mode == 1 || p.out_mode == 3) {
+        float mean = 0.f;
+        if (p.out_mode == 3) {                            // centred in registers; the stream itself is written already
+            float sum = 0.f;
+#pragma unroll
+            for (int n = 0; n < NV; ++n)
+                if ((n * nt + t) * V < W)
+#pragma unroll
+                    for (int e = 0; e < V; ++e) sum += xv[n][e];
+            mean = block_sum(sum, red[2]) / (float)W;
+        }
         float ss = 0.f;
 #pragma unroll
         for (int n = 0; n < NV; ++n)
             if ((n * nt + t) * V < W)
 #pragma unroll
-                for (int e = 0; e < V; ++e) ss = fmaf(xv[n][e], xv[n][e], ss);
+                for (int e = 0; e < V; ++e) {
+                    xv[n][e] -= mean;
+                    ss = fmaf(xv[n][e], xv[n][e], ss);
+                }
         const float inv = 1.f / sqrtf(block_sum(ss, red[1]) / (float)W + p.eps);
         T* o = (T*)p.out + row * W;
 #pragma unroll
@@ -106,28 +120,32 @@ residual_norm_kernel(sk_residual_params p) {
     }
 }
 
-// gate_up row = [gate | up]: y = g * sigmoid(slope * g) * (u + 1), g and u clamped
-template <typename T, int V>
+// KIND SKB_GLU_CLAMPED: y = g * sigmoid(slope * g) * (u + 1), g and u clamped; SKB_GLU_SILU: y = g * sigmoid(g) * u
+template <typename T, int V, int KIND>
 __global__ void __launch_bounds__(256)
-glu_clamped_kernel(const T* __restrict__ gu, int64_t rows, int ff, int64_t ld, float limit, float slope, T* __restrict__ out) {
+glu_kernel(const T* __restrict__ gate, const T* __restrict__ up, int64_t rows, int ff, int64_t ld, float limit, float slope,
+           T* __restrict__ out, int64_t out_ld) {
     const int i = (blockIdx.x * 256 + threadIdx.x) * V;
     if (i >= ff) return;
     for (int64_t row = blockIdx.y; row < rows; row += gridDim.y) {
         float g[V], u[V], r[V];
-        load_vec<T, V>(gu + row * ld + i, g);
-        load_vec<T, V>(gu + row * ld + ff + i, u);
+        load_vec<T, V>(gate + row * ld + i, g);
+        load_vec<T, V>(up + row * ld + i, u);
 #pragma unroll
         for (int e = 0; e < V; ++e) {
-            const float a = fminf(g[e], limit), b = fminf(fmaxf(u[e], -limit), limit);
-            r[e] = a * sigmoid_scaled<T>(a, slope) * (b + 1.f);
+            if (KIND == SKB_GLU_CLAMPED) {
+                const float a = fminf(g[e], limit), b = fminf(fmaxf(u[e], -limit), limit);
+                r[e] = a * sigmoid_scaled<T>(a, slope) * (b + 1.f);
+            } else {
+                r[e] = silu<T>(g[e]) * u[e];
+            }
         }
-        store_vec<T, V>(out + row * ff + i, r);
+        store_vec<T, V>(out + row * out_ld + i, r);
     }
 }
 
-// The newest tokens of a portion into a ring of `ring` rows (row of position p: p % ring).  Only the
-// positions of the last block of `ring` positions are written: earlier ones are not visible any more,
-// and no two tokens of a portion meet in one row.
+// The newest tokens of a portion, from token s0 on, into a ring of `ring` rows (row of position p: p % ring).
+// s0 leaves out what no later token sees, so that no two tokens of a portion meet in one row.
 template <typename T>
 __global__ void __launch_bounds__(256)
 ring_append_kernel(const T* __restrict__ k, const T* __restrict__ v, int64_t k_bs, int64_t k_ss, int64_t v_bs,
@@ -136,11 +154,13 @@ ring_append_kernel(const T* __restrict__ k, const T* __restrict__ v, int64_t k_b
     const int s = s0 + blockIdx.x, b = blockIdx.y;
     const int64_t slot = (first_position(pos, start) + s) % ring;
     const T* ks = k + b * k_bs + s * k_ss;
-    const T* vs = v + b * v_bs + s * v_ss;
     T* kd = k_cache + ((int64_t)b * ring + slot) * k_row;
-    T* vd = v_cache + ((int64_t)b * ring + slot) * v_row;
     for (int i = threadIdx.x; i < k_row; i += blockDim.x) kd[i] = ks[i];
-    for (int i = threadIdx.x; i < v_row; i += blockDim.x) vd[i] = vs[i];
+    if (v != nullptr) {
+        const T* vs = v + b * v_bs + s * v_ss;
+        T* vd = v_cache + ((int64_t)b * ring + slot) * v_row;
+        for (int i = threadIdx.x; i < v_row; i += blockDim.x) vd[i] = vs[i];
+    }
 }
 
 template <typename T, typename TY, int V>
@@ -181,22 +201,32 @@ int launch_residual_norm(const sk_residual_params& p, cudaStream_t st) {
     return v4 ? residual_dispatch<bf, bf, 4>(p, st) : residual_dispatch<bf, bf, 1>(p, st);
 }
 
-int launch_glu_clamped(const void* gate_up, int dtype, int64_t rows, int ff, int64_t ld, float limit, float slope,
-                       void* out, cudaStream_t st) {
-    const bool v4 = ff % 4 == 0 && ld % 4 == 0, v8 = dtype == SK_BF16 && ff % 8 == 0 && ld % 8 == 0;
+int launch_glu(const void* gate, const void* up, int dtype, int64_t rows, int ff, int64_t ld, int kind, float limit, float slope,
+               void* out, int64_t out_ld, cudaStream_t st) {
+    const size_t es = dtype == SK_BF16 ? 2 : 4;
+    auto vec = [&](int v) {
+        return ff % v == 0 && ld % v == 0 && out_ld % v == 0 &&
+               ((uintptr_t)gate | (uintptr_t)up | (uintptr_t)out) % (v * es) == 0;
+    };
+    const bool v4 = vec(4), v8 = dtype == SK_BF16 && vec(8);
     const int V = v8 ? 8 : (v4 ? 4 : 1);
     dim3 grid((unsigned)((ff + 256 * V - 1) / (256 * V)), (unsigned)(rows < 32768 ? rows : 32768));
-#define SK_GLU(T, V) glu_clamped_kernel<T, V><<<grid, 256, 0, st>>>((const T*)gate_up, rows, ff, ld, limit, slope, (T*)out)
+#define SK_GLU(T, V)                                                                                                       \
+    do {                                                                                                                   \
+        auto kern = kind == SKB_GLU_CLAMPED ? glu_kernel<T, V, SKB_GLU_CLAMPED> : glu_kernel<T, V, SKB_GLU_SILU>;          \
+        kern<<<grid, 256, 0, st>>>((const T*)gate, (const T*)up, rows, ff, ld, limit, slope, (T*)out, out_ld);             \
+    } while (0)
     if (dtype == SK_BF16) { if (v8) SK_GLU(__nv_bfloat16, 8); else if (v4) SK_GLU(__nv_bfloat16, 4); else SK_GLU(__nv_bfloat16, 1); }
     else { if (v4) SK_GLU(float, 4); else SK_GLU(float, 1); }
 #undef SK_GLU
-    return check_launch("glu_clamped_kernel");
+    return check_launch("glu_kernel");
 }
 
 int launch_ring_append(const void* k, const void* v, int dtype, int B, int S, int64_t k_bs, int64_t k_ss, int64_t v_bs,
-                       int64_t v_ss, int k_row, int v_row, int ring, const int64_t* pos, int64_t start, void* k_cache,
+                       int64_t v_ss, int k_row, int v_row, int ring, int keep, const int64_t* pos, int64_t start, void* k_cache,
                        void* v_cache, cudaStream_t st) {
-    const int64_t first = (start + S - 1) / ring * ring;       // first position of the last block
+    // first position to write: of the last block of `ring` positions, or of the last `ring` positions
+    const int64_t first = keep == SKB_RING_CHUNK ? (start + S - 1) / ring * ring : start + S - ring;
     const int s0 = pos == nullptr && first > start ? (int)(first - start) : 0;   // a device position: one token
     dim3 grid((unsigned)(S - s0), (unsigned)B);
     if (dtype == SK_BF16)

@@ -1,16 +1,21 @@
-"""Token mixers and the feed-forward built on the block library (`block_ops.py`): chunk-masked attention
-with a learned distance bias, attention on a low-rank latent, a selective state-space layer, and a
-clamped gated unit.  Every size and constant is a parameter, so that any decoder can list them.
+"""Token mixers and feed-forwards built on the block library (`block_ops.py`): chunk-masked attention
+with a learned distance bias, attention on a low-rank latent, sliding-window attention whose values are
+its unrotated keys, a selective state-space layer, a matrix memory, and gated units.  Every size and
+constant is a parameter, so that any decoder can list them.
 
 A mixer maps hidden rows [B*S, width] of a portion to rows of the same shape and advances its cache:
 `make_cache(...)` builds it, `forward(h, cache, at)` uses it.  `at` (`Portion`) says where the portion
 sits; a decode step is the portion of one token whose position is read on the device.
+
+The mixers of a `ParallelLayer` leave their large projections to the layer, which runs them together with
+the feed-forward's as one matrix product in and one out: they name them (`in_sizes`, `out_size`) and
+`mix(parts, h, cache, at, out)` takes the projected rows to the rows in front of the output projection.
 """
 from __future__ import annotations
 
 import math
 from dataclasses import dataclass
-from typing import Optional
+from typing import Dict, List, Optional, Tuple
 
 import torch
 import torch.nn as nn
@@ -46,6 +51,13 @@ def projection(rows: int, cols: int) -> nn.Parameter:
 
 def vector(n: int) -> nn.Parameter:
     return nn.Parameter(torch.zeros(n), requires_grad=False)
+
+
+def matmul_f32(x: Tensor, w: Tensor) -> Tensor:
+    """x w^T whose fp32 sums are not rounded."""
+    if x.dtype == torch.float32:
+        return torch.mm(x, w.t())
+    return torch.mm(x, w.t(), out_dtype=torch.float32)
 
 
 # ---------------------------------------------------------------------------------- attention
@@ -101,8 +113,8 @@ class ChunkedAttention(nn.Module):
     def make_cache(self, batch: int, length: int, dtype, device) -> RingCache:
         return RingCache(batch, min(self.chunk, length), self.G, self.D, self.E, dtype, device)
 
-    def decode_shapes(self, cache: RingCache, batch: int):
-        return (batch, 1, self.H, self.D), cache.k, cache.v
+    def workspace_bytes(self, cache: RingCache, batch: int) -> int:
+        return ops.attn_workspace((batch, 1, self.H, self.D), cache.k, cache.v, scale=1.0, ring=True, chunk=cache.k.shape[1])
 
     def forward(self, h: Tensor, cache: RingCache, at: Portion) -> Tensor:
         B, S = at.B, at.S
@@ -128,11 +140,36 @@ class ChunkedAttention(nn.Module):
 
 
 # ---------------------------------------------------------------------------------- latent attention
-def rotary_angles(length: int, dims: int, base: float, device) -> Tensor:
-    """[length, dims / 2, 2] = (cos, sin) of position * base^(-2i / dims), fp32."""
+@dataclass(frozen=True)
+class YarnScaling:
+    """Stretched rotary positions: pairs that turn more than `fast` times within `original` tokens keep their
+    frequency, pairs that turn less than `slow` times turn `factor` times slower, pairs between are blended; the
+    rotation is scaled by 0.1 ln(factor) + 1."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+
+def rotary_frequencies(dims: int, base: float, scaling: Optional[YarnScaling] = None) -> Tensor:
+    """Angle per position of each of the dims / 2 pairs (float64)."""
     f = base ** (-torch.arange(0, dims, 2, dtype=torch.float64) / dims)
-    a = torch.outer(torch.arange(length, dtype=torch.float64), f)
-    return torch.stack([torch.cos(a), torch.sin(a)], -1).float().contiguous().to(device)
+    if scaling is None:
+        return f
+
+    def pair(turns: float) -> float:               # the pair that turns so often within the original length
+        return dims * math.log(scaling.original / (2 * math.pi * turns)) / (2 * math.log(base))
+
+    lo, hi = max(math.floor(pair(scaling.fast)), 0), min(math.ceil(pair(scaling.slow)), dims - 1)
+    ramp = ((torch.arange(dims // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    return f / scaling.factor * ramp + f * (1 - ramp)
+
+
+def rotary_angles(length: int, dims: int, base: float, device, scaling: Optional[YarnScaling] = None) -> Tensor:
+    """[length, dims / 2, 2] = (cos, sin) of position * frequency, times the scaling's gain, fp32 (computed in double)."""
+    a = torch.outer(torch.arange(length, dtype=torch.float64), rotary_frequencies(dims, base, scaling))
+    gain = 1.0 if scaling is None else 0.1 * math.log(scaling.factor) + 1.0
+    return (torch.stack([torch.cos(a), torch.sin(a)], -1) * gain).float().contiguous().to(device)
 
 
 class LatentCache:
@@ -183,9 +220,10 @@ class LatentAttention(nn.Module):
         return LatentCache(batch, length, self.row, rotary_angles(length, self.rot_dims, self.rot_base, device), dtype,
                            device)
 
-    def decode_shapes(self, cache: LatentCache, batch: int):
+    def workspace_bytes(self, cache: LatentCache, batch: int) -> int:
         rows = cache.rows.unsqueeze(2)
-        return (batch, self.expand_from - 1, self.H, self.row), rows, rows[..., :self.K]
+        return max(ops.attn_workspace((batch, s, self.H, self.row), rows, rows[..., :self.K], scale=1.0)
+                   for s in (1, self.expand_from - 1))
 
     def forward(self, h: Tensor, cache: LatentCache, at: Portion) -> Tensor:
         B, S = at.B, at.S
@@ -207,6 +245,113 @@ class LatentAttention(nn.Module):
             v = kv[..., self.q_rows:].unflatten(-1, (self.H, self.E))
             y = ops.attn(q.view(B, S, -1).unflatten(-1, (self.H, self.D + self.R)), k, v, **args)
         return torch.mm(y.view(B * S, self.H * self.E), self.wo.t())
+
+
+# ---------------------------------------------------------------------------------- window attention
+class RingRows:
+    """The last rows [key as projected | its turned elements] of a sequence: position p lives in row p % ring."""
+
+    def __init__(self, batch: int, ring: int, kv_heads: int, row: int, angles: Tensor, dtype, device):
+        self.rows = torch.zeros(batch, ring, kv_heads, row, dtype=dtype, device=device)
+        self.angles = angles
+
+
+class WindowAttention(nn.Module):
+    """Grouped-query attention over the last `window` positions (a token itself included): rotary positions on the
+    first `rot_dims` elements of queries and keys, capped scores, a learned sink per head, and the keys as projected
+    for values.  Keys and values share their cache rows; as many rows as the window are kept.  A mixer of
+    `ParallelLayer`."""
+
+    def __init__(self, heads: int, kv_heads: int, dim: int, window: int, scale: float, rot_dims: int, rot_base: float,
+                 rot_scaling: Optional[YarnScaling], softcap: float):
+        super().__init__()
+        self.H, self.G, self.D = heads, kv_heads, dim
+        self.window, self.scale, self.softcap = window, scale, softcap
+        self.rot_dims, self.rot_base, self.rot_scaling = rot_dims, rot_base, rot_scaling
+        self.in_sizes = {"q": heads * dim, "k": kv_heads * dim}
+        self.out_size = heads * dim
+        self.sink = vector(heads)
+        self.register_buffer("sink_f32", torch.zeros(heads), persistent=False)
+        self._angles: Optional[Tensor] = None
+
+    def tensors(self) -> Dict[str, Tensor]:
+        return {"sink": self.sink}
+
+    def finish_loading(self) -> None:
+        self.sink_f32 = self.sink.float()
+
+    def make_cache(self, batch: int, length: int, dtype, device) -> RingRows:
+        if self._angles is None or self._angles.shape[0] < length or self._angles.device != torch.device(device):
+            self._angles = rotary_angles(length, self.rot_dims, self.rot_base, device, self.rot_scaling)
+        return RingRows(batch, min(self.window, length), self.G, self.D + self.rot_dims, self._angles, dtype, device)
+
+    def workspace_bytes(self, cache: RingRows, batch: int) -> int:
+        k, v = self.keys_values(cache.rows)
+        return ops.attn_workspace((batch, 1, self.H, self.D), k, v, scale=1.0, ring=True, window=self.window)
+
+    def keys_values(self, rows: Tensor) -> Tuple[Tensor, Tensor]:
+        return rows[..., self.rot_dims:], rows[..., :self.D]
+
+    def mix(self, parts: List[Tensor], h: Tensor, cache: RingRows, at: Portion, out: Tensor) -> None:
+        B, S = at.B, at.S
+        q, k = parts[0].unflatten(-1, (self.H, self.D)), parts[1].unflatten(-1, (self.G, self.D))
+        ring = cache.rows[:B]
+        args = dict(scale=self.scale, softcap=self.softcap, window=self.window, sink=self.sink_f32, status=at.status,
+                    workspace=at.workspace, out=out.view(B, S, self.H, self.D))
+        if at.pos is not None:
+            q = ops.rotary_rows(q, k, cache.angles, self.rot_dims, ring, B=B, S=S, pos=at.pos, status=at.status)
+            ops.attn(q, *self.keys_values(ring), pos=at.pos, ring=True, **args)
+        else:
+            prev = min(at.start, self.window - 1)          # earlier positions that the portion's tokens see
+            rows = torch.empty(B, prev + S, *ring.shape[2:], dtype=ring.dtype, device=ring.device)
+            q = ops.rotary_rows(q, k, cache.angles, self.rot_dims, rows, B=B, S=S, start=at.start, ring=ring, prev=prev,
+                                status=at.status)
+            ops.attn(q, *self.keys_values(rows), start=at.start, kv_start=at.start - prev, **args)
+            ops.ring_append(rows[:, prev:], None, ring, None, start=at.start, keep="window")
+
+
+# ---------------------------------------------------------------------------------- matrix memory
+class MemoryState:
+    """Recurrent state per sequence and head, fp32: the memory, its normaliser, the running maximum of the gates."""
+
+    def __init__(self, batch: int, heads: int, dim: int, vdim: int, device):
+        self.S = torch.zeros(batch, heads, dim, vdim, dtype=torch.float32, device=device)
+        self.n = torch.zeros(batch, heads, dim, dtype=torch.float32, device=device)
+        self.m = torch.zeros(batch, heads, dtype=torch.float32, device=device)
+
+
+class MatrixMemory(nn.Module):
+    """Matrix memory of the xLSTM (mLSTM) with capped exponential input gates and sigmoid forget gates, a norm per
+    head and a sigmoid output gate.  The gates' pre-activations are a matrix product of their own, whose fp32 sums
+    are not rounded.  A mixer of `ParallelLayer`."""
+
+    def __init__(self, width: int, heads: int, dim: int, vdim: int, gate_cap: float, eps: float):
+        super().__init__()
+        self.H, self.N, self.P, self.cap, self.eps = heads, dim, vdim, gate_cap, eps
+        self.in_sizes = {"q": heads * dim, "k": heads * dim, "v": heads * vdim, "g": heads * vdim}
+        self.out_size = heads * vdim
+        self.w_gates = projection(padded_rows(2 * heads), width)
+        self.i_b, self.f_b, self.norm_w = vector(heads), vector(heads), vector(heads * vdim)
+        for name in ("i_b_f32", "f_b_f32"):
+            self.register_buffer(name, torch.zeros(heads), persistent=False)
+
+    def tensors(self) -> Dict[str, Tensor]:
+        return {"i": self.w_gates[:self.H], "f": self.w_gates[self.H:2 * self.H], "i.b": self.i_b, "f.b": self.f_b,
+                "norm": self.norm_w}
+
+    def finish_loading(self) -> None:
+        self.i_b_f32, self.f_b_f32 = self.i_b.float(), self.f_b.float()
+
+    def make_cache(self, batch: int, length: int, dtype, device) -> MemoryState:
+        return MemoryState(batch, self.H, self.N, self.P, device)
+
+    def workspace_bytes(self, cache: MemoryState, batch: int) -> int:
+        return 0
+
+    def mix(self, parts: List[Tensor], h: Tensor, cache: MemoryState, at: Portion, out: Tensor) -> None:
+        B = at.B
+        ops.mlstm(*parts, matmul_f32(h, self.w_gates), self.i_b_f32, self.f_b_f32, self.norm_w, cache.S[:B], cache.n[:B],
+                  cache.m[:B], out, S=at.S, cap=self.cap, q_scale=self.N ** -0.5, eps=self.eps, start=at.start, pos=at.pos)
 
 
 # ---------------------------------------------------------------------------------- state space
@@ -247,6 +392,9 @@ class Mamba2(nn.Module):
     def make_cache(self, batch: int, length: int, dtype, device) -> StateCache:
         return StateCache(batch, self.H, self.N, self.P, self.channels, self.taps, dtype, device)
 
+    def workspace_bytes(self, cache: StateCache, batch: int) -> int:
+        return 0
+
     def forward(self, h: Tensor, cache: StateCache, at: Portion) -> Tensor:
         proj = torch.mm(h, self.w_in.t())
         y = ops.ssm(proj, self.inner, self.conv_w, self.conv_b, self.dt_bias_f32, self.A_log_f32, self.skip_f32,
@@ -271,3 +419,45 @@ class ClampedFeedForward(nn.Module):
 
     def forward(self, h: Tensor) -> Tensor:
         return torch.mm(ops.glu_clamped(torch.mm(h, self.w13.t()), self.ff, self.limit), self.w2.t())
+
+
+class ParallelLayer(nn.Module):
+    """A layer whose mixer and feed-forward (silu-gated; ff = 0: none) read the same normed rows and add to the
+    stream together: one matrix product makes every projection of both, one takes [mixer | feed-forward] to what
+    the stream gets, summed in fp32."""
+
+    def __init__(self, width: int, mixer: nn.Module, ff: int):
+        super().__init__()
+        self.mixer, self.ff = mixer, ff
+        self.norm1 = vector(width)
+        sizes = list(mixer.in_sizes.values()) + ([ff, ff] if ff else [])
+        self.in_slices, rows = [], 0
+        for n in sizes:                            # every slice starts at a multiple of 8 columns of the projected rows
+            self.in_slices.append(slice(rows, rows + n))
+            rows += padded_rows(n)
+        self.w_in = projection(rows, width)
+        self.ff_at = padded_rows(mixer.out_size)
+        self.cols = self.ff_at + padded_rows(ff)
+        self.gaps = self.cols != mixer.out_size + ff
+        self.w_out = projection(width, self.cols)
+
+    def tensors(self) -> Dict[str, Tensor]:
+        out = {"norm1": self.norm1, "mix.o": self.w_out[:, :self.mixer.out_size]}
+        for name, s in zip(self.mixer.in_sizes, self.in_slices):
+            out["mix." + name] = self.w_in[s]
+        out.update({"mix." + k: v for k, v in self.mixer.tensors().items()})
+        if self.ff:
+            gate, up = self.in_slices[-2:]
+            out.update({"mlp.gate": self.w_in[gate], "mlp.up": self.w_in[up],
+                        "mlp.down": self.w_out[:, self.ff_at:self.ff_at + self.ff]})
+        return out
+
+    def forward(self, h: Tensor, cache, at: Portion) -> Tensor:
+        proj = torch.mm(h, self.w_in.t())
+        parts = [proj[:, s] for s in self.in_slices]
+        make = torch.zeros if self.gaps else torch.empty           # columns between the two parts meet zero weights
+        inner = make(h.shape[0], self.cols, dtype=h.dtype, device=h.device)
+        self.mixer.mix(parts[:len(self.mixer.in_sizes)], h, cache, at, inner[:, :self.mixer.out_size])
+        if self.ff:
+            ops.glu_silu(*parts[-2:], out=inner[:, self.ff_at:self.ff_at + self.ff])
+        return matmul_f32(inner, self.w_out)

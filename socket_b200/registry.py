@@ -68,6 +68,11 @@ def _radapel(config: Mapping, shapes: Optional[Mapping[str, Tuple[int, ...]]]) -
     return Radapel(RadapelConfig.from_dict(config, shapes))
 
 
+def _timalorn(config: Mapping, shapes) -> Decoder:
+    from .timalorn import Timalorn, TimalornConfig
+    return Timalorn(TimalornConfig.from_dict(config))
+
+
 def _transformer(config: Mapping, shapes) -> Decoder:
     from .model import ModelArgs, Transformer
     return Transformer(ModelArgs(**{k: v for k, v in config.items() if k != "architecture"}))
@@ -75,6 +80,7 @@ def _transformer(config: Mapping, shapes) -> Decoder:
 
 ARCHITECTURES = {
     "Radapel": (_radapel, ("blocks",)),
+    "Timalorn": (_timalorn, ("blocks",)),
     "Transformer": (_transformer, ("step",)),
 }
 
