@@ -32,6 +32,7 @@ def test_block_library_exports_every_declared_symbol():
 
 
 @pytest.mark.parametrize("struct,cls", [("sk_residual_params", _lib.ResidualParams), ("sk_attn_params", _lib.AttnParams),
+                                        ("sk_rotary_rows_params", _lib.RotaryRowsParams), ("sk_mlstm_params", _lib.MlstmParams),
                                         ("sk_latent_params", _lib.LatentParams), ("sk_ssm_params", _lib.SsmParams)])
 def test_block_structs_match_the_header(struct, cls):
     text = open(os.path.join(ROOT, "include", "socket_b200_blocks.h")).read()
