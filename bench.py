@@ -1,6 +1,6 @@
 """Benchmark of the sparse-attention decode path (one layer, one decode step per "step").
 
-    python bench.py [--gpus N] [--steps K] [--warmup W] [--workload c3|c2|c4|radapel] [--impl reference]
+    python bench.py [--gpus N] [--steps K] [--warmup W] [--workload c3|c2|c4|radapel|timalorn] [--impl reference]
 
 Default workload: the 128K long-context configuration (`c3`: batch 4, 32 query / 8 KV heads,
 context 131072, top-k 2048 + 64 + 256).  With N > 1 GPUs its 8 KV heads are split over the ranks
@@ -63,10 +63,11 @@ def parse_args():
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=1000)
     ap.add_argument("--warmup", type=int, default=20)
-    ap.add_argument("--workload", default="c3", choices=sorted(PRESETS) + ["c4", "c4-128k", "c4-128k-b4", "c5", "radapel"],
+    ap.add_argument("--workload", default="c3", choices=sorted(PRESETS) + ["c4", "c4-128k", "c4-128k-b4", "c5", "radapel", "timalorn"],
                     help="c1-c3: one attention layer (op level); c4 / c5: whole-model greedy decode, "
                          "Llama-3-8B / Llama-3-70B shape with random weights; radapel: the Radapel decoder "
-                         "beside the Transformer, and its kernels one by one")
+                         "beside the Transformer, and its kernels one by one; timalorn: the Timalorn decoder beside "
+                         "Radapel, the same way")
     ap.add_argument("--model-record", default="auto", choices=["auto", "on", "off"],
                     help="also run the whole-model decode comparison (c4) and attach it to the line; "
                          "auto = on a single GPU only")
@@ -859,20 +860,8 @@ def time_op(fn, flush, n=20):
     return times[0] - times[1]
 
 
-def measure_radapel_kernels(size, S, T, B, dev):
-    """Every kernel of the design beside the like kernel of the Llama-shaped model, at one size: prefill
-    kernels on S tokens from position 0, decode kernels for B sequences at context T."""
-    import torch.nn.functional as F
-    from flash_attn import flash_attn_func, flash_attn_with_kvcache
-    from socket_b200 import block_ops as ops
-    from socket_b200.mixers import LatentCache, Mamba2, Portion, rotary_angles  # noqa: F401
-    from socket_b200.model import apply_rotary_emb
-    W, H, G, D, FF, K, M = RADAPEL_SIZES[size]
-    R, N, P = RADAPEL_ROT, RADAPEL_STATE, 64
-    bf = torch.bfloat16
-    rn = lambda *s: torch.randn(*s, device=dev, dtype=bf)  # noqa: E731
-    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
-    peaks = measured_peaks()
+def kernel_table(peaks):
+    """(rows, add): add(...) appends one kernel with its share of the roofline, beside a like kernel and its share."""
     rows = []
 
     def add(name, us, like, like_us, flops=0.0, nbytes=0.0, like_flops=None, like_bytes=None):
@@ -888,6 +877,24 @@ def measure_radapel_kernels(size, S, T, B, dev):
             r.update(like=like, like_us=round(like_us, 2), like_roofline_frac=round(frac(like_us, lf, lb), 3))
             r["like_frac_over_frac"] = round(r["like_roofline_frac"] / max(r["roofline_frac"], 1e-9), 2)
         rows.append(r)
+    return rows, add
+
+
+def measure_radapel_kernels(size, S, T, B, dev):
+    """Every kernel of the design beside the like kernel of the Llama-shaped model, at one size: prefill
+    kernels on S tokens from position 0, decode kernels for B sequences at context T."""
+    import torch.nn.functional as F
+    from flash_attn import flash_attn_func, flash_attn_with_kvcache
+    from socket_b200 import block_ops as ops
+    from socket_b200.mixers import LatentCache, Mamba2, Portion, rotary_angles  # noqa: F401
+    from socket_b200.model import apply_rotary_emb
+    W, H, G, D, FF, K, M = RADAPEL_SIZES[size]
+    R, N, P = RADAPEL_ROT, RADAPEL_STATE, 64
+    bf = torch.bfloat16
+    rn = lambda *s: torch.randn(*s, device=dev, dtype=bf)  # noqa: E731
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    peaks = measured_peaks()
+    rows, add = kernel_table(peaks)
 
     # ---- attention of a prompt
     q, k, v = rn(1, S, H, D), rn(1, S, G, D), rn(1, S, G, D)
@@ -1031,10 +1038,179 @@ def run_radapel(args, dev):
         "peaks": measured_peaks(), "clocks": clocks.stop(), "radapel": out}))
 
 
+# ------------------------------------------------------------------------------- Timalorn
+TIMALORN_MEMORY = {"2k": (8, 128, 256), "4k": (8, 256, 512)}     # heads, key size, value size
+TIMALORN_WINDOW, TIMALORN_ROT, TIMALORN_CAP = 4096, 64, 50.0
+
+
+def timalorn_config(size):
+    """Attention and memory in turn, 7 layers, two of which use the tensors of earlier ones; width, heads and
+    feed-forward of the Radapel size."""
+    W, H, G, D, F, *_ = RADAPEL_SIZES[size]
+    MH, N, P = TIMALORN_MEMORY[size]
+    mlp = {"kind": "dense", "ff": F}
+    att = {"type": "attention", "mlp": mlp,
+           "mixer": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "softcap": TIMALORN_CAP,
+                     "mask": {"size": TIMALORN_WINDOW},
+                     "rot": {"base": 500000.0, "dims": TIMALORN_ROT,
+                             "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}}
+    mem = {"type": "mlstm", "mlp": mlp, "mixer": {"heads": MH, "dim": N, "vdim": P, "gate_cap": 15.0}}
+    return {"architecture": "Timalorn", "vocab": 32768, "width": W, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "layers": [att, mem, att, mem, dict(att, weights_of=0), dict(mem, weights_of=1), att]}
+
+
+def weights_per_token(model):
+    """Elements of the matrices a token passes through (shared ones as often as they are used)."""
+    layers = sum(p.numel() for r in model.runs for p in model.layer_of(r).parameters())
+    return layers + model.head.numel()
+
+
+def measure_timalorn_kernels(size, S, T, B, dev):
+    """Every kernel of the design beside the like kernel of Radapel, at one size: prefill kernels on S tokens from
+    position 0, decode kernels for B sequences at context T."""
+    from socket_b200 import block_ops as ops
+    from socket_b200.mixers import Mamba2, YarnScaling, rotary_angles
+    W, H, G, D, FF, K, M = RADAPEL_SIZES[size]
+    MH, N, P = TIMALORN_MEMORY[size]
+    R, WIN, RN, RP = TIMALORN_ROT, TIMALORN_WINDOW, RADAPEL_STATE, 64
+    bf = torch.bfloat16
+    rn = lambda *s: torch.randn(*s, device=dev, dtype=bf)  # noqa: E731
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    t = lambda fn: time_op(fn, flush)  # noqa: E731
+    rows, add = kernel_table(measured_peaks())
+    ws = torch.empty(64 << 20, dtype=torch.uint8, device=dev)
+    # ---- attention of a prompt
+    sink, bias = torch.randn(H, device=dev), torch.randn(H, 1025, device=dev)
+    q, k, v = rn(1, S, H, D), rn(1, S, G, D), rn(1, S, G, D)
+    kv = rn(1, S, G, D + R)
+    kw = dict(scale=D ** -0.5, window=WIN, sink=sink)
+    pairs, full = sum(min(i + 1, WIN) for i in range(S)), S * (S + 1) / 2
+    like = t(lambda: ops.attn(q, k, v, scale=D ** -0.5, chunk=RADAPEL_CHUNK, bias=bias))
+    lk = dict(like="chunked attention", like_us=like, like_flops=full * H * 4 * D)
+    add(f"window attention, capped scores, prefill (window {WIN})",
+        t(lambda: ops.attn(q, kv[..., R:], kv[..., :D], softcap=TIMALORN_CAP, **kw)), flops=pairs * H * 4 * D, **lk)
+    big = q * (4 * TIMALORN_CAP)                   # scores at the cap: the form without the polynomial
+    add("the same, scores at the cap", t(lambda: ops.attn(big, kv[..., R:], kv[..., :D], softcap=TIMALORN_CAP, **kw)),
+        flops=pairs * H * 4 * D, **lk)
+    add("the same without a cap", t(lambda: ops.attn(q, kv[..., R:], kv[..., :D], **kw)), flops=pairs * H * 4 * D, **lk)
+    # ---- attention of a decoded token
+    pos = torch.tensor([T - 1], device=dev)
+    q1, ring = rn(B, 1, H, D), rn(B, WIN, G, D + R)
+    kr, vr = rn(B, WIN, G, D), rn(B, WIN, G, D)
+    ringpos = torch.tensor([WIN - 1], device=dev)
+    add(f"window attention, decode (ring {WIN} full)",
+        t(lambda: ops.attn(q1, ring[..., R:], ring[..., :D], pos=pos, ring=True, softcap=TIMALORN_CAP, workspace=ws, **kw)),
+        "chunked attention, ring as long",
+        t(lambda: ops.attn(q1, kr, vr, scale=D ** -0.5, pos=ringpos, chunk=WIN, ring=True, bias=bias, workspace=ws)),
+        nbytes=B * WIN * G * (D + R) * 2, like_bytes=B * WIN * G * 2 * D * 2)
+    # ---- rotation and cache rows
+    ang = rotary_angles(max(S, T), R, 500000.0, dev, YarnScaling(4.0, 8192, 32.0, 1.0))
+    ang_l = rotary_angles(max(S, T), RADAPEL_ROT, 500000.0, dev)
+    cols = (H + G) * D
+
+    def rotary(n, start, rows_out, **more):
+        proj = rn(n, cols)
+        qq, kk = proj[:, :H * D].unflatten(-1, (H, D)), proj[:, H * D:].unflatten(-1, (G, D))
+        return t(lambda: ops.rotary_rows(qq, kk, ang, R, rows_out, start=start, **more))
+
+    def latent(n, s, cache, **more):
+        dkv, qq, lw = rn(n, K + RADAPEL_ROT), rn(n, H * (D + RADAPEL_ROT)), rn(K)
+        return t(lambda: ops.latent_append(dkv, qq, lw, ang_l, cache, S=s, n_heads=H, dim=D, rot=RADAPEL_ROT, rank=K, eps=1e-5, **more))
+
+    add("rotary rows, prefill", rotary(S, 0, torch.empty(1, S, G, D + R, dtype=bf, device=dev), B=1, S=S),
+        "latent append + rotation", latent(S, S, rn(1, S, K + RADAPEL_ROT)),
+        nbytes=S * 2 * (2 * H * D + G * (2 * D + R)), like_bytes=S * (4 * (K + RADAPEL_ROT) + 4 * H * RADAPEL_ROT))
+    add("rotary rows, decode", rotary(B, 0, ring, B=B, S=1, pos=pos), "latent append + rotation",
+        latent(B, 1, rn(B, T, K + RADAPEL_ROT), pos=pos),
+        nbytes=B * 2 * (2 * H * D + G * (2 * D + R)), like_bytes=B * (4 * (K + RADAPEL_ROT) + 4 * H * RADAPEL_ROT))
+    add("ring append of a prompt", t(lambda: ops.ring_append(kv, None, ring[:1], None, start=0, keep="window")),
+        "ring append of a chunk", t(lambda: ops.ring_append(k, v, kr[:1], vr[:1], start=0)),
+        nbytes=WIN * G * (D + R) * 4, like_bytes=WIN * G * 2 * D * 4)
+    # ---- residual stream, gated unit
+    for name, n in (("prefill", S), ("decode", B)):
+        x, y, y16, w = torch.randn(n, W, device=dev), torch.randn(n, W, device=dev), rn(n, W), rn(W)
+        add(f"residual + layer norm, {name}", t(lambda: ops.residual_norm(x, 1e-5, y=y, w_out=w, centred=True)),
+            "residual + two norms", t(lambda: ops.residual_norm(x, 1e-5, y=y16, w_in=w, w_out=w)),
+            nbytes=n * W * 14 + 2 * W, like_bytes=n * W * 12 + 4 * W)
+        gu, wide = rn(n, 2 * FF), rn(n, FF + H * D)
+        add(f"silu unit, {name}", t(lambda: ops.glu_silu(gu[:, :FF], gu[:, FF:], out=wide[:, H * D:])),
+            "clamped unit", t(lambda: ops.glu_clamped(gu, FF, 7.0)), nbytes=n * FF * 6)
+    # ---- recurrences
+    mix = Mamba2(W, M, RP, RN, 8, 4, 8, 1e-5).to(device=dev, dtype=bf)
+    mix.finish_loading()
+    inner, chans = mix.inner, mix.channels
+    sargs = (mix.conv_w, mix.conv_b, mix.dt_bias_f32, mix.A_log_f32, mix.skip_f32)
+    st = mix.make_cache(B, T, bf, dev)
+    Ss, ns, ms = (torch.zeros(s, device=dev) for s in ((B, MH, N, P), (B, MH, N), (B, MH)))
+    ib, fb, nw = torch.zeros(MH, device=dev), torch.full((MH,), 3.0, device=dev), rn(MH * P)
+
+    def memory(n, s, **more):
+        proj, gates = rn(n, 2 * MH * (N + P)), torch.randn(n, 2 * MH, device=dev)
+        a, b = MH * N, 2 * MH * N
+        parts = (proj[:, :a], proj[:, a:b], proj[:, b:b + MH * P], proj[:, b + MH * P:])
+        nb = n // s
+        out = torch.empty(n, MH * P, dtype=bf, device=dev)
+        return t(lambda: ops.mlstm(*parts, gates, ib, fb, nw, Ss[:nb], ns[:nb], ms[:nb], out, S=s, cap=15.0, q_scale=N ** -0.5,
+                                   eps=1e-5, **more))
+
+    def state_space(n, s, **more):
+        proj, nb = rn(n, mix.w_in.shape[0]), n // s
+
+        def run():
+            y = ops.ssm(proj, inner, *sargs, st.conv[:nb], st.state[:nb], S=s, groups=8, **more)
+            ops.gated_group_norm(y, proj, mix.norm_w, 8, 1e-5)
+        return t(run)
+
+    blk = 64                                       # causal half of a block's products, and the state's
+    add("matrix memory, prefill (gates, blocks, norm and gate)", memory(S, S), "state space (convolution, blocks, gated norm)", state_space(S, S),
+        flops=S * MH * (blk * N + blk * P + 4 * N * P), nbytes=S * MH * 2 * (2 * N + 3 * P),
+        like_flops=S * M * (blk * RN + blk * RP + 4 * RN * RP), like_bytes=S * (inner * 6 + chans * 6))
+    add("matrix memory, decode (step, norm and gate)", memory(B, 1, pos=pos), "state space (convolution, step, gated norm)",
+        state_space(B, 1, pos=pos), nbytes=B * MH * N * P * 8, like_bytes=B * M * RN * RP * 8)
+    h, wg = rn(S, W), rn(2 * MH, W)
+    from socket_b200.mixers import matmul_f32
+    add("gates' projection, prefill (library product)", t(lambda: matmul_f32(h, wg)), None, 0, nbytes=S * W * 2)
+    add("gates' projection, decode (library product)", t(lambda: matmul_f32(h[:B], wg)), None, 0, nbytes=2 * MH * W * 2)
+    return rows
+
+
+def run_timalorn(args, dev):
+    """Prefill and decode throughput of Timalorn at two sizes beside Radapel with as many layer runs, the same
+    width, heads and feed-forward, and the kernels one by one."""
+    from socket_b200.registry import build_model
+    torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
+    K, W = min(args.steps, 64), max(3, min(args.warmup, 8))
+    clocks = ClockSampler(dev.index or 0)
+    out = {}
+    for size in RADAPEL_SIZES:
+        rec = {"width": RADAPEL_SIZES[size][0]}
+        for name, cfg in (("timalorn", timalorn_config(size)), ("radapel", radapel_config(size))):
+            model = build_model(cfg, dtype=torch.bfloat16, device=dev).init_random(args.seed)
+            rec[f"{name} layer runs"], rec[f"{name} weights per token"] = len(model.runs), weights_per_token(model)
+            for B, T in [(1, 2048), (1, 8000), (1, 32000), (8, 8000)]:
+                rec[f"{name} B={B} T={T}"] = measure_throughput(model, cfg["vocab"], B, T, K, W, dev)
+            rec[f"{name} device flags"] = model.device_flags()
+            del model
+            torch.cuda.empty_cache()
+        rec["kernels S=8192, decode B=1 T=32768"] = measure_timalorn_kernels(size, 8192, 32768, 1, dev)
+        torch.cuda.empty_cache()
+        out[size] = rec
+    main_rec = out["4k"]["timalorn B=1 T=32000"]
+    print(json.dumps({
+        "metric": "decode_tokens_per_s", "value": main_rec["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": K,
+        "warmup": W, "ms_per_step": main_rec["decode_ms_per_token"], "higher_is_better": True, "scaling": "weak",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "config": {"model": "Timalorn 4k, 7 layers, random weights", "global_batch": 1, "seq_len": 32000,
+                   "parallelism": "single GPU", "timing": "CUDA events around K graph-replayed decode tokens; weights exceed L2; "
+                   "kernels one by one with L2 flushed"},
+        "e2e": {"value": main_rec["e2e_decode_tokens_per_s"], "unit": "tokens/s", "h2d_bytes_per_step": 0, "d2h_bytes_per_step": 8},
+        "peaks": measured_peaks(), "clocks": clocks.stop(), "timalorn": out}))
+
+
 def main():
     args = parse_args()
     if args.impl == "reference":
-        if args.workload in MODEL_WORKLOADS or args.workload == "radapel":
+        if args.workload in MODEL_WORKLOADS or args.workload in ("radapel", "timalorn"):
             if int(os.environ.get("RANK", "0")) == 0:
                 print(json.dumps({"impl": "reference", "unavailable": "the whole-model workloads have no CPU arm: the "
                                   "reference's CPU path is timed at the op level (c1-c3)"}))
@@ -1057,6 +1233,9 @@ def main():
 
     if args.workload == "radapel":
         run_radapel(args, torch.device("cuda", local_rank))
+        return
+    if args.workload == "timalorn":
+        run_timalorn(args, torch.device("cuda", local_rank))
         return
     if args.workload in MODEL_WORKLOADS:
         K = min(K, MODEL_WORKLOADS[args.workload][3] - 1)

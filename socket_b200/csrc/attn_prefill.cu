@@ -6,7 +6,8 @@
 // thread per query row: they read the row's 128 scores, scale / bias / mask them, keep the running maximum and sum,
 // and write the weights back over the scores as bf16.  While one tile is in its softmax the tensor
 // core works on the other.  The accumulator is rescaled only when a row's maximum has grown by more than
-// 2^8 since the last time (the final division by the sum makes the choice of reference invisible).
+// 2^8 since the last time (the final division by the sum makes the choice of reference invisible).  Scores under
+// a cap are bounded, so weights are taken relative to zero: no maximum, no rescaling.
 //
 // Visibility is causal, optionally restricted to the query's own chunk of positions or to a sliding window; tiles
 // that no row of a query tile can see are not visited.  Out-of-range rows and columns of a tile are zero-filled by TMA.
@@ -44,7 +45,11 @@ struct FpShape {            // what the kernel needs beside the tensor maps
     int64_t o_bs, o_ss, o_hs, start, kv_start, bias_len;
     int S, H, G, dqk, dv, chunk, window, nk, nv;      // nk, nv: stages of the K and V rings
     float scale_log2, cap_in, cap_out;        // softcap: s <- cap_out tanh(s cap_in), log2 units
+    float cap_poly[5], cap_small;             // the same for s^2 <= cap_small: s times a polynomial in s^2
 };
+// Softcap: none, any, or one so low that exp of a capped score and sums of it stay far inside the fp32 range
+enum { FP_CAP_NONE = 0, FP_CAP = 1, FP_CAP_BOUND = 2 };
+constexpr float FP_CAP_BOUND_LOG2 = 80.f;
 
 // first key row (in key-row coordinates, may be negative) that query row i sees
 __device__ __forceinline__ int64_t fp_first_row(const FpShape& p, int64_t i) {
@@ -54,7 +59,38 @@ __device__ __forceinline__ int64_t fp_first_row(const FpShape& p, int64_t i) {
     return lo;
 }
 
-template <bool BIAS, bool CAP>
+// s <- cap_out tanh(s cap_in) for 32 scores from c0 on; the caller's loops are unrolled
+template <int N> __device__ __forceinline__ void fp_cap32(const FpShape& p, float (&s)[N], int c0) {
+    uint64_t t[16];
+    float top[2] = {0.f, 0.f};
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+        const uint64_t x = pack2(s[c0 + 2 * i], s[c0 + 2 * i + 1]);
+        t[i] = mul2(x, x);
+        float a, b;
+        unpack2(t[i], a, b);
+        top[i & 1] = max3(top[i & 1], a, b);
+    }
+    if (__any_sync(FULL, !(fmaxf(top[0], top[1]) <= p.cap_small))) {
+#pragma unroll
+        for (int c = 0; c < 32; ++c) s[c0 + c] = p.cap_out * tanh_exp2(s[c0 + c] * p.cap_in);
+    } else {
+        const uint64_t k0 = pack2(p.cap_poly[0], p.cap_poly[0]), k1 = pack2(p.cap_poly[1], p.cap_poly[1]),
+                       k2 = pack2(p.cap_poly[2], p.cap_poly[2]), k3 = pack2(p.cap_poly[3], p.cap_poly[3]),
+                       k4 = pack2(p.cap_poly[4], p.cap_poly[4]);
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            uint64_t r = fma2(t[i], k4, k3);
+            r = fma2(t[i], r, k2);
+            r = fma2(t[i], r, k1);
+            r = fma2(t[i], r, k0);
+            r = mul2(r, pack2(s[c0 + 2 * i], s[c0 + 2 * i + 1]));
+            unpack2(r, s[c0 + 2 * i], s[c0 + 2 * i + 1]);
+        }
+    }
+}
+
+template <bool BIAS, int CAP>
 __global__ void __launch_bounds__(FP_THREADS, 1)
 attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_v, const FpShape p) {
@@ -201,11 +237,11 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         const uint32_t lane_base = (uint32_t)(quad * 32) << 16;
         const uint32_t s_addr = tmem + lane_base + t * FP_TILE, o_addr = tmem + lane_base + 2 * FP_TILE + t * FP_TILE;
         const int64_t i = i0[t] + a;                          // query row in key-row coordinates
-        const float cc = BIAS || CAP ? 1.f : p.scale_log2;    // log2 units per unit of s below
+        const float cc = BIAS || CAP != FP_CAP_NONE ? 1.f : p.scale_log2;    // log2 units per unit of s below
         const int64_t lo_row = fp_first_row(p, i), lo_last = fp_first_row(p, i0[t] + FP_TILE - 1);
         float* bt = bias_s + (warp - FP_SOFTMAX_WARP0) * FP_BIAS_SPAN;
         const float* bias_h = BIAS ? p.bias + (int64_t)h * p.bias_len : nullptr;
-        float m = -INFINITY, l = 0.f;
+        float m = CAP == FP_CAP_BOUND ? 0.f : -INFINITY, l = 0.f;
         bool ok = true;
         for (int j = beg[t]; j < end[t]; ++j) {
             const int it = j - beg[t];
@@ -225,69 +261,92 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 break;
             }
             tc_fence_after();
-            float s[FP_TILE];
-            tmem_ld128(s_addr, reinterpret_cast<uint32_t(&)[FP_TILE]>(s));
-            if (CAP) {                                        // small scores: a polynomial, off the exponential's unit
-                float top[4] = {0.f, 0.f, 0.f, 0.f};
+            const bool partial = r0 + FP_TILE - 1 > i0[t] || r0 < lo_last;    // some row does not see the whole tile
+            const int hi_c = (int)(i - r0 < FP_TILE ? i - r0 : FP_TILE), lo_c = (int)(lo_row - r0 > 0 ? lo_row - r0 : 0);
+            if constexpr (CAP == FP_CAP_BOUND) {
+                // nothing depends on the whole row: 32 scores at a time become 16 columns of weights, which overwrite
+                // only scores that have been read
+                uint64_t ls[2] = {0, 0};                      // two pairs of sums
 #pragma unroll
-                for (int c = 0; c < FP_TILE; ++c) top[c & 3] = fmaxf(top[c & 3], fabsf(s[c]));
-                const float t4 = fmaxf(fmaxf(top[0], top[1]), fmaxf(top[2], top[3]));
-                if (__any_sync(FULL, !(t4 * p.cap_in <= TANH_POLY_RANGE))) {
+                for (int c0 = 0; c0 < FP_TILE; c0 += 32) {
+                    float s[32];
+                    tmem_ld32(s_addr + c0, reinterpret_cast<uint32_t(&)[32]>(s));
+                    fp_cap32(p, s, 0);
+                    if (partial) {
 #pragma unroll
-                    for (int c = 0; c < FP_TILE; ++c) s[c] = p.cap_out * tanh_exp2(s[c] * p.cap_in);
-                } else {
+                        for (int c = 0; c < 32; ++c)
+                            if (c0 + c > hi_c || c0 + c < lo_c) s[c] = -INFINITY;
+                    }
+                    uint32_t w[16];
 #pragma unroll
-                    for (int c = 0; c < FP_TILE; ++c) {
-                        const float x = s[c] * p.cap_in;
-                        s[c] = (s[c] * p.scale_log2) * tanh_over_x(x * x);
+                    for (int c = 0; c < 16; ++c) {
+                        const float x = exp2_fast(s[2 * c]), y = exp2_fast(s[2 * c + 1]);
+                        ls[c & 1] = add2(ls[c & 1], pack2(x, y));
+                        const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
+                        w[c] = *reinterpret_cast<const uint32_t*>(&v);
+                    }
+                    tmem_st16(s_addr + c0 / 2, w);
+                }
+                float l0, l1;
+                unpack2(add2(ls[0], ls[1]), l0, l1);
+                l += l0 + l1;
+            } else {
+                float s[FP_TILE];
+                tmem_ld128(s_addr, reinterpret_cast<uint32_t(&)[FP_TILE]>(s));
+                if (CAP != FP_CAP_NONE) {                         // small scores: a polynomial, off the exponential's unit
+#pragma unroll
+                    for (int c = 0; c < FP_TILE; c += 32) fp_cap32(p, s, c);
+                }
+                if (BIAS) {
+#pragma unroll
+                    for (int c = 0; c < FP_TILE; ++c) s[c] = fmaf(s[c], CAP != FP_CAP_NONE ? 1.f : p.scale_log2, bt[lane + FP_TILE - 1 - c]);
+                }
+                if (partial) {
+#pragma unroll
+                    for (int c = 0; c < FP_TILE; ++c)
+                        if (c > hi_c || c < lo_c) s[c] = -INFINITY;
+                }
+                float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+                for (int c = 0; c < FP_TILE; c += 2) mx[(c >> 1) & 3] = max3(mx[(c >> 1) & 3], s[c], s[c + 1]);
+                const float mn = fmaxf(m, fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])));
+                if (it == 0) {
+                    m = mn;
+                } else if (__any_sync(FULL, (mn - m) * cc > FP_RESCALE)) {
+                    // the scores of this tile were issued after the previous tile's P V, so O is complete
+                    const float f = mn == -INFINITY ? 1.f : exp2_fast((m - mn) * cc);
+                    l *= f;
+                    m = mn;
+                    for (int c = 0; c < p.dv; c += 32) {
+                        uint32_t r[32];
+                        tmem_ld32(o_addr + c, r);
+#pragma unroll
+                        for (int e = 0; e < 32; ++e) r[e] = __float_as_uint(__uint_as_float(r[e]) * f);
+                        tmem_st32(o_addr + c, r);
                     }
                 }
-            }
-            if (BIAS) {
+                const float mc = m == -INFINITY ? 0.f : m * cc;
+                const uint64_t scale2 = pack2(cc, cc), shift2 = pack2(-mc, -mc);
+                uint64_t ls[2] = {0, 0};
 #pragma unroll
-                for (int c = 0; c < FP_TILE; ++c) s[c] = fmaf(s[c], CAP ? 1.f : p.scale_log2, bt[lane + FP_TILE - 1 - c]);
-            }
-            if (r0 + FP_TILE - 1 > i0[t] || r0 < lo_last) {   // some row does not see the whole tile
-                const int hi_c = (int)(i - r0 < FP_TILE ? i - r0 : FP_TILE), lo_c = (int)(lo_row - r0 > 0 ? lo_row - r0 : 0);
+                for (int half = 0; half < 2; ++half) {
+                    uint32_t w[32];
 #pragma unroll
-                for (int c = 0; c < FP_TILE; ++c)
-                    if (c > hi_c || c < lo_c) s[c] = -INFINITY;
-            }
-            float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-#pragma unroll
-            for (int c = 0; c < FP_TILE; ++c) mx[c & 3] = fmaxf(mx[c & 3], s[c]);
-            const float mn = fmaxf(m, fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])));
-            if (it == 0) {
-                m = mn;
-            } else if (__any_sync(FULL, (mn - m) * cc > FP_RESCALE)) {
-                // the scores of this tile were issued after the previous tile's P V, so O is complete
-                const float f = mn == -INFINITY ? 1.f : exp2_fast((m - mn) * cc);
-                l *= f;
-                m = mn;
-                for (int c = 0; c < p.dv; c += 32) {
-                    uint32_t r[32];
-                    tmem_ld32(o_addr + c, r);
-#pragma unroll
-                    for (int e = 0; e < 32; ++e) r[e] = __float_as_uint(__uint_as_float(r[e]) * f);
-                    tmem_st32(o_addr + c, r);
+                    for (int c = 0; c < 32; ++c) {
+                        float x = s[half * 64 + 2 * c], y = s[half * 64 + 2 * c + 1];
+                        unpack2(fma2(pack2(x, y), scale2, shift2), x, y);
+                        x = exp2_fast(x);
+                        y = exp2_fast(y);
+                        ls[c & 1] = add2(ls[c & 1], pack2(x, y));
+                        const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
+                        w[c] = *reinterpret_cast<const uint32_t*>(&v);
+                    }
+                    tmem_st32(s_addr + half * 32, w);
                 }
+                float l0, l1;
+                unpack2(add2(ls[0], ls[1]), l0, l1);
+                l += l0 + l1;
             }
-            const float mc = m == -INFINITY ? 0.f : m * cc;
-            float ls[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                uint32_t w[32];
-#pragma unroll
-                for (int c = 0; c < 32; ++c) {
-                    const float x = exp2_fast(fmaf(s[half * 64 + 2 * c], cc, -mc));
-                    const float y = exp2_fast(fmaf(s[half * 64 + 2 * c + 1], cc, -mc));
-                    ls[c & 3] += x + y;
-                    const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
-                    w[c] = *reinterpret_cast<const uint32_t*>(&v);
-                }
-                tmem_st32(s_addr + half * 32, w);
-            }
-            l += (ls[0] + ls[1]) + (ls[2] + ls[3]);
             tmem_wait_st();
             tc_fence_before();
             __syncwarp();
@@ -379,13 +438,18 @@ int launch_attn_prefill_tc(const sk_attn_params& p, cudaStream_t st) {
     f.scale_log2 = p.scale * FP_LOG2E;
     f.cap_in = p.softcap > 0.f ? p.scale / p.softcap : 0.f;
     f.cap_out = p.softcap * FP_LOG2E;
+    double c = p.scale * 1.4426950408889634, c2 = (double)f.cap_in * f.cap_in;
+    for (int k = 0; k < 5; ++k, c *= c2) f.cap_poly[k] = (float)(TANH_POLY[k] * c);
+    f.cap_small = f.cap_in > 0.f ? (TANH_POLY_RANGE / f.cap_in) * (TANH_POLY_RANGE / f.cap_in) : 0.f;
     const uint32_t smem = plan_smem(p.dqk, p.dv, p.bias != nullptr, &f.nk, &f.nv);
     CUtensorMap mq, mk, mv;
     if (int rc = make_head_map(&mq, p.q, p.dqk, p.H, p.S, p.B, p.q_hs, p.q_ss, p.q_bs, FP_TILE)) return rc;
     if (int rc = make_head_map(&mk, p.k, p.dqk, p.G, p.kv_rows, p.B, p.k_hs, p.k_ts, p.k_bs, FP_TILE)) return rc;
     if (int rc = make_head_map(&mv, p.v, p.dv, p.G, p.kv_rows, p.B, p.v_hs, p.v_ts, p.v_bs, FP_TILE)) return rc;
-    auto kern = p.softcap > 0.f ? (p.bias != nullptr ? attn_prefill_kernel<true, true> : attn_prefill_kernel<false, true>)
-                                : (p.bias != nullptr ? attn_prefill_kernel<true, false> : attn_prefill_kernel<false, false>);
+    auto kern = p.bias != nullptr ? attn_prefill_kernel<true, FP_CAP_NONE> : attn_prefill_kernel<false, FP_CAP_NONE>;
+    if (p.softcap > 0.f)
+        kern = p.bias != nullptr ? attn_prefill_kernel<true, FP_CAP>
+                                 : (f.cap_out <= FP_CAP_BOUND_LOG2 ? attn_prefill_kernel<false, FP_CAP_BOUND> : attn_prefill_kernel<false, FP_CAP>);
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return fail(SK_ERR_CUDA, "attn_prefill_kernel smem attribute: %s", cudaGetErrorString(e));
     dim3 grid((unsigned)((p.S + 2 * FP_TILE - 1) / (2 * FP_TILE)), (unsigned)p.H, (unsigned)p.B);

@@ -87,12 +87,7 @@ __device__ __forceinline__ float tanh_exp2(float x) {
 }
 // tanh(x) / x for |x| <= 1/2 as a polynomial in x^2: interpolation at Chebyshev nodes, error 1.3e-8
 constexpr float TANH_POLY_RANGE = 0.5f;
-__device__ __forceinline__ float tanh_over_x(float x2) {
-    float r = fmaf(x2, 0.017141319f, -0.0529892412f);
-    r = fmaf(x2, r, 0.13324829f);
-    r = fmaf(x2, r, -0.333330719f);
-    return fmaf(x2, r, 0.999999987f);
-}
+constexpr double TANH_POLY[5] = {0.999999987, -0.333330719, 0.13324829, -0.0529892412, 0.017141319};
 __device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 // position of the first token of a portion: on the device (decode) or given by the host
