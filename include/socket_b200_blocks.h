@@ -155,7 +155,7 @@ SK_API int skb_latent_up(const void* o, int dtype, const void* uv, int64_t rows,
  * inputs conv_state [B, taps - 1, channels].  skb_ssm_scan: the recurrence on those rows,
  * state [B, H, N, P] fp32, y [B, S, H P] (with the skip D x).  Position 0 starts from zero state.
  * `path`: SKB_SSM_STEPS walks token by token, SKB_SSM_CHUNKS uses matrix products per block of tokens. */
-enum { SKB_SSM_AUTO = 0, SKB_SSM_STEPS = 1, SKB_SSM_CHUNKS = 2 };
+enum { SKB_SSM_AUTO = 0, SKB_SSM_STEPS = 1, SKB_SSM_CHUNKS = 2, SKB_SSM_TENSOR = 3 };
 typedef struct sk_ssm_params {
     const void *xbc_in, *dt_in, *conv_w, *conv_b;
     void *conv_state, *xbc, *y;
@@ -180,7 +180,8 @@ SK_API int skb_ssm_path(const sk_ssm_params* p);
  *   out = o / rms(o) * norm_w * sigmoid(z)              out rows [H P], out_ld apart
  * State: S [B, H, N, P], n [B, H, N], m [B, H], all fp32; position 0 starts from zero state and m = 0.
  * num [B S, H P] (of dtype), den [B S, H] and m_next [B, H] (fp32) are scratch.
- * `path`: SKB_SSM_STEPS walks token by token, SKB_SSM_CHUNKS uses matrix products per block of tokens. */
+ * `path`: SKB_SSM_STEPS walks token by token, SKB_SSM_CHUNKS uses warp-level matrix products per block of 64
+ * tokens, SKB_SSM_TENSOR tensor-memory ones per chunk of 128, all chunks of a portion side by side. */
 typedef struct sk_mlstm_params {
     const void *q, *k, *v, *z, *norm_w;
     const float *gates, *i_bias, *f_bias;
@@ -189,6 +190,7 @@ typedef struct sk_mlstm_params {
     float *den, *m_next;
     void* out;
     const int64_t* pos;
+    int32_t* status;
     void* workspace;
     size_t workspace_bytes;
     int64_t in_ld, gates_ld, out_ld, start;

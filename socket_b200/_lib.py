@@ -150,7 +150,7 @@ class MlstmParams(C.Structure):
     _fields_ = [
         ("q", _p), ("k", _p), ("v", _p), ("z", _p), ("norm_w", _p), ("gates", _p), ("i_bias", _p), ("f_bias", _p),
         ("S_state", _p), ("n_state", _p), ("m_state", _p), ("num", _p), ("den", _p), ("m_next", _p), ("out", _p),
-        ("pos", _p), ("workspace", _p), ("workspace_bytes", _sz), ("in_ld", _i64), ("gates_ld", _i64),
+        ("pos", _p), ("status", _p), ("workspace", _p), ("workspace_bytes", _sz), ("in_ld", _i64), ("gates_ld", _i64),
         ("out_ld", _i64), ("start", _i64), ("dtype", _i), ("B", _i), ("S", _i), ("H", _i), ("N", _i), ("P", _i),
         ("path", _i), ("cap", _f), ("q_scale", _f), ("eps", _f),
     ]

@@ -14,7 +14,7 @@ from ._lib import blocks, check_blocks, dtype_code, ptr, stream_ptr
 from .ops import _require_cuda
 
 ATTN_PATHS = {"auto": 0, "rows": 1, "prefill_tc": 2, "decode": 3}
-SSM_PATHS = {"auto": 0, "steps": 1, "chunks": 2}
+SSM_PATHS = {"auto": 0, "steps": 1, "chunks": 2, "tensor": 3}
 IN_NONE, IN_ADD_NORM, IN_REPLACE, IN_ADD = 0, 1, 2, 3
 OUT_NONE, OUT_NORM, OUT_CONCAT, OUT_LAYER_NORM = 0, 1, 2, 3
 GLU_CLAMPED, GLU_SILU = 0, 1
@@ -274,7 +274,7 @@ def ssm(proj: Tensor, inner: int, conv_w: Tensor, conv_b: Tensor, dt_bias: Tenso
 
 def mlstm(q: Tensor, k: Tensor, v: Tensor, z: Tensor, gates: Tensor, i_bias: Tensor, f_bias: Tensor, norm_w: Tensor,
           S_state: Tensor, n_state: Tensor, m_state: Tensor, out: Tensor, *, S: int, cap: float, q_scale: float, eps: float,
-          start: int = 0, pos: Optional[Tensor] = None, path: str = "auto") -> Tensor:
+          start: int = 0, pos: Optional[Tensor] = None, status: Optional[Tensor] = None, path: str = "auto") -> Tensor:
     """Matrix memory of B * S tokens: q, k [rows, H * N], v, z [rows, H * P] are slices of the same projection rows;
     gates [rows, >= 2 H] = [input | forget] fp32 before their biases.  S_state [B, H, N, P], n_state [B, H, N] and
     m_state [B, H] (fp32) are advanced by the portion; out [rows, H * P] (may be a slice) is normed per head and gated."""
@@ -295,6 +295,7 @@ def mlstm(q: Tensor, k: Tensor, v: Tensor, z: Tensor, gates: Tensor, i_bias: Ten
     p.q, p.k, p.v, p.z, p.norm_w, p.gates, p.i_bias, p.f_bias = (ptr(t) for t in (q, k, v, z, norm_w, gates, i_bias, f_bias))
     p.S_state, p.n_state, p.m_state, p.num, p.den, p.m_next, p.out = (ptr(t) for t in (S_state, n_state, m_state, num, den,
                                                                                        m_next, out))
+    p.status = ptr(status)
     p.pos, p.start, p.in_ld, p.gates_ld, p.out_ld = ptr(pos), start, q.stride(0), gates.stride(0), out.stride(0)
     p.dtype, p.B, p.S, p.H, p.N, p.P, p.path = dtype_code(q), B, S, H, N, P, SSM_PATHS[path]
     p.cap, p.q_scale, p.eps = float(cap), float(q_scale), float(eps)

@@ -29,7 +29,7 @@ FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-O3", "-lineinfo", "-std
          "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",
          "--expt-relaxed-constexpr"]
 LIBRARIES = {"step": LIB, "blocks": BLOCKS_LIB}
-BLOCK_SOURCES = ("abi_blocks", "attn_decode", "attn_prefill", "attn_rows", "latent", "mlstm",
+BLOCK_SOURCES = ("abi_blocks", "attn_decode", "attn_prefill", "attn_rows", "latent", "mlstm", "mlstm_tc",
                  "recurrence_chunks", "residual", "rotary_rows", "ssm")
 SHARED_SOURCES = ("host",)
 

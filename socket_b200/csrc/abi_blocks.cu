@@ -40,6 +40,7 @@ int check_ssm(const sk_ssm_params* p) {
     SK_REQUIRE(block_dtype(p->dtype), "skb_ssm: bad dtype");
     SK_REQUIRE(p->B > 0 && p->S > 0 && p->H > 0 && p->P > 0 && p->N > 0 && p->G > 0 && p->start >= 0,
                "skb_ssm: sizes must be positive");
+    SK_REQUIRE(p->path >= SKB_SSM_AUTO && p->path <= SKB_SSM_CHUNKS, "skb_ssm: unknown path %d", p->path);
     SK_REQUIRE(p->H % p->G == 0, "skb_ssm: %d heads are not a multiple of %d groups", p->H, p->G);
     SK_REQUIRE(p->xbc_ld >= p->H * p->P + 2 * p->G * p->N, "skb_ssm: row stride smaller than row");
     return SK_OK;
@@ -64,7 +65,13 @@ int check_mlstm(const sk_mlstm_params* p) {
 
 int mlstm_path(const sk_mlstm_params& p) {
     if (p.path != SKB_SSM_AUTO) return p.path;
+    if (p.S >= 256 && mlstm_tc_applicable(p)) return SKB_SSM_TENSOR;
     return p.S >= 16 && mlstm_chunks_applicable(p) ? SKB_SSM_CHUNKS : SKB_SSM_STEPS;
+}
+
+size_t mlstm_workspace(const sk_mlstm_params& p) {
+    const int path = mlstm_path(p);
+    return path == SKB_SSM_TENSOR ? mlstm_tc_workspace(p) : path == SKB_SSM_CHUNKS ? mlstm_chunks_workspace(p) : 0;
 }
 
 }  // namespace
@@ -198,7 +205,7 @@ int skb_ssm_scan(const sk_ssm_params* p, void* stream) {
 }
 
 size_t skb_mlstm_workspace_bytes(const sk_mlstm_params* p) {
-    return p != nullptr && mlstm_path(*p) == SKB_SSM_CHUNKS ? mlstm_chunks_workspace(*p) : 0;
+    return p != nullptr ? mlstm_workspace(*p) : 0;
 }
 
 int skb_mlstm_path(const sk_mlstm_params* p) { return p != nullptr ? mlstm_path(*p) : SKB_SSM_STEPS; }
@@ -206,16 +213,14 @@ int skb_mlstm_path(const sk_mlstm_params* p) { return p != nullptr ? mlstm_path(
 int skb_mlstm(const sk_mlstm_params* p, void* stream) {
     if (int rc = check_mlstm(p)) return rc;
     const cudaStream_t st = (cudaStream_t)stream;
-    if (mlstm_path(*p) == SKB_SSM_CHUNKS) {
-        if (!mlstm_chunks_applicable(*p)) return fail(SK_ERR_UNSUPPORTED, "skb_mlstm: shape outside the block kernel");
-        if (p->workspace == nullptr || p->workspace_bytes < mlstm_chunks_workspace(*p))
-            return fail(SK_ERR_WORKSPACE, "skb_mlstm: workspace of %zu bytes needed, %zu given", mlstm_chunks_workspace(*p),
-                        p->workspace_bytes);
-        if (int rc = launch_mlstm_chunks(*p, st)) return rc;
-    } else if (int rc = launch_mlstm_steps(*p, st)) {
-        return rc;
-    }
-    return launch_mlstm_finish(*p, st);
+    const int path = mlstm_path(*p);
+    if (path == SKB_SSM_CHUNKS ? !mlstm_chunks_applicable(*p) : path == SKB_SSM_TENSOR && !mlstm_tc_applicable(*p))
+        return fail(SK_ERR_UNSUPPORTED, "skb_mlstm: shape outside the block kernels");
+    if (mlstm_workspace(*p) > 0 && (p->workspace == nullptr || p->workspace_bytes < mlstm_workspace(*p)))
+        return fail(SK_ERR_WORKSPACE, "skb_mlstm: workspace of %zu bytes needed, %zu given", mlstm_workspace(*p), p->workspace_bytes);
+    const int rc = path == SKB_SSM_TENSOR ? launch_mlstm_tc(*p, st) : path == SKB_SSM_CHUNKS ? launch_mlstm_chunks(*p, st)
+                                                                                            : launch_mlstm_steps(*p, st);
+    return rc != SK_OK ? rc : launch_mlstm_finish(*p, st);
 }
 
 int skb_gated_group_norm(const void* y, const void* z, int64_t z_ld, const void* w, int dtype, int64_t rows, int inner,

@@ -124,6 +124,9 @@ int launch_gated_group_norm(const void* y, const void* z, int64_t z_ld, const vo
 bool mlstm_chunks_applicable(const sk_mlstm_params& p);
 size_t mlstm_chunks_workspace(const sk_mlstm_params& p);
 int launch_mlstm_chunks(const sk_mlstm_params& p, cudaStream_t st);
+bool mlstm_tc_applicable(const sk_mlstm_params& p);
+size_t mlstm_tc_workspace(const sk_mlstm_params& p);
+int launch_mlstm_tc(const sk_mlstm_params& p, cudaStream_t st);
 int launch_mlstm_steps(const sk_mlstm_params& p, cudaStream_t st);
 int launch_mlstm_finish(const sk_mlstm_params& p, cudaStream_t st);
 

@@ -24,13 +24,6 @@ constexpr int SC_TOK = 64, SC_P = 32, SC_THR = 256;
 constexpr int SC_PS = SC_P + 8;              // shared-memory row of 32 columns
 constexpr float SC_LOG2E = 1.4426950408889634f;
 
-__device__ __forceinline__ void split_bf16(float x, float y, uint32_t& hi, uint32_t& lo) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-    const __nv_bfloat162 r = __floats2bfloat162_rn(x - __low2float(h), y - __high2float(h));
-    hi = *reinterpret_cast<const uint32_t*>(&h);
-    lo = *reinterpret_cast<const uint32_t*>(&r);
-}
-
 // dt[b][h][t] = softplus(step column + bias), cum[b][h][t] = running sum of -exp(A_log) dt log2(e) inside t's block;
 // tokens past the portion's end get dt = 0 and leave the sum as it is.  A CTA: 64 tokens of 32 heads.
 __global__ void __launch_bounds__(256)

@@ -189,6 +189,7 @@ __host__ __device__ constexpr uint32_t umma_idesc_bf16(int n, bool b_mn_major) {
     return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn_major ? 1u << 16 : 0u) | ((uint32_t)(n >> 3) << 17) |
            ((128u >> 4) << 24);
 }
+constexpr uint32_t UMMA_A_MN = 1u << 15;             // the K index of A runs over the rows, as b_mn_major says of B
 // D (tensor memory) (+)= A (shared memory) B (shared memory)
 __device__ __forceinline__ void umma_ss(uint32_t tmem_d, uint64_t da, uint64_t db, uint32_t idesc, uint32_t accumulate) {
     asm volatile(

@@ -351,7 +351,8 @@ class MatrixMemory(nn.Module):
     def mix(self, parts: List[Tensor], h: Tensor, cache: MemoryState, at: Portion, out: Tensor) -> None:
         B = at.B
         ops.mlstm(*parts, matmul_f32(h, self.w_gates), self.i_b_f32, self.f_b_f32, self.norm_w, cache.S[:B], cache.n[:B],
-                  cache.m[:B], out, S=at.S, cap=self.cap, q_scale=self.N ** -0.5, eps=self.eps, start=at.start, pos=at.pos)
+                  cache.m[:B], out, S=at.S, cap=self.cap, q_scale=self.N ** -0.5, eps=self.eps, start=at.start, pos=at.pos,
+                  status=at.status)
 
 
 # ---------------------------------------------------------------------------------- state space

@@ -349,14 +349,15 @@ def _plain_memory(c, proj, cols, gates, bias, norm, B, S, eps, dtype=D64):
 
 def _run_memory(c, part, cols, gates, bias, norm, state, n, eps, path, **kw):
     out = torch.full((part.shape[0], norm.numel() + 8), 7.0, dtype=part.dtype, device=DEV)
+    status = torch.zeros(1, dtype=torch.int32, device=DEV)
     ops.mlstm(*(part[:, s] for s in cols), gates, *(b.to(DEV) for b in bias), norm.to(DEV), *state, out[:, 8:], S=n, cap=c["cap"],
-              q_scale=c["N"] ** -0.5, eps=eps, path=path, **kw)
-    assert (out[:, :8] == 7).all()
+              q_scale=c["N"] ** -0.5, eps=eps, path=path, status=status, **kw)
+    assert (out[:, :8] == 7).all() and int(status) == 0
     return out[:, 8:]
 
 
 @pytest.mark.parametrize("case", range(len(MEM)))
-@pytest.mark.parametrize("path", ["steps32", "steps", "chunks"])
+@pytest.mark.parametrize("path", ["steps32", "steps", "chunks", "tensor"])
 def test_matrix_memory_in_portions(case, path):
     """One long portion, and the same tokens in portions of all kinds of sizes (also single tokens by a position on
     the device): the same outputs, the same final state; dirty state is not seen at position 0."""
@@ -364,12 +365,12 @@ def test_matrix_memory_in_portions(case, path):
     dtype = F32 if path == "steps32" else BF16
     path = "steps" if path == "steps32" else path
     H, N, P = c["H"], c["N"], c["P"]
-    if path == "chunks" and (N % 8 or P % 8):
+    if path in ("chunks", "tensor") and (N % 8 or P % 8):
         pytest.skip("sizes of the step kernel only")
     proj, cols, gates, bias, norm = _memory_inputs(c, B, S, dtype)
     want, want_st = _plain_memory(c, proj, cols, gates, bias, norm, B, S, eps)
     pg, gg = proj.to(DEV).view(B, S, -1), gates.to(DEV).view(B, S, -1)
-    for sizes in ([S], [1, 2, 2, 59, 64, 1, 65, 16], [64, 128, 3, 15], [2] * 105):
+    for sizes in ([S], [1, 2, 2, 59, 64, 1, 65, 16], [64, 128, 3, 15], [128, 82], [2] * 105):
         state = [torch.full(s, 3.0, device=DEV) for s in ((B, H, N, P), (B, H, N), (B, H))]
         out, at = [], 0
         for n in sizes:
@@ -384,14 +385,15 @@ def test_matrix_memory_in_portions(case, path):
             _close(got.view(w.shape), w, dtype, tol16=1e-4, tol32=1e-5)
 
 
-def test_block_form_keeps_more_than_bf16():
-    """With the same bf16 inputs the block form and the token-by-token fp32 form differ by far less than the
+@pytest.mark.parametrize("form", ["chunks", "tensor"])
+def test_block_forms_keep_more_than_bf16(form):
+    """With the same bf16 inputs the block forms and the token-by-token fp32 form differ by far less than the
     output's own rounding; a slowly forgetting head over a long portion included."""
     c, B, S, eps = dict(H=2, N=64, P=32, cap=15.0), 1, 1000, 1e-5
     proj, cols, gates, bias, norm = _memory_inputs(c, B, S, BF16, seed=9)
     bias[1] = torch.tensor([12.0, 0.0])
     states, outs = [], []
-    for path in ("steps", "chunks"):
+    for path in ("steps", form):
         st = [torch.zeros(s, device=DEV) for s in ((1, 2, 64, 32), (1, 2, 64), (1, 2))]
         outs.append(_run_memory(c, proj.to(DEV), cols, gates.to(DEV), bias, norm, st, S, eps, path).float())
         states.append(st)
@@ -400,7 +402,7 @@ def test_block_form_keeps_more_than_bf16():
     assert (outs[0] - outs[1]).abs().max() <= 1e-2 * outs[0].abs().max()
 
 
-@pytest.mark.parametrize("path", ["steps32", "chunks"])
+@pytest.mark.parametrize("path", ["steps32", "chunks", "tensor"])
 def test_gates_at_their_extremes(path):
     """The running maximum: a strong input gate long ago that fades slowly, gates closed from the start (m stays at
     or below zero and the floor exp(-m) rules), a jump inside a block, values of the floor and of |n . q| both
@@ -435,6 +437,30 @@ def test_gates_at_their_extremes(path):
             assert err.max() <= limit + 4 * rounding[:, s].max() and err.median() <= limit, (h, float(err.max()), top)
         for a, b, r in zip(state, want_st, st_rounding):
             assert (a.cpu().to(D64).view(b.shape) - b).abs().max() <= (1e-4 if dtype == BF16 else 1e-5) * b.abs().max() + 4 * r
+
+
+@pytest.mark.parametrize("S", [255, 256, 700])
+def test_long_portions_take_the_tensor_form_and_go_on_from_any_state(S):
+    import ctypes
+
+    from socket_b200 import _lib
+    from socket_b200._lib import blocks
+    c, B, eps = dict(H=3, N=72, P=136, cap=10.0), 2, 1e-5
+    p = _lib.MlstmParams()
+    p.dtype, p.B, p.S, p.H, p.N, p.P, p.in_ld = _lib.SK_BF16, B, S, 3, 72, 136, 2 * 3 * (72 + 136)
+    assert blocks().skb_mlstm_path(ctypes.byref(p)) == ops.SSM_PATHS["tensor" if S >= 256 else "chunks"]
+    proj, cols, gates, bias, norm = _memory_inputs(c, B, S + 40, BF16, seed=6)
+    want, want_st = _plain_memory(c, proj, cols, gates, bias, norm, B, S + 40, eps)
+    state = [torch.full(s, -2.0, device=DEV) for s in ((B, 3, 72, 136), (B, 3, 72), (B, 3))]
+    pg, gg = proj.to(DEV).view(B, S + 40, -1), gates.to(DEV).view(B, S + 40, -1)
+    out = []
+    for a, b in ((0, 30), (30, S + 30), (S + 30, S + 40)):
+        y = _run_memory(c, pg[:, a:b].reshape(B * (b - a), -1), cols, gg[:, a:b].reshape(B * (b - a), -1), bias, norm, state, b - a, eps,
+                        "auto", start=a)
+        out.append(y.view(B, b - a, -1))
+    _close(torch.cat(out, 1).reshape(want.shape), want, BF16)
+    for got, w in zip(state, want_st):
+        _close(got.view(w.shape), w, BF16, tol16=1e-4)
 
 
 def test_a_memory_larger_than_the_block_form_takes():
