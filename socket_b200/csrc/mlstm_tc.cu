@@ -160,10 +160,11 @@ mlstm_tc_carry_kernel(const __grid_constant__ MtShape p) {
 // ---------------------------------------------------------------- states
 constexpr int ST_P = 64;                                      // value columns of a CTA; 128 key columns
 constexpr int ST_THREADS = 288;                               // warps 0-3: tensor memory; 4-7: weighted values; 8: TMA and MMA
-constexpr uint32_t ST_SMEM = 2 * 2 * MT_PANEL + 2 * 2 * MT_PANEL + 2 * MT_PANEL + 1024;
+constexpr int ST_KSTAGES = 4;                                 // chunks of K in flight
+constexpr uint32_t ST_SMEM = (ST_KSTAGES + 2 + 1) * 2 * MT_PANEL + 1024;   // K; two stages of weighted V; the outgoing state
 
 struct StShared {
-    uint64_t k_full[2], v_full[2], v_empty[2], s_ready, mma_done, drained;
+    uint64_t k_full[ST_KSTAGES], v_full[2], v_empty[2], s_ready, mma_done, drained;
     uint32_t tmem_base;
     int failed;
 };
@@ -195,15 +196,15 @@ mlstm_tc_states_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     extern __shared__ char st_raw[];
     __shared__ StShared sh;
     char* k_s = reinterpret_cast<char*>((reinterpret_cast<uintptr_t>(st_raw) + 1023) & ~(uintptr_t)1023);   // [stage][panel]
-    char* v_s = k_s + 2 * 2 * MT_PANEL;                       // [stage][value, remainder]
+    char* v_s = k_s + ST_KSTAGES * 2 * MT_PANEL;              // [stage][value, remainder]
     char* o_s = v_s + 2 * 2 * MT_PANEL;                       // [value, remainder]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int p0 = blockIdx.x * ST_P, n0 = blockIdx.y * 128, b = blockIdx.z / p.H, h = blockIdx.z - b * p.H;
     const int64_t head = (int64_t)b * p.H + h;
     volatile int* failed = &sh.failed;
     if (tid == 0) {
+        for (int s = 0; s < ST_KSTAGES; ++s) mbar_init_count(&sh.k_full[s], 1);
         for (int s = 0; s < 2; ++s) {
-            mbar_init_count(&sh.k_full[s], 1);
             mbar_init_count(&sh.v_full[s], 4);
             mbar_init_count(&sh.v_empty[s], 1);
         }
@@ -306,33 +307,40 @@ mlstm_tc_states_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         const bool live_col = p0 + piece * 8 < p.P;
         const __nv_bfloat16* v = p.v + (int64_t)b * p.S * p.in_ld + (int64_t)h * p.P + p0 + piece * 8;
         const float* a = p.a + head * p.chunks * MT_TOK;
-        uint4 raw[8];
-        float e[8], mi, tp;
-        auto load = [&](int c) {
+        // a chunk's values are requested two chunks ahead
+        uint4 raw[2][8];
+        float e[2][8], mi[2], tp[2];
+        auto load = [&](int c, uint4 (&r)[8], float (&x)[8], float& m, float& t) {
 #pragma unroll
             for (int it = 0; it < 8; ++it) {
                 const int s = it * 16 + vw * 4 + (lane >> 3), tok = c * MT_TOK + s;
-                raw[it] = live_col && tok < p.S ? __ldg(reinterpret_cast<const uint4*>(v + (int64_t)tok * p.in_ld)) : make_uint4(0, 0, 0, 0);
-                e[it] = a[(int64_t)c * MT_TOK + s];
+                r[it] = live_col && tok < p.S ? __ldg(reinterpret_cast<const uint4*>(v + (int64_t)tok * p.in_ld)) : make_uint4(0, 0, 0, 0);
+                x[it] = a[(int64_t)c * MT_TOK + s];
             }
-            mi = m_in[c];
-            tp = top_end[(int64_t)c * MT_TOK];
+            m = m_in[c];
+            t = top_end[(int64_t)c * MT_TOK];
         };
-        load(0);
-        for (int c = 0; c < p.chunks; ++c) {
-            const int stage = c & 1;
+        load(0, raw[0], e[0], mi[0], tp[0]);
+        if (p.chunks > 1) load(1, raw[1], e[1], mi[1], tp[1]);
+        bool ok = true;
+        for (int c2 = 0; ok && c2 < p.chunks; c2 += 2)
+#pragma unroll
+        for (int stage = 0; stage < 2; ++stage) {
+            const int c = c2 + stage;
+            if (c >= p.chunks) break;
             if (c >= 2 && (__any_sync(FULL, *failed != 0) ||
                            !__all_sync(FULL, mbar_wait_bounded(&sh.v_empty[stage], (uint32_t)(((c >> 1) - 1) & 1))))) {
                 *failed = 1;
+                ok = false;
                 break;
             }
-            const float mm = fmaxf(mi, tp);
+            const float mm = fmaxf(mi[stage], tp[stage]);
             char* dst = v_s + stage * 2 * MT_PANEL;
 #pragma unroll
             for (int it = 0; it < 8; ++it) {
                 const int s = it * 16 + vw * 4 + (lane >> 3);
-                const float w = exp2f(e[it] - mm);
-                const uint32_t q[4] = {raw[it].x, raw[it].y, raw[it].z, raw[it].w};
+                const float w = exp2_fast(e[stage][it] - mm);
+                const uint32_t q[4] = {raw[stage][it].x, raw[stage][it].y, raw[stage][it].z, raw[stage][it].w};
                 float x[8];
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
@@ -348,47 +356,41 @@ mlstm_tc_states_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
             asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
             __syncwarp();
             if (lane == 0) mbar_arrive(&sh.v_full[stage]);
-            if (c + 1 < p.chunks) load(c + 1);
+            if (c + 2 < p.chunks) load(c + 2, raw[stage], e[stage], mi[stage], tp[stage]);
         }
     } else if (lane == 0) {
         // ---- K by TMA, MMAs: S += K^T (weighted V)
         auto fetch = [&](int c) {
-            char* dst = k_s + (c & 1) * 2 * MT_PANEL;
-            mbar_expect(&sh.k_full[c & 1], 2 * MT_PANEL);
-            for (int q = 0; q < 2; ++q) tma_load_4d(dst + q * MT_PANEL, &map_k, n0 + q * 64, h, c * MT_TOK, b, &sh.k_full[c & 1]);
+            const int s = c % ST_KSTAGES;
+            char* dst = k_s + s * 2 * MT_PANEL;
+            mbar_expect(&sh.k_full[s], 2 * MT_PANEL);
+            for (int q = 0; q < 2; ++q) tma_load_4d(dst + q * MT_PANEL, &map_k, n0 + q * 64, h, c * MT_TOK, b, &sh.k_full[s]);
         };
         const uint32_t idesc = umma_idesc_bf16(ST_P, true) | UMMA_A_MN;
         const uint32_t ka = smem_addr(k_s), va = smem_addr(v_s);
-        int sent = 1;
-        fetch(0);
-        if (p.chunks > 1) {
-            fetch(1);
-            sent = 2;
-        }
+        int sent = 0;
+        for (; sent < p.chunks && sent < ST_KSTAGES; ++sent) fetch(sent);
         bool ok = true;
         int c = 0;
         for (; c < p.chunks && !*failed; ++c) {
             const int stage = c & 1;
             ok = mbar_wait_bounded(&sh.s_ready, (uint32_t)(c & 1));           // which follows the MMAs of chunk c - 1
             if (!ok) break;
-            if (c >= 1 && c + 1 < p.chunks) {
-                fetch(c + 1);
-                sent = c + 2;
-            }
-            ok = mbar_wait_bounded(&sh.k_full[stage], (uint32_t)((c >> 1) & 1)) &&
+            if (c >= 1 && sent < p.chunks) fetch(sent++);                     // into the stage chunk c - 1 has left
+            ok = mbar_wait_bounded(&sh.k_full[c % ST_KSTAGES], (uint32_t)((c / ST_KSTAGES) & 1)) &&
                  mbar_wait_bounded(&sh.v_full[stage], (uint32_t)((c >> 1) & 1));
             if (!ok) break;
             tc_fence_after();
             for (int part = 0; part < 2; ++part)
                 for (int k = 0; k < MT_TOK / 16; ++k)
-                    umma_ss(tmem, umma_desc_sw128_mn(ka + stage * 2 * MT_PANEL + k * 2048, MT_PANEL),
+                    umma_ss(tmem, umma_desc_sw128_mn(ka + (c % ST_KSTAGES) * 2 * MT_PANEL + k * 2048, MT_PANEL),
                             umma_desc_sw128_mn(va + (stage * 2 + part) * MT_PANEL + k * 2048, MT_PANEL), idesc, 1);
             umma_commit(&sh.mma_done);
             umma_commit(&sh.v_empty[stage]);
         }
         if (!ok) *failed = 1;
         if (c < p.chunks)                                     // left early: no copy stays in flight
-            for (int q = c; q < sent; ++q) mbar_wait_bounded(&sh.k_full[q & 1], (uint32_t)((q >> 1) & 1));
+            for (int q = c; q < sent; ++q) mbar_wait_bounded(&sh.k_full[q % ST_KSTAGES], (uint32_t)((q / ST_KSTAGES) & 1));
         umma_commit(&sh.drained);
         mbar_wait_bounded(&sh.drained, 0);
     }
