@@ -205,4 +205,10 @@ def random_weights(cfg: dict, seed: int) -> Dict[str, Tensor]:
         else:
             x = x / shape[-1] ** 0.5
         out[name] = x.to(torch.bfloat16)
+    # a query almost orthogonal to the only key of a memory (the first token's, say) has an output whose sign is
+    # rounding's; keys that lean towards their queries keep outputs well-conditioned
+    for i, e in enumerate(cfg["layers"]):
+        if e["type"] == "mlstm" and e.get("weights_of") is None:
+            k = out[f"l{i}.mix.k"].float() + out[f"l{i}.mix.q"].float()
+            out[f"l{i}.mix.k"] = (k / 2 ** 0.5).to(torch.bfloat16)
     return out

@@ -98,6 +98,27 @@ def test_portions_and_token_by_token_decoding(name, dtype):
     assert m.device_flags() == 0
 
 
+@pytest.mark.parametrize("dtype", [F32, BF16])
+def test_long_prompts(dtype):
+    """Portions long enough for every form of the recurrence, one after the other, and decoding after them."""
+    name = "wide"
+    m = _model(name, dtype)
+    tok = _tokens(name, 420, seed=11)
+    want = _want(name, tok)
+    m.setup_caches(1, 424)
+    m.setup_decode(1)
+    for sizes in ([420], [300, 100], [7, 260, 20, 3], [129, 256]):
+        rows, at = [], 0
+        for n in sizes:
+            rows.append(m.forward_portion(_idx(tok[at:at + n]), at, range(n))[0])
+            at += n
+        while at < len(tok):
+            rows.append(m.decode_given_token(_idx(tok[at:at + 1]), at).clone())
+            at += 1
+        _check(torch.cat(rows), want, dtype)
+    assert m.device_flags() == 0
+
+
 @pytest.mark.parametrize("name", ["shared", "odd", "wide"])
 def test_decoding_from_the_first_token_on(name):
     """Long decoding without any prompt: position 0 itself through the decode step, several rounds of every ring."""
