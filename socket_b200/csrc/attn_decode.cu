@@ -13,6 +13,8 @@
 #include "tensor_map.cuh"
 #include "warp_mma.cuh"
 
+#include <type_traits>
+
 namespace sk {
 namespace {
 
@@ -101,13 +103,13 @@ __device__ __forceinline__ DmRow dm_row(const sk_attn_params& p, const DmRange& 
     r.hi = !live ? -1 : rg.wrap ? rg.hi : (int)min(r.origin, (int64_t)rg.hi);      // an absent row sees nothing
     return r;
 }
-// scaled score in log2 units, without bias
-__device__ __forceinline__ float dm_score(const sk_attn_params& p, float dot) {
-    return p.softcap > 0.f ? p.softcap * DM_LOG2E * tanh_exp2(dot * (p.scale / p.softcap)) : dot * (p.scale * DM_LOG2E);
+// scaled score in log2 units, without bias: in, out = scale / softcap, softcap under a cap, else out = scale
+template <bool CAP> __device__ __forceinline__ float dm_score(float dot, float in, float out) {
+    return CAP ? out * tanh_exp2(dot * in) : dot * out;
 }
 
 // Up to 16 query rows: a warp computes the scores of 8 keys of a tile.  NVT: 8-column value tiles per warp
-template <int NVT>
+template <int NVT, bool CAP>
 __global__ void __launch_bounds__(DM_WARPS * 32)
 attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const __grid_constant__ sk_attn_params p,
                    int splits, int groups, int np, int nvp, int k_off, int q_stride, size_t part_floats) {
@@ -170,6 +172,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
         see[k] = dm_row(p, rg, s, row < n_rows);
         brow[k] = p.bias != nullptr && row < n_rows ? p.bias + (int64_t)(g * rep + row - s * rep) * p.bias_len : nullptr;
     }
+    const float cap_in = CAP ? p.scale / p.softcap : 0.f, sl = (CAP ? p.softcap : p.scale) * DM_LOG2E;
     float m_own[2] = {-INFINITY, -INFINITY}, l_own[2] = {0.f, 0.f};
     float acc[NVT][4];
 #pragma unroll
@@ -194,30 +197,37 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
         const uint32_t qa = saddr(qs + ((lane & 15)) * q_stride + (lane >> 4) * 8);
         const uint32_t ka = saddr(ks + stage * np * DM_PANEL + (kg * 8 + (lane & 7)) * 128);
         const int sw = lane & 7, kp = k_off / 8;                // the keys begin at 16-byte piece kp of a row
-        int kk = 0;
+        auto dot = [&](auto shifted) {                          // keys that begin a row: panels and pieces by kk alone
+            auto piece = [&](int kk, int i) {
+                const int c = kk * 2 + i + (shifted.value ? kp : 0);
+                return shifted.value ? ka + (c >> 3) * DM_PANEL + (((c & 7) ^ sw) << 4)
+                                     : ka + (kk >> 2) * DM_PANEL + ((((kk & 3) * 2 + i) ^ sw) << 4);
+            };
+            int kk = 0;
 #pragma unroll 4
-        for (; kk + 2 <= k16; kk += 2) {                        // 32 head dimensions at a time
-            uint32_t a0[4], a1[4], bb[4];
-            const int c = kk * 2 + (lane >> 3) + kp;
-            ldsm4(ka + (c >> 3) * DM_PANEL + (((c & 7) ^ sw) << 4), bb);
-            ldsm4(qa + kk * 32, a0);
-            ldsm4(qa + kk * 32 + 32, a1);
-            mma16816(sc[0], a0, bb[0], bb[1]);
-            mma16816(sc[1], a1, bb[2], bb[3]);
-        }
-        if (kk < k16) {
-            uint32_t a0[4], b0, b1;
-            const int c = kk * 2 + ((lane >> 3) & 1) + kp;
-            ldsm2(ka + (c >> 3) * DM_PANEL + (((c & 7) ^ sw) << 4), b0, b1);
-            ldsm4(qa + kk * 32, a0);
-            mma16816(sc[0], a0, b0, b1);
-        }
+            for (; kk + 2 <= k16; kk += 2) {                    // 32 head dimensions at a time
+                uint32_t a0[4], a1[4], bb[4];
+                ldsm4(piece(kk, lane >> 3), bb);
+                ldsm4(qa + kk * 32, a0);
+                ldsm4(qa + kk * 32 + 32, a1);
+                mma16816(sc[0], a0, bb[0], bb[1]);
+                mma16816(sc[1], a1, bb[2], bb[3]);
+            }
+            if (kk < k16) {
+                uint32_t a0[4], b0, b1;
+                ldsm2(piece(kk, (lane >> 3) & 1), b0, b1);
+                ldsm4(qa + kk * 32, a0);
+                mma16816(sc[0], a0, b0, b1);
+            }
+        };
+        if (kp == 0) dot(std::false_type{});
+        else dot(std::true_type{});
         const int r0 = rg.lo + t * DM_KEYS + kg * 8;            // key row of column 0 of this warp
         float mt[2] = {-INFINITY, -INFINITY};
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const int k = e >> 1, r = r0 + fc + (e & 1);
-            float v = dm_score(p, sc[0][e] + sc[1][e]);
+            float v = dm_score<CAP>(sc[0][e] + sc[1][e], cap_in, sl);
             if (r >= see[k].lo && r <= see[k].hi) {
                 if (brow[k] != nullptr) {
                     int64_t d = see[k].origin - r;
@@ -322,7 +332,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
 // registers and no key is read from shared memory twice; the partial scores meet in shared memory, where eight
 // lanes own a row: they sum, mask, keep its maximum and sum of weights, and write the weights for P V.
 // KS: 16-column steps of the head dimension per warp, NVT: 8-column value tiles per warp
-template <int KS, int NVT>
+template <int KS, int NVT, bool CAP>
 __global__ void __launch_bounds__(DM_WARPS * 32)
 attn_decode_wide_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                         const __grid_constant__ sk_attn_params p, int splits, int groups, int np, int nvp, int k_off, size_t part_floats) {
@@ -382,6 +392,7 @@ attn_decode_wide_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     const bool live_row = own_row < n_rows;
     const DmRow see = dm_row(p, rg, own_s, live_row);
     const float* brow = p.bias != nullptr && live_row ? p.bias + (int64_t)(g * rep + own_row - own_s * rep) * p.bias_len : nullptr;
+    const float cap_in = CAP ? p.scale / p.softcap : 0.f, sl = (CAP ? p.softcap : p.scale) * DM_LOG2E;
     float m = -INFINITY, l = 0.f;
     float acc[2][NVT][4];
 #pragma unroll
@@ -461,7 +472,7 @@ attn_decode_wide_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 #pragma unroll
             for (int e = 0; e < 8; ++e) {
                 const int r = rg.lo + t * DM_KEYS + (e >> 2) * 32 + (lane & 7) * 4 + (e & 3);
-                float x = dm_score(p, v[e]);
+                float x = dm_score<CAP>(v[e], cap_in, sl);
                 if (r >= see.lo && r <= see.hi) {
                     if (brow != nullptr) {
                         int64_t d = see.origin - r;
@@ -633,6 +644,35 @@ attn_decode_merge_kernel(sk_attn_params p, int splits, int groups, int rows_per_
     }
 }
 
+template <bool CAP>
+int launch_splits(const sk_attn_params& p, const DmPlan& d, const CUtensorMap& mk, const CUtensorMap& mv, dim3 grid, cudaStream_t st) {
+#define SK_DM(kernel, ...)                                                                                               \
+    do {                                                                                                                 \
+        auto kern = kernel;                                                                                              \
+        const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)d.smem);      \
+        if (e != cudaSuccess) return fail(SK_ERR_CUDA, "attn_decode kernel smem attribute: %s", cudaGetErrorString(e));  \
+        kern<<<grid, DM_WARPS * 32, d.smem, st>>>(mk, mv, p, d.splits, d.groups, d.np, d.nvp, d.k_off, __VA_ARGS__);     \
+    } while (0)
+#define SK_DM_WIDE(KS)                                                                                    \
+    do {                                                                                                  \
+        if (d.nvt == 2) SK_DM((attn_decode_wide_kernel<KS, 2, CAP>), d.part_floats);                           \
+        else if (d.nvt == 4) SK_DM((attn_decode_wide_kernel<KS, 4, CAP>), d.part_floats);                      \
+        else SK_DM((attn_decode_wide_kernel<KS, 8, CAP>), d.part_floats);                                      \
+    } while (0)
+    if (d.mt == 1) {
+        if (d.nvt == 2) SK_DM((attn_decode_kernel<2, CAP>), d.q_stride, d.part_floats);
+        else if (d.nvt == 4) SK_DM((attn_decode_kernel<4, CAP>), d.q_stride, d.part_floats);
+        else SK_DM((attn_decode_kernel<8, CAP>), d.q_stride, d.part_floats);
+    } else if (p.dqk <= 256) {
+        SK_DM_WIDE(4);
+    } else {
+        SK_DM_WIDE(10);
+    }
+#undef SK_DM_WIDE
+#undef SK_DM
+    return check_launch("attn_decode_kernel");
+}
+
 }  // namespace
 
 bool attn_decode_mma_applicable(const sk_attn_params& p) {
@@ -654,31 +694,8 @@ int launch_attn_decode_mma(const sk_attn_params& p, cudaStream_t st) {
     if (int rc = make_head_map(&mk, d.shared_v ? p.v : p.k, d.k_off + p.dqk, p.G, p.kv_rows, p.B, p.k_hs, p.k_ts, p.k_bs, DM_KEYS)) return rc;
     if (int rc = make_head_map(&mv, p.v, p.dv, p.G, p.kv_rows, p.B, p.v_hs, p.v_ts, p.v_bs, DM_KEYS)) return rc;
     dim3 grid((unsigned)d.splits, (unsigned)(p.G * d.groups), (unsigned)p.B);
-#define SK_DM(kernel, ...)                                                                                               \
-    do {                                                                                                                 \
-        auto kern = kernel;                                                                                              \
-        const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)d.smem);      \
-        if (e != cudaSuccess) return fail(SK_ERR_CUDA, "attn_decode kernel smem attribute: %s", cudaGetErrorString(e));  \
-        kern<<<grid, DM_WARPS * 32, d.smem, st>>>(mk, mv, p, d.splits, d.groups, d.np, d.nvp, d.k_off, __VA_ARGS__);     \
-    } while (0)
-#define SK_DM_WIDE(KS)                                                                                    \
-    do {                                                                                                  \
-        if (d.nvt == 2) SK_DM((attn_decode_wide_kernel<KS, 2>), d.part_floats);                           \
-        else if (d.nvt == 4) SK_DM((attn_decode_wide_kernel<KS, 4>), d.part_floats);                      \
-        else SK_DM((attn_decode_wide_kernel<KS, 8>), d.part_floats);                                      \
-    } while (0)
-    if (d.mt == 1) {
-        if (d.nvt == 2) SK_DM((attn_decode_kernel<2>), d.q_stride, d.part_floats);
-        else if (d.nvt == 4) SK_DM((attn_decode_kernel<4>), d.q_stride, d.part_floats);
-        else SK_DM((attn_decode_kernel<8>), d.q_stride, d.part_floats);
-    } else if (p.dqk <= 256) {
-        SK_DM_WIDE(4);
-    } else {
-        SK_DM_WIDE(10);
-    }
-#undef SK_DM_WIDE
-#undef SK_DM
-    if (int rc = check_launch("attn_decode_kernel")) return rc;
+    const int rc_split = p.softcap > 0.f ? launch_splits<true>(p, d, mk, mv, grid, st) : launch_splits<false>(p, d, mk, mv, grid, st);
+    if (rc_split != SK_OK) return rc_split;
     const int col_blocks = (p.dv + DG_COLS - 1) / DG_COLS;
     const cudaError_t e = launch_after(attn_decode_merge_kernel, dim3((unsigned)(p.S * (p.H / p.G) * col_blocks), (unsigned)p.G, (unsigned)p.B),
                                        dim3(DG_WARPS * 32), 0, st, p, d.splits, d.groups, 16 * d.mt, d.part_floats, col_blocks);

@@ -105,7 +105,7 @@ struct RecurrenceParams {
     const float *m_state, *skip;
     const float *e0, *e1, *e2;               // [B, H, blocks, 64]: running decay, step size | a, its running maximum, b
     const int64_t* pos;
-    int64_t q_ld, k_ld, v_ld, start;
+    int64_t ld, start;                       // elements between tokens in q, k and v
     int S, H, P, N, rep, ns, blocks;
     float q_scale;
 };
@@ -134,9 +134,9 @@ recurrence_chunks_kernel(const __grid_constant__ RecurrenceParams p) {
     const int64_t head = (int64_t)b * p.H + h;
     const float skip = MEMORY ? 0.f : p.skip[h];
     float m_in = MEMORY && !fresh ? p.m_state[head] * SC_LOG2E : 0.f;
-    const bf* q_rows = p.q + (int64_t)b * p.S * p.q_ld + (int64_t)g * p.N;
-    const bf* k_rows = p.k + (int64_t)b * p.S * p.k_ld + (int64_t)g * p.N;
-    const bf* v_rows = p.v + (int64_t)b * p.S * p.v_ld + (int64_t)h * p.P + p0;
+    const bf* q_rows = p.q + (int64_t)b * p.S * p.ld + (int64_t)g * p.N;
+    const bf* k_rows = p.k + (int64_t)b * p.S * p.ld + (int64_t)g * p.N;
+    const bf* v_rows = p.v + (int64_t)b * p.S * p.ld + (int64_t)h * p.P + p0;
     const int nc = p.N / 8, xc = pc / 8;
     const int64_t e_at = head * blocks * SC_TOK;
     const float* e_h[3] = {p.e0 + e_at, p.e1 + e_at, MEMORY ? p.e2 + e_at : nullptr};
@@ -145,9 +145,9 @@ recurrence_chunks_kernel(const __grid_constant__ RecurrenceParams p) {
         const int t0 = blk * SC_TOK;
         for (int r = warp; r < SC_TOK; r += SC_THR / 32) {    // a warp per token, lanes along its row
             const bool live = t0 + r < p.S;
-            const int64_t tok = live ? t0 + r : p.S - 1;
-            const bf* bsrc = k_rows + tok * p.k_ld;
-            const bf* csrc = q_rows + tok * p.q_ld;
+            const int64_t off = (int64_t)(live ? t0 + r : p.S - 1) * p.ld;
+            const bf* bsrc = k_rows + off;
+            const bf* csrc = q_rows + off;
             const uint32_t bd = saddr(b_s + (stage * SC_TOK + r) * ns), cd = saddr(c_s + (stage * SC_TOK + r) * ns);
             for (int c = lane; c < 2 * nc; c += 32) {
                 if (c < nc) cp16(bd + c * 16, bsrc + c * 8, live);
@@ -158,7 +158,7 @@ recurrence_chunks_kernel(const __grid_constant__ RecurrenceParams p) {
             const bool live = t0 + r < p.S;
             if ((tid & 3) < xc)
                 cp16(saddr(x_s + (stage * SC_TOK + r) * SC_PS + (tid & 3) * 8),
-                     v_rows + (int64_t)(live ? t0 + r : p.S - 1) * p.v_ld + (tid & 3) * 8, live);
+                     v_rows + (int64_t)(live ? t0 + r : p.S - 1) * p.ld + (tid & 3) * 8, live);
         }
 #pragma unroll
         for (int e = 0; e < NE; ++e) {
@@ -229,9 +229,9 @@ recurrence_chunks_kernel(const __grid_constant__ RecurrenceParams p) {
         const float* e1 = e_sh[1][stage];
         // exponent of a token's row factor, without the state's; of the last token: the state's own
         auto row_exp = [&](int t) { return MEMORY ? -fmaxf(m_in, e1[t]) : e0[t]; };
-        auto weight = [&](float row, int s) { return MEMORY ? exp2f(e0[s] + row) : exp2f(row - e0[s]) * e1[s]; };
+        auto weight = [&](float row, float c, float d) { return MEMORY ? exp2f(c + row) : exp2f(row - c) * d; };
         const float total = row_exp(SC_TOK - 1);
-        if (tid < SC_TOK) w_sh[tid] = weight(total, tid);
+        if (tid < SC_TOK) w_sh[tid] = weight(total, e0[tid], e1[tid]);
         // ---- C . B of 16 tokens x 32 keys, C . S of 16 tokens x 16 value columns
         float gacc[4][4], y[2][4];
 #pragma unroll
@@ -268,7 +268,7 @@ recurrence_chunks_kernel(const __grid_constant__ RecurrenceParams p) {
         const float row_r[2] = {row_exp(tr[0]), row_exp(tr[1])};
 #pragma unroll
         for (int k = 0; k < 2; ++k) {
-            const float f = exp2f(row_r[k] + m_in);
+            const float f = exp2f(MEMORY ? row_r[k] + m_in : row_r[k]);
 #pragma unroll
             for (int v = 0; v < 2; ++v) {
                 y[v][2 * k] *= f;
@@ -290,10 +290,11 @@ recurrence_chunks_kernel(const __grid_constant__ RecurrenceParams p) {
 #pragma unroll
                 for (int v = 0; v < 2; ++v) {
                     const int s = s0 + v * 8 + fc;
+                    const float c0 = e0[s], c1 = e0[s + 1], d0 = MEMORY ? 1.f : e1[s], d1 = MEMORY ? 1.f : e1[s + 1];
 #pragma unroll
                     for (int r = 0; r < 2; ++r) {
-                        const float w0 = s <= tr[r] ? gacc[2 * k + v][2 * r] * weight(row_r[r], s) : 0.f;
-                        const float w1 = s + 1 <= tr[r] ? gacc[2 * k + v][2 * r + 1] * weight(row_r[r], s + 1) : 0.f;
+                        const float w0 = s <= tr[r] ? gacc[2 * k + v][2 * r] * weight(row_r[r], c0, d0) : 0.f;
+                        const float w1 = s + 1 <= tr[r] ? gacc[2 * k + v][2 * r + 1] * weight(row_r[r], c1, d1) : 0.f;
                         split_bf16(w0, w1, a[0][2 * v + r], a[1][2 * v + r]);
                     }
                 }
@@ -352,7 +353,7 @@ recurrence_chunks_kernel(const __grid_constant__ RecurrenceParams p) {
             }
         }
         // ---- state: (weighted B)^T . x on top of the decayed state
-        const float f = exp2f(total + m_in);
+        const float f = exp2f(MEMORY ? total + m_in : total);
 #pragma unroll
         for (int u = 0; u < NM; ++u) {
             const int n0 = (warp + 8 * u) * 16;
@@ -441,7 +442,7 @@ int launch_ssm_chunks(const sk_ssm_params& p, cudaStream_t st) {
     r.v = x;
     r.k = x + I;
     r.q = r.k + p.G * p.N;
-    r.q_ld = r.k_ld = r.v_ld = p.xbc_ld;
+    r.ld = p.xbc_ld;
     r.y = (__nv_bfloat16*)p.y;
     r.state = p.state;
     r.skip = p.D;
@@ -478,7 +479,7 @@ int launch_mlstm_chunks(const sk_mlstm_params& p, cudaStream_t st) {
     r.q = (const __nv_bfloat16*)p.q;
     r.k = (const __nv_bfloat16*)p.k;
     r.v = (const __nv_bfloat16*)p.v;
-    r.q_ld = r.k_ld = r.v_ld = p.in_ld;
+    r.ld = p.in_ld;
     r.y = (__nv_bfloat16*)p.num;
     r.state = p.S_state;
     r.n_state = p.n_state;

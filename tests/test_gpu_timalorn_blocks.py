@@ -220,18 +220,23 @@ def test_window_and_capped_scores_of_a_portion(case, path):
 
 @pytest.mark.parametrize("path", ["rows32", "rows", "prefill_tc", "decode"])
 @pytest.mark.parametrize("size", [0.05, 1.0, 30.0])
-def test_score_cap_of_small_and_of_saturated_scores(size, path):
-    """Scores far below the cap (a polynomial in the tensor-core kernel), near it and far beyond it: with one key
-    made to lead by little, the weights depend on the capped difference."""
-    S, H, D, cap = 130, 1, 32, 10.0
+@pytest.mark.parametrize("cap", [10.0, 80.0])
+def test_score_cap_of_small_and_of_saturated_scores(cap, size, path):
+    """Scores far below the cap (a polynomial in the tensor-core kernel), near it and far beyond it, for a cap whose
+    exponentials need no running maximum and for one whose do."""
+    S, H, D = 130, 1, 32
     dtype = F32 if path == "rows32" else BF16
     S = 1 if path == "decode" else S
     k, v = _rand(130, 1, D, seed=1, dtype=dtype), _rand(130, 1, D, seed=2, dtype=dtype)
     q = _rand(S, H, D, seed=3, dtype=dtype)
     kw = dict(scale=size * cap / D ** 0.5 / 2, softcap=cap, start=130 - S)
-    got = ops.attn(q[None].to(DEV), k[None].to(DEV), v[None].to(DEV), path="rows" if path == "rows32" else path, **kw)
-    want = _plain_attention(q.to(D64), k.to(D64), v.to(D64), kw["scale"], kw["start"], 0, softcap=cap)
-    _close(got[0], want, dtype, tol16=8e-3)
+    for sink in (None, -60.0, cap - 1.0, 95.0):
+        s = None if sink is None else torch.full((1,), sink)
+        got = ops.attn(q[None].to(DEV), k[None].to(DEV), v[None].to(DEV), path="rows" if path == "rows32" else path,
+                       sink=None if s is None else s.to(DEV), **kw)
+        want = _plain_attention(q.to(D64), k.to(D64), v.to(D64), kw["scale"], kw["start"], 0, softcap=cap,
+                                sink=None if s is None else s.to(D64))
+        _close(got[0], want, dtype, tol16=8e-3, tol32=4e-5)
 
 
 DECODE = [
